@@ -86,7 +86,7 @@ class InlineRotarySpec(PartSpec):
     angle = position * base^(-2i/dims), computed in float32 inside the kernels (no position table,
     so no longest position).  `yarn` rescales the frequencies and magnifies cos and sin; `bands` rescales
     them by wavelength (short waves kept, long ones divided by the factor, a blend in between); at most one
-    of the two.
+    of the two.  `interleaved` pairs channel 2i with channel 2i + 1 instead (mixers that rotate that way say so).
     """
 
     kind: str = field(init=False, default="rotary_inline")
@@ -94,6 +94,7 @@ class InlineRotarySpec(PartSpec):
     base: float = 10000.0
     yarn: YarnScaling | None = None
     bands: Llama3Scaling | None = None
+    interleaved: bool = False
 
 
 @dataclass(frozen=True)
@@ -219,7 +220,11 @@ class GatedAttentionSpec(PartSpec):
     `weights` "sigmoid" makes a visible key's weight sigmoid(score) without any normalisation over
     the keys; `output_gate_scope` "head" gates with one number a head (`g` is [num_heads, hidden]);
     `chunk` n > 0 lets query i see key j only if floor(i / n) = floor(j / n), positions counted from the
-    request's first token; `softcap` c > 0 turns the scaled product into c tanh(q . k * scale / c).
+    request's first token; `softcap` c > 0 turns the scaled product into c tanh(q . k * scale / c);
+    `qk_norm_weight` False (scope "head" only): the norm of every head of q and k has no weight (such a norm is the
+    same before the rotation and after it); `values` "keys": the values are the keys as projected, before norm and
+    rotation, and there is no tensor `v`; `sink` s: a score s without a key or a value takes part in every softmax's
+    sum, so that the weights add up to less than one.
     """
 
     kind: str = field(init=False, default="gated_attention")
@@ -244,6 +249,9 @@ class GatedAttentionSpec(PartSpec):
     output_gate_scope: str = "channel"   # "channel": a gate a value channel; "head": one a head
     chunk: int = 0                       # 0: no chunks
     softcap: float = 0.0                 # 0: scores are not capped
+    qk_norm_weight: bool = True
+    values: str = "projected"            # "projected": by the tensor `v`; "keys": the keys as projected
+    sink: float | None = None            # None: no sink
 
 
 @dataclass(frozen=True)
@@ -285,6 +293,10 @@ class GatedDeltaRuleSpec(PartSpec):
     per head and key channel; each head's o is RMS-normed (weight shared by the heads) and multiplied
     by sigmoid(W_g2 W_g1 h).  The inner sizes of the two low-rank projections are the checkpoint's
     (`decay_rank`, `gate_rank` only serve to draw random weights).
+
+    `decay_scope` "head": one decay a head, a = exp(-exp(A_log) softplus(W_a h + dt_bias)) with tensors `a`
+    [heads, hidden] and `dt_bias` [heads] in place of a1, a2.  `gate` "silu": the heads are multiplied by silu(W_g h)
+    with one tensor `g` in place of g1, g2.
     """
 
     kind: str = field(init=False, default="gated_delta_rule")
@@ -299,6 +311,27 @@ class GatedDeltaRuleSpec(PartSpec):
     out_norm_eps: float = 1e-6
     decay_rank: int = 0
     gate_rank: int = 0
+    decay_scope: str = "channel"         # "channel": a decay a key channel, low-rank; "head": one a head
+    gate: str = "low_rank_sigmoid"       # or "silu"
+
+
+@dataclass(frozen=True)
+class TimeMixingSpec(PartSpec):
+    """
+    RWKV-style time mixing over a matrix state per request and head.  With h' the previous token's input (zeros for
+    the first), r, k, v, the gate and the decay each read a blend of their own, h + (h' - h) mu; the decay is
+    a = exp(-exp(W_w2 tanh(W_w1 m_w) + w0)) per head and channel;
+    o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, S_t = diag(a_t) S_(t-1) + k_t v_t^T; each head's o is RMS-normed, the
+    heads concatenated, multiplied by a weight over all heads and by silu(W_g m_g).  The inner size of the decay's
+    projection is the checkpoint's (`decay_rank` only serves to draw random weights).
+    """
+
+    kind: str = field(init=False, default="time_mixing")
+    hidden_size: int = 0
+    num_heads: int = 0
+    head_dim: int = 0                    # channels of r, k, v and the gate a head
+    decay_rank: int = 0
+    out_norm_eps: float = 1e-6
 
 
 @dataclass(frozen=True)
@@ -327,10 +360,15 @@ class ParallelMixerSpec(PartSpec):
     """
     Mixers side by side on one input: sum_b scale_b * mixer_b(h).  `branches` holds (mixer description,
     prefix of its tensors behind the mixer's own prefix, scale).  At most one branch keeps keys and values.
+    `norm_names` (one tensor name a branch; empty: none) norms each branch's output over the model width first:
+    sum_b scale_b * rms_norm(mixer_b(h)) * w_b.
     """
 
     kind: str = field(init=False, default="parallel")
     branches: tuple[tuple[PartSpec, str, float], ...] = ()
+    hidden_size: int = 0                 # with norms: the width they run over
+    norm_names: tuple[str, ...] = ()
+    norm_eps: float = 1e-6
 
 
 @dataclass(frozen=True)
@@ -408,20 +446,21 @@ class BlockSpec:
     live under.  `arrangement` picks the wiring (the registry of arrangements); "pre_norm" is
     x + mixer(norm(x)) followed by x + ffn(norm(x)) with the adds deferred into the next norm;
     "sandwich_norm" norms each sublayer's output as well, x + norm_b(mixer(norm(x))), around a
-    float32 residual stream; "pre_norm_stream" is "pre_norm" around a float32 residual stream.
+    float32 residual stream; "pre_norm_stream" is "pre_norm" around a float32 residual stream;
+    "post_norm_stream" norms the sublayers' outputs only, x + norm(mixer(x)), around a float32 stream.
     """
 
     arrangement: str
     mixer: PartSpec
     feed_forward: PartSpec | None    # None (arrangements that allow it): the block has no feed-forward
-    mixer_norm: PartSpec
+    mixer_norm: PartSpec | None      # None ("post_norm_stream"): the sublayers' inputs are not normed
     feed_forward_norm: PartSpec | None
     prefix: str                      # e.g. "model.layers.3."
     mixer_prefix: str = "self_attn."
     feed_forward_prefix: str = "mlp."
     mixer_norm_prefix: str = "input_layernorm."
     feed_forward_norm_prefix: str = "post_attention_layernorm."
-    # arrangements that also norm each sublayer's output ("sandwich_norm")
+    # arrangements that norm each sublayer's output ("sandwich_norm", "post_norm_stream")
     mixer_post_norm: PartSpec | None = None
     feed_forward_post_norm: PartSpec | None = None
     mixer_post_norm_prefix: str = ""

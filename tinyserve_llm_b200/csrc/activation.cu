@@ -89,7 +89,7 @@ __global__ void unary_activation_kernel(const T* __restrict__ x, T* __restrict__
 
 TS_API int ts_unary_activation_rows(const void* x, void* out, long long total, int kind, float a, float b, int dtype,
                                     cudaStream_t stream) {
-    TS_REQUIRE(total >= 0 && (kind == TS_UNARY_RELU2 || kind == TS_UNARY_XIELU), "unary_activation: bad arguments");
+    TS_REQUIRE(total >= 0 && kind >= TS_UNARY_RELU2 && kind <= TS_UNARY_LAST, "unary_activation: bad arguments");
     if (total == 0) return 0;
     const int vn = dtype == TS_F32 ? 4 : 8;
     const bool vec = total % vn == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)out % 16 == 0;

@@ -22,7 +22,8 @@
 // Options of the mask and of the score (ts_paged_attention_bf16_masked): chunks of n positions outside of
 // which a query sees nothing (it sees keys max(p - window + 1, floor(p / n) n) .. p); scores capped as
 // c tanh(q . k scale / c) before the softmax (the CAP form of the kernels); a value pool with fewer heads than
-// the key pool (key head j reads value head j / (key heads / value heads)) and a geometry of its own.
+// the key pool (key head j reads value head j / (key heads / value heads)) and a geometry of its own; a sink: a score
+// that takes part in the softmax's sum without a key or a value.
 #include "attention_bf16.h"
 
 #include "common.cuh"
@@ -238,6 +239,7 @@ struct AttnParams {
     int value_group;           // key heads a value head (1: as many value heads as key heads)
     KVGeometry geo_v;          // the value pool's geometry
     const int* prefill_seqs;   // requests that feed more than one token, for the prefill grid (-1: none); null: every request
+    float sink2;               // the sink's score times log2(e) (-inf: no sink)
     // decode only
     float* partial_o;      // [seq][head][split][HD]
     float* partial_ml;     // [seq][head][split][2]
@@ -344,6 +346,7 @@ __global__ void __launch_bounds__(128) prefill_attention_kernel(AttnParams p) {
     for (int r = 0; r < 2; ++r) {
         st.l[r] += __shfl_xor_sync(0xffffffffu, st.l[r], 1);
         st.l[r] += __shfl_xor_sync(0xffffffffu, st.l[r], 2);
+        if (!SIG && p.sink2 > -INFINITY) st.l[r] += fast_exp2_any(p.sink2 - st.m[r]);   // +inf where every score is far below it
     }
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
@@ -579,6 +582,7 @@ __global__ void __launch_bounds__(GROUPS * HD) decode_combine_kernel(AttnParams 
         l += group_ml[g].y * f;
         o += group_o[g][d] * f;
     }
+    if (!SIG && p.sink2 > -INFINITY) l += fast_exp2_any(p.sink2 - top);
     p.out[((long long)q_begin * p.nh + head) * HD + d] =
         __float2bfloat16_rn(SIG ? o * head_gate(p, q_begin, head) : (l > 0.f ? o / l : 0.f));
 }
@@ -637,7 +641,7 @@ int run(const void* q, long long q_stride, void* out, const void* k_pool, const 
         float scale, int window, float* scratch, long long scratch_floats, const int* prefill_seqs, int num_prefill_seqs,
         bool sigmoid, const float* slopes, const float* head_bias, const void* gate, long long gate_stride,
         cudaStream_t stream, int chunk = 0, float softcap = 0.f, int value_heads = 0, long long v_page_stride = -1,
-        long long v_entry_offset = -1) {
+        long long v_entry_offset = -1, float sink = -INFINITY) {
     TS_REQUIRE(ts_attention_bf16_supported(hd, page_tokens, nh, nkv),
                "paged_attention_bf16: head_dim %d / page %d / heads %d:%d is not taken by the tensor-core kernels", hd,
                page_tokens, nh, nkv);
@@ -670,6 +674,7 @@ int run(const void* q, long long q_stride, void* out, const void* k_pool, const 
     p.cap_pre = softcap > 0.f ? scale / softcap : 0.f;
     p.window = window;
     p.chunk = chunk;
+    p.sink2 = sink > -INFINITY ? sink * LOG2E : -INFINITY;
     p.value_group = value_heads > 0 ? nkv / value_heads : 1;
     p.geo_v = v_page_stride >= 0 ? KVGeometry{v_page_stride, v_entry_offset, page_tokens, num_pages} : p.geo;
     p.max_splits = (max_ctx_len + SPLIT - 1) / SPLIT;
@@ -726,7 +731,8 @@ TS_API int ts_paged_attention_bf16_sigmoid(const void* q, long long q_stride, vo
 }
 
 // Softmax attention with the options of the mask and of the score: chunks, capped scores, a value pool of
-// `value_heads` heads (0: as many as key heads) with a geometry of its own.  Queries in a matrix of their own.
+// `value_heads` heads (0: as many as key heads) with a geometry of its own, a sink (a score without a key or a value
+// in the softmax's sum; -inf: none).  Queries in a matrix of their own.
 TS_API int ts_paged_attention_bf16_masked(const void* q, long long q_stride, void* out, const void* k_pool,
                                           const void* v_pool, long long page_stride, long long entry_offset,
                                           long long v_page_stride, long long v_entry_offset, int page_tokens, int num_pages,
@@ -734,10 +740,10 @@ TS_API int ts_paged_attention_bf16_masked(const void* q, long long q_stride, voi
                                           int num_seqs, int max_q_len, int min_q_len, int max_ctx_len, int nh, int nkv,
                                           int hd, float scale, int window, int chunk, float softcap, int value_heads,
                                           float* scratch, long long scratch_floats, const int* prefill_seqs,
-                                          int num_prefill_seqs, cudaStream_t stream) {
+                                          int num_prefill_seqs, float sink, cudaStream_t stream) {
     TS_REQUIRE(q_stride % 8 == 0 && (uintptr_t)q % 16 == 0, "paged_attention_bf16: query rows must start on 16-byte boundaries");
     return run(q, q_stride, out, k_pool, v_pool, page_stride, entry_offset, page_tokens, num_pages, block_table, table_width,
                cu_q, ctx_lens, num_seqs, max_q_len, min_q_len, max_ctx_len, nh, nkv, hd, scale, window, scratch,
                scratch_floats, prefill_seqs, num_prefill_seqs, false, nullptr, nullptr, nullptr, 0, stream, chunk, softcap,
-               value_heads, v_page_stride, v_entry_offset);
+               value_heads, v_page_stride, v_entry_offset, sink);
 }

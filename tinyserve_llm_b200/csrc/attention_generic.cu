@@ -18,6 +18,7 @@
 //   softcap c > 0: the scaled product becomes c tanh(q_i . k_j * scale / c) before the other terms
 //   chunk n > 0: a query also sees no key before floor(i / n) * n (positions count from the request's first token)
 //   out_f32: the output is written in float32 whatever the activation dtype
+//   sink: a score that takes part in the softmax's sum without a value (-inf: none); rows then sum to less than one
 //   value_heads g > 0: the value pool holds g heads (a divisor of nkv), head h reads value head h / (nh / g): several
 //     key heads, each with query heads of its own, over one set of values
 #include "common.cuh"
@@ -31,6 +32,7 @@ struct AttentionExtras {
     int chunk;                 // 0: none
     int value_heads;           // 0: as many as key heads
     int out_f32;               // 1: `out` is float32 whatever the activation dtype
+    float sink;                // a score without a value in the softmax's sum (-inf: none)
 };
 
 template <typename T>
@@ -153,9 +155,10 @@ paged_attention_generic_kernel(const T* __restrict__ q, long long q_stride, T* _
     // merge the lanes
     float f = 1.f, inv = 1.f;
     if (!SIGMOID) {
-        const float m_all = warp_max(m);
+        const float m_all = fmaxf(warp_max(m), extras.sink);
         f = (m == -INFINITY) ? 0.f : expf(m - m_all);
-        const float l_all = warp_sum(l * f);
+        float l_all = warp_sum(l * f);
+        if (extras.sink > -INFINITY) l_all += expf(extras.sink - m_all);
         inv = l_all > 0.f ? 1.f / l_all : 0.f;
     }
     if (extras.gate)
@@ -205,8 +208,8 @@ TS_API int ts_paged_attention_scored(const void* q, long long q_stride, void* ou
                                      int table_width, const int* positions, const int* seq_of_token, int num_tokens,
                                      int nh, int nkv, int hd, int vd, float scale, int window, int dtype, int sigmoid,
                                      const float* slopes, const float* head_bias, const void* gate, long long gate_stride,
-                                     float softcap, int chunk, int value_heads, int out_f32, cudaStream_t stream) {
-    const AttentionExtras extras{slopes, head_bias, gate, gate_stride, softcap, chunk, value_heads, out_f32};
+                                     float softcap, int chunk, int value_heads, int out_f32, float sink, cudaStream_t stream) {
+    const AttentionExtras extras{slopes, head_bias, gate, gate_stride, softcap, chunk, value_heads, out_f32, sink};
     TS_REQUIRE(softcap >= 0.f && chunk >= 0 && value_heads >= 0, "paged_attention: bad softcap, chunk or value heads");
     TS_REQUIRE(value_heads == 0 || (nkv % value_heads == 0 && nh % value_heads == 0),
                "paged_attention: %d value heads do not divide %d key heads", value_heads, nkv);
@@ -244,7 +247,7 @@ TS_API int ts_paged_attention_split(const void* q, long long q_stride, void* out
     return ts_paged_attention_scored(q, q_stride, out, k_pool, v_pool, page_stride, entry_offset, v_page_stride,
                                      v_entry_offset, page_tokens, num_pages, block_table, table_width, positions,
                                      seq_of_token, num_tokens, nh, nkv, hd, vd, scale, window, dtype, 0, nullptr, nullptr,
-                                     nullptr, 0, 0.f, 0, 0, 0, stream);
+                                     nullptr, 0, 0.f, 0, 0, 0, -INFINITY, stream);
 }
 
 // Queries, keys and values of one head size in the columns [q | k | v] of one projection's output.

@@ -216,6 +216,7 @@ struct FlashParams {
     int chunk;                        // n > 0: a query sees no key before floor(p / n) * n
     float cap_pre;                    // scores are capped: tanh(product * cap_pre), and scale_log2 is cap * log2(e); 0: not capped
     int value_heads;                  // heads of the value pool (a divisor of nkv)
+    float sink2;                      // a score (times log2(e)) that joins the softmax's sum without a key or a value; -inf: none
     // keys and values in matrices of their own instead of pages: [rows, nkv * HD], request s's key j in row kv_start[s] + j
     const int* kv_start;              // null: keys and values come from the paged pools
 };
@@ -572,6 +573,7 @@ __global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(c
             half_sum[half][r] = l_run;
             pair_barrier(quadrant);
             l_run += half_sum[half ^ 1][r];
+            if (p.sink2 > -INFINITY) l_run += fast_exp2_any(p.sink2 - m_run);    // +inf where every score is far below it
         }
         if (ok && !failed) {                         // every thread of the warp takes part in the loads; only real rows store
             float inv = l_run > 0.f ? 1.f / l_run : 0.f;
@@ -649,7 +651,7 @@ int run_prefill(const void* q, long long q_cols, long long q_stride, void* out, 
                 float scale, const int* prefill_seqs, int num_prefill_seqs, int* error, bool sigmoid, int window,
                 const float* slopes, const float* head_bias, const void* gate, long long gate_stride, cudaStream_t stream,
                 bool bounded = false, int chunk = 0, float softcap = 0.f, int value_heads = 0, const int* kv_start = nullptr,
-                long long dense_rows = 0) {
+                long long dense_rows = 0, float sink = -INFINITY) {
     TS_REQUIRE(ts_attention_tcgen05_supported(hd, page_tokens, nh, nkv, 0), "attention_tcgen05: sizes not taken (head_dim %d, page %d)", hd, page_tokens);
     TS_REQUIRE(sigmoid || bounded || window == 0, "attention_tcgen05: the plain form takes no window");
     TS_REQUIRE(window >= 0 && chunk >= 0 && softcap >= 0.f, "attention_tcgen05: a negative window, chunk or cap");
@@ -693,6 +695,7 @@ int run_prefill(const void* q, long long q_cols, long long q_stride, void* out, 
     p.cap_pre = softcap > 0.f ? scale / softcap : 0.f;
     p.chunk = chunk;
     p.value_heads = value_heads;
+    p.sink2 = sink > -INFINITY ? sink * LOG2E : -INFINITY;
     p.kv_start = kv_start;
     p.error = error;
     p.window = window;
@@ -753,19 +756,21 @@ TS_API int ts_prefill_attention_tcgen05_sigmoid(const void* q, long long q_strid
 
 // Softmax attention behind a mask with a lower bound: query i sees keys max(i - window + 1, floor(i / chunk) chunk) .. i
 // (0: no such bound); `softcap` c > 0 turns the scaled product into c tanh(. / c); the value pool holds `value_heads`
-// heads (0: as many as key heads; key head j reads value head j / (nkv / value_heads)) in the same pages and entries.
-// Queries [T, nh * hd] in a matrix of their own, q_stride elements a row.
+// heads (0: as many as key heads; key head j reads value head j / (nkv / value_heads)) in the same pages and entries;
+// `sink` is a score that joins the softmax's sum without a key or a value (-inf: none).  With a sink and no bound, cap or
+// shared values, the plain form of the kernel runs.  Queries [T, nh * hd] in a matrix of their own, q_stride elements a row.
 TS_API int ts_prefill_attention_tcgen05_masked(const void* q, long long q_stride, void* out, const void* k_pool,
                                                const void* v_pool, int num_pages, int entries, int entry, int page_tokens,
                                                const int* block_table, int table_width, const int* cu_q,
                                                const int* ctx_lens, int num_seqs, int num_tokens, int max_q_len, int nh,
                                                int nkv, int hd, float scale, int window, int chunk, float softcap,
                                                int value_heads, const int* prefill_seqs, int num_prefill_seqs, int* error,
-                                               cudaStream_t stream) {
+                                               float sink, cudaStream_t stream) {
+    const bool bounded = window > 0 || chunk > 0 || softcap > 0.f || (value_heads > 0 && value_heads != nkv);
     return run_prefill(q, (long long)nh * hd, q_stride, out, k_pool, v_pool, num_pages, entries, entry, page_tokens,
                        block_table, table_width, cu_q, ctx_lens, num_seqs, num_tokens, max_q_len, nh, nkv, hd, scale,
-                       prefill_seqs, num_prefill_seqs, error, false, window, nullptr, nullptr, nullptr, 0, stream, true, chunk,
-                       softcap, value_heads);
+                       prefill_seqs, num_prefill_seqs, error, false, window, nullptr, nullptr, nullptr, 0, stream, bounded,
+                       chunk, softcap, value_heads, nullptr, 0, sink);
 }
 
 // Causal softmax attention of prompt portions over keys and values that lie in matrices of their own,

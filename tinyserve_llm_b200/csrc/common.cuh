@@ -70,11 +70,13 @@ __device__ __forceinline__ float ts_gated_activation(int kind, float g, float u,
 }
 
 // Activations of one argument, act(z) with two numbers a, b of the layer:  0: relu(z)^2;
-// 1 (xIELU): a z^2 + z/2 for z > 0, b (exp(z) - 1 - z) + z/2 for z <= 0 (the host gives a = softplus(p), b = 1/2 + softplus(q)).
-enum { TS_UNARY_RELU2 = 0, TS_UNARY_XIELU = 1 };
+// 1 (xIELU): a z^2 + z/2 for z > 0, b (exp(z) - 1 - z) + z/2 for z <= 0 (the host gives a = softplus(p), b = 1/2 + softplus(q));
+// 2: tanh(z).
+enum { TS_UNARY_RELU2 = 0, TS_UNARY_XIELU = 1, TS_UNARY_TANH = 2, TS_UNARY_LAST = TS_UNARY_TANH };
 
 __device__ __forceinline__ float ts_unary_activation(int kind, float z, float a, float b) {
     if (kind == TS_UNARY_XIELU) return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
+    if (kind == TS_UNARY_TANH) return tanhf(z);
     const float r = fmaxf(z, 0.f);
     return r * r;
 }

@@ -22,10 +22,16 @@
 // A second kernel norms each head's o over the value channels (with or without a weight),
 // multiplies by silu(gate) or sigmoid(gate) and rounds to the activation dtype for the output projection.
 //
-// The scan also runs the delta rule (`beta` given):
+// The scan also runs the delta rule:
 //   S <- diag(a_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
 // where the read S^T k_t feeds back into the state, so the sixteen threads that share a column of S
 // are lanes of one warp and add up their shares with shuffles, token by token.
+// Its decay may also be one number per token and head; then S^T k is taken of the state before the decay and
+// multiplied by it, so that the decay is off the chain from token to token.
+// A third form reads the state before the token's own write and weighs that write by a bonus u per channel:
+//   o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t,   S_t = diag(a_t) S_(t-1) + k_t v_t^T
+// of which sum_i u_i k_i q_i, one number per token and head, arrives prepared (`coef`) and multiplies v_t.
+// q and k may belong to several value heads each (`qk_group`: value heads a q/k head).
 // A value column past `v_cols` is the constant 1: with it the state carries the sum of the (decayed)
 // keys beside the matrix, and o's extra column is that sum's product with q (the normaliser of a
 // matrix memory with exponential gates).  The inputs of these variants are prepared by kernels of
@@ -71,11 +77,16 @@ __global__ void recurrence_prepare_kernel(const T* __restrict__ q, const T* __re
     }
 }
 
+enum { LR_PLAIN = 0, LR_DELTA = 1, LR_DELTA_HEAD = 2, LR_BONUS = 3 };
+
 struct RecurrenceArgs {
-    const float* prepared; long long total;           // [3][tokens, heads * dim]: q, k, decay as they enter the recurrence
+    const float* qk; long long qk_total;              // [2][tokens, heads / qk_group * dim]: q, k as they enter the recurrence
+    int qk_group;
+    const float* decay;                               // [tokens, heads * dim]; LR_DELTA_HEAD: [tokens, heads]
     const void* v; long long v_stride;                // elements between tokens; a head's values start at h * v_cols
     int v_cols;                                       // value columns read from v; columns from here to vdim are 1
-    const float* beta;                                // [tokens, heads]: the delta rule's step size (null: plain recurrence)
+    const float* coef;                                // [tokens, heads]: the delta rule's step size, or the bonus form's
+                                                      // sum of u k q; null: plain recurrence
     const int* cu_q; const int* slots;
     float* state; long long slot_stride;              // floats between slots; a slot holds [heads, dim, vdim]
     float* out;                                       // [tokens, heads * vdim] float32
@@ -84,12 +95,13 @@ struct RecurrenceArgs {
 
 // COLS: value channels of a CTA (16; the delta rule, whose tokens are a chain of dependent steps, runs 8 a CTA so that
 // a prompt alone spreads over twice the SMs)
-template <typename T, int MAXM, bool DELTA, int COLS>
+template <typename T, int MAXM, int MODE, int COLS>
 __global__ void __launch_bounds__(LR_ROWGROUPS * COLS)
 linear_recurrence_kernel(RecurrenceArgs p) {
     // staged rows are padded with zeros to LR_ROWGROUPS * MAXM channels: the inner loop needs no bound and reads
     // four channels a load
     constexpr int PITCH = LR_ROWGROUPS * MAXM;
+    constexpr bool DELTA = MODE == LR_DELTA || MODE == LR_DELTA_HEAD, HEADA = MODE == LR_DELTA_HEAD, COEF = MODE != LR_PLAIN;
     extern __shared__ __align__(16) float smem[];
     const int dim = p.dim, vdim = p.vdim;
     float* q_s = smem;                                   // [LR_TILE][PITCH]
@@ -97,7 +109,8 @@ linear_recurrence_kernel(RecurrenceArgs p) {
     float* a_s = k_s + LR_TILE * PITCH;
     float* v_s = a_s + LR_TILE * PITCH;                  // [LR_TILE][COLS]
     float* part = v_s + LR_TILE * COLS;               // [LR_TILE][LR_ROWGROUPS][COLS]
-    float* b_s = part + LR_TILE * LR_ROWGROUPS * COLS; // [LR_TILE] (delta rule)
+    float* b_s = part + LR_TILE * LR_ROWGROUPS * COLS; // [LR_TILE] (delta rule, bonus)
+    float* ha_s = b_s + LR_TILE;                      // [LR_TILE] (one decay a head)
     const int seq = blockIdx.z, h = blockIdx.y, j0 = blockIdx.x * COLS;
     const int slot = p.slots[seq];
     const int begin = p.cu_q[seq], end = p.cu_q[seq + 1];
@@ -121,13 +134,14 @@ linear_recurrence_kernel(RecurrenceArgs p) {
         S[m] = (live && i < dim) ? st[(long long)i * vdim + j] : 0.f;
     }
     const T* v = (const T*)p.v;
-    const long long row_width = (long long)p.heads * dim;
+    const long long row_width = (long long)p.heads * dim, qk_width = row_width / p.qk_group;
+    const int qk_head = h / p.qk_group;
     // What a tile needs from global memory is asked for one tile ahead and held in registers while the tile
     // before it is worked on.
     constexpr int ROUNDS = LR_TILE * PITCH / (LR_ROWGROUPS * COLS);
     float raw_q[ROUNDS], raw_k[ROUNDS], raw_a[ROUNDS];
     T raw_v;                                             // as loaded: converting would wait for the load
-    float raw_b = 0.f;
+    float raw_b = 0.f, raw_h = 0.f;
     auto fetch = [&](int t0, int n) {
 #pragma unroll
         for (int round = 0; round < ROUNDS; ++round) {
@@ -135,16 +149,20 @@ linear_recurrence_kernel(RecurrenceArgs p) {
             const int tt = e / PITCH, i = e % PITCH;
             raw_q[round] = raw_k[round] = raw_a[round] = 0.f;
             if (tt < n && i < dim) {
-                const long long at = (long long)(t0 + tt) * row_width + (long long)h * dim + i;
-                raw_q[round] = p.prepared[at];
-                raw_k[round] = p.prepared[p.total + at];
-                raw_a[round] = p.prepared[2 * p.total + at];
+                const long long at = (long long)(t0 + tt) * qk_width + (long long)qk_head * dim + i;
+                raw_q[round] = p.qk[at];
+                raw_k[round] = p.qk[p.qk_total + at];
+                if (!HEADA) raw_a[round] = p.decay[(long long)(t0 + tt) * row_width + (long long)h * dim + i];
             }
         }
         const int tt = threadIdx.x / COLS, c = threadIdx.x % COLS;       // LR_TILE * COLS = one value a thread
         raw_v = from_float<T>(j0 + c >= p.v_cols && j0 + c < vdim ? 1.f : 0.f);
         if (tt < n && j0 + c < p.v_cols) raw_v = v[(long long)(t0 + tt) * p.v_stride + (long long)h * p.v_cols + j0 + c];
-        if (DELTA && threadIdx.x < LR_TILE) raw_b = threadIdx.x < n ? p.beta[(long long)(t0 + threadIdx.x) * p.heads + h] : 0.f;
+        if (COEF && threadIdx.x < LR_TILE) {
+            const bool ok = threadIdx.x < n;
+            raw_b = ok ? p.coef[(long long)(t0 + threadIdx.x) * p.heads + h] : 0.f;
+            if (HEADA) raw_h = ok ? p.decay[(long long)(t0 + threadIdx.x) * p.heads + h] : 0.f;
+        }
     };
     fetch(begin, min(LR_TILE, end - begin));
     for (int t0 = begin; t0 < end; t0 += LR_TILE) {
@@ -155,10 +173,13 @@ linear_recurrence_kernel(RecurrenceArgs p) {
             const int e = round * (LR_ROWGROUPS * COLS) + threadIdx.x;
             q_s[e] = raw_q[round];
             k_s[e] = raw_k[round];
-            a_s[e] = raw_a[round];
+            if (!HEADA) a_s[e] = raw_a[round];
         }
         v_s[threadIdx.x] = to_float<T>(raw_v);
-        if (DELTA && threadIdx.x < LR_TILE) b_s[threadIdx.x] = raw_b;
+        if (COEF && threadIdx.x < LR_TILE) {
+            b_s[threadIdx.x] = raw_b;
+            if (HEADA) ha_s[threadIdx.x] = raw_h;
+        }
         if (t0 + LR_TILE < end) fetch(t0 + LR_TILE, min(LR_TILE, end - t0 - LR_TILE));   // under way during this tile's work
         __syncthreads();
         if (DELTA) {
@@ -166,22 +187,27 @@ linear_recurrence_kernel(RecurrenceArgs p) {
             // token needs from shared memory is loaded one token ahead, so that the chain waits for nothing else; its
             // sums are kept in four pieces so that no piece waits for more than MAXM / 4 products.
             float4 kc[MAXM / 4], ac4[MAXM / 4], qc[MAXM / 4];
-            float vc, bc;
+            float vc, bc, hc;
             auto load_token = [&](int tt, float4 (&k4)[MAXM / 4], float4 (&a4)[MAXM / 4], float4 (&q4)[MAXM / 4], float& vv,
-                                  float& bb) {
+                                  float& bb, float& hh) {
                 const float4* qt = reinterpret_cast<const float4*>(q_s + tt * PITCH + first);
                 const float4* kt = reinterpret_cast<const float4*>(k_s + tt * PITCH + first);
                 const float4* at = reinterpret_cast<const float4*>(a_s + tt * PITCH + first);
 #pragma unroll
-                for (int m4 = 0; m4 < MAXM / 4; ++m4) { k4[m4] = kt[m4 * STEP4]; a4[m4] = at[m4 * STEP4]; q4[m4] = qt[m4 * STEP4]; }
+                for (int m4 = 0; m4 < MAXM / 4; ++m4) {
+                    k4[m4] = kt[m4 * STEP4];
+                    if (!HEADA) a4[m4] = at[m4 * STEP4];
+                    q4[m4] = qt[m4 * STEP4];
+                }
                 vv = v_s[tt * COLS + jj];
                 bb = b_s[tt];
+                hh = HEADA ? ha_s[tt] : 1.f;
             };
-            load_token(0, kc, ac4, qc, vc, bc);
+            load_token(0, kc, ac4, qc, vc, bc, hc);
             for (int tt = 0; tt < n; ++tt) {
                 float4 kn[MAXM / 4], an[MAXM / 4], qn[MAXM / 4];
-                float vn, bn;
-                load_token(min(tt + 1, LR_TILE - 1), kn, an, qn, vn, bn);      // the tile's last row again: not used
+                float vn, bn, hn;
+                load_token(min(tt + 1, LR_TILE - 1), kn, an, qn, vn, bn, hn);      // the tile's last row again: not used
                 float rd[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int m4 = 0; m4 < MAXM / 4; ++m4) {
@@ -190,14 +216,18 @@ linear_recurrence_kernel(RecurrenceArgs p) {
 #pragma unroll
                     for (int c = 0; c < 4; ++c) {
                         const int m = 4 * m4 + c;
-                        S[m] *= aa[c];
+                        if (!HEADA) S[m] *= aa[c];
                         rd[c] = fmaf(S[m], kk[c], rd[c]);
                     }
                 }
                 float read = (rd[0] + rd[1]) + (rd[2] + rd[3]);
 #pragma unroll
                 for (int o = LR_ROWGROUPS / 2; o > 0; o >>= 1) read += __shfl_xor_sync(0xffffffffu, read, o);
-                const float u = bc * (vc - read);
+                if (HEADA) {                              // beside the shuffles: nothing of the read waits for it
+#pragma unroll
+                    for (int m = 0; m < MAXM; ++m) S[m] *= hc;
+                }
+                const float u = bc * (vc - hc * read);    // hc is 1 where the decay is already in the state
                 float ac[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int m4 = 0; m4 < MAXM / 4; ++m4) {
@@ -215,6 +245,7 @@ linear_recurrence_kernel(RecurrenceArgs p) {
                 for (int m4 = 0; m4 < MAXM / 4; ++m4) { kc[m4] = kn[m4]; ac4[m4] = an[m4]; qc[m4] = qn[m4]; }
                 vc = vn;
                 bc = bn;
+                hc = hn;
             }
         } else {
             // no thread waits for another here; a token's staged inputs are loaded one token ahead of their use
@@ -241,8 +272,9 @@ linear_recurrence_kernel(RecurrenceArgs p) {
 #pragma unroll
                     for (int c = 0; c < 4; ++c) {
                         const int m = 4 * m4 + c;
+                        if (MODE == LR_BONUS) acc = fmaf(S[m], qq[c], acc);      // the state before this token's write
                         S[m] = fmaf(aa[c], S[m], kk[c] * vc);
-                        acc = fmaf(S[m], qq[c], acc);
+                        if (MODE != LR_BONUS) acc = fmaf(S[m], qq[c], acc);
                     }
                 }
                 part[(tt * LR_ROWGROUPS + r) * COLS + jj] = acc;
@@ -258,6 +290,7 @@ linear_recurrence_kernel(RecurrenceArgs p) {
             float o = 0.f;
 #pragma unroll
             for (int g = 0; g < LR_ROWGROUPS; ++g) o += part[(tt * LR_ROWGROUPS + g) * COLS + c];
+            if (MODE == LR_BONUS) o = fmaf(b_s[tt], v_s[tt * COLS + c], o);
             p.out[(long long)(t0 + tt) * p.heads * vdim + (long long)h * vdim + j0 + c] = o;
         }
     }
@@ -269,49 +302,54 @@ linear_recurrence_kernel(RecurrenceArgs p) {
 }
 
 template <typename T>
-static int launch_recurrence(const RecurrenceArgs& p, int num_seqs, cudaStream_t stream) {
-#define TS_RECURRENCE(MAXM, DELTA, COLS)                                                                           \
+static int launch_recurrence(const RecurrenceArgs& p, int mode, int num_seqs, cudaStream_t stream) {
+#define TS_RECURRENCE(MAXM, MODE, COLS)                                                                            \
     do {                                                                                                           \
         const dim3 grid((p.vdim + COLS - 1) / COLS, p.heads, num_seqs);                                            \
         const size_t smem = (size_t)(3 * LR_TILE * LR_ROWGROUPS * MAXM + LR_TILE * COLS +                          \
-                                     LR_TILE * LR_ROWGROUPS * COLS + LR_TILE) * sizeof(float);                     \
+                                     LR_TILE * LR_ROWGROUPS * COLS + 2 * LR_TILE) * sizeof(float);                 \
         if (smem > 48 * 1024)                                                                                      \
-            cudaFuncSetAttribute(linear_recurrence_kernel<T, MAXM, DELTA, COLS>,                                   \
+            cudaFuncSetAttribute(linear_recurrence_kernel<T, MAXM, MODE, COLS>,                                    \
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                          \
-        linear_recurrence_kernel<T, MAXM, DELTA, COLS><<<grid, LR_ROWGROUPS * COLS, smem, stream>>>(p);            \
+        linear_recurrence_kernel<T, MAXM, MODE, COLS><<<grid, LR_ROWGROUPS * COLS, smem, stream>>>(p);            \
     } while (0)
-    if (p.beta) {
-        if (p.dim <= 4 * LR_ROWGROUPS) TS_RECURRENCE(4, true, 8);
-        else if (p.dim <= 8 * LR_ROWGROUPS) TS_RECURRENCE(8, true, 8);
-        else TS_RECURRENCE(16, true, 16);
-    } else {
-        if (p.dim <= 4 * LR_ROWGROUPS) TS_RECURRENCE(4, false, 16);
-        else if (p.dim <= 8 * LR_ROWGROUPS) TS_RECURRENCE(8, false, 16);
-        else TS_RECURRENCE(16, false, 16);
-    }
+#define TS_RECURRENCE_SIZES(MODE, COLS)                                                                            \
+    do {                                                                                                           \
+        if (p.dim <= 4 * LR_ROWGROUPS) TS_RECURRENCE(4, MODE, COLS);                                               \
+        else if (p.dim <= 8 * LR_ROWGROUPS) TS_RECURRENCE(8, MODE, COLS);                                          \
+        else TS_RECURRENCE(16, MODE, 16);                                                                          \
+    } while (0)
+    if (mode == LR_DELTA) TS_RECURRENCE_SIZES(LR_DELTA, 8);
+    else if (mode == LR_DELTA_HEAD) TS_RECURRENCE_SIZES(LR_DELTA_HEAD, 8);
+    else if (mode == LR_BONUS) TS_RECURRENCE_SIZES(LR_BONUS, 16);
+    else TS_RECURRENCE_SIZES(LR_PLAIN, 16);
+#undef TS_RECURRENCE_SIZES
 #undef TS_RECURRENCE
     TS_LAUNCH_CHECK("linear_recurrence");
     return 0;
 }
 
-// The scan alone, from inputs a kernel of the caller's prepared: prepared [3][tokens, heads * dim] float32
-// (q, k and the decay as they enter the recurrence), v [tokens, heads * v_cols] in float32 or the activation
-// dtype, beta [tokens, heads] or null.  A slot holds [heads, dim, vdim] floats.
-TS_API int ts_recurrence_scan(const float* prepared, const void* v, long long v_stride, int v_cols, int v_dtype,
-                              const float* beta, const int* cu_q, const int* slots, int num_seqs, float* state,
-                              long long slot_stride, float* out, int heads, int dim, int vdim, int num_tokens,
-                              cudaStream_t stream) {
+// The scan alone, from inputs a kernel of the caller's prepared: qk [2][tokens, heads / qk_group * dim] float32
+// (q and k as they enter the recurrence), decay [tokens, heads * dim], v [tokens, heads * v_cols] in float32 or the
+// activation dtype.  `mode` 0: plain; 1: delta rule with the step sizes `coef` [tokens, heads]; 2: the same with the
+// decay [tokens, heads]; 3: bonus form with `coef` [tokens, heads].  A slot holds [heads, dim, vdim] floats.
+TS_API int ts_recurrence_scan(const float* qk, int qk_group, const float* decay, int mode, const void* v,
+                              long long v_stride, int v_cols, int v_dtype, const float* coef, const int* cu_q,
+                              const int* slots, int num_seqs, float* state, long long slot_stride, float* out, int heads,
+                              int dim, int vdim, int num_tokens, cudaStream_t stream) {
     TS_REQUIRE(heads > 0 && dim > 0 && vdim > 0 && num_seqs >= 0 && num_tokens >= 0, "recurrence_scan: bad sizes");
     TS_REQUIRE(dim <= 16 * LR_ROWGROUPS, "recurrence_scan: %d key channels a head are not supported (up to %d)", dim,
                16 * LR_ROWGROUPS);
     TS_REQUIRE(v_cols >= 0 && v_cols <= vdim, "recurrence_scan: %d of %d value columns", v_cols, vdim);
+    TS_REQUIRE(mode >= LR_PLAIN && mode <= LR_BONUS && (mode == LR_PLAIN || coef), "recurrence_scan: mode %d", mode);
+    TS_REQUIRE(qk_group > 0 && heads % qk_group == 0, "recurrence_scan: %d heads in groups of %d", heads, qk_group);
     TS_REQUIRE(slot_stride >= (long long)heads * dim * vdim, "recurrence_scan: a state slot is too small");
     TS_REQUIRE(num_seqs <= 65535 && heads <= 65535, "recurrence_scan: grid too large");
     if (num_seqs == 0 || num_tokens == 0) return 0;
-    const long long total = (long long)num_tokens * heads * dim;
-    RecurrenceArgs p{prepared, total, v, v_stride, v_cols, beta, cu_q, slots, state, slot_stride, out, heads, dim, vdim};
-    if (v_dtype == TS_F32) return launch_recurrence<float>(p, num_seqs, stream);
-    if (v_dtype == TS_BF16) return launch_recurrence<__nv_bfloat16>(p, num_seqs, stream);
+    RecurrenceArgs p{qk, (long long)num_tokens * (heads / qk_group) * dim, qk_group, decay, v, v_stride, v_cols, coef, cu_q,
+                     slots, state, slot_stride, out, heads, dim, vdim};
+    if (v_dtype == TS_F32) return launch_recurrence<float>(p, mode, num_seqs, stream);
+    if (v_dtype == TS_BF16) return launch_recurrence<__nv_bfloat16>(p, mode, num_seqs, stream);
     return ts_fail("recurrence_scan: unknown dtype code %d", v_dtype);
 }
 
@@ -344,9 +382,10 @@ TS_API int ts_linear_recurrence(const void* q, const void* k, const void* v, lon
     else
         return ts_fail("linear_recurrence: unknown dtype code %d", dtype);
     TS_LAUNCH_CHECK("linear_recurrence (prepare)");
-    RecurrenceArgs p{prepared, total, v, v_stride, vdim, nullptr, cu_q, slots, state, slot_stride, out, heads, dim, vdim};
-    if (dtype == TS_F32) return launch_recurrence<float>(p, num_seqs, stream);
-    return launch_recurrence<__nv_bfloat16>(p, num_seqs, stream);
+    RecurrenceArgs p{prepared, total, 1, prepared + 2 * total, v, v_stride, vdim, nullptr, cu_q, slots, state, slot_stride, out,
+                     heads, dim, vdim};
+    if (dtype == TS_F32) return launch_recurrence<float>(p, LR_PLAIN, num_seqs, stream);
+    return launch_recurrence<__nv_bfloat16>(p, LR_PLAIN, num_seqs, stream);
 }
 
 // out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight * act(gate[t, h, :]) * scale; one warp a

@@ -14,12 +14,26 @@
 // Statistics, weights, the sum and the stream are float32; the branch and `out` have the activation
 // dtype.  The weights are given as they multiply (an offset of the stored weight is added by the host).
 //
+// With a second branch (`branch2`) the sublayer is two mixers side by side whose outputs are normed one by one:
+//   b = branch_scale * branch / sqrt(mean(branch^2) + eps) * w_branch + branch_scale2 * (the same of branch2 with w_branch2)
+// takes the place of the branch; with a closing weight of null and no plain add, b itself goes to `out` (no stream).
+//
 // `flags`: TS_NORM_CENTERED makes the opening norm a layer norm without bias,
 //   opening(s) = (s - mean(s)) / sqrt(mean((s - mean(s))^2) + eps) * w_open;
-// TS_NORM_PLAIN_ADD adds the branch as it is (a block that norms only the inputs of its sublayers).
+// TS_NORM_PLAIN_ADD adds the branch as it is (a block that norms only the inputs of its sublayers);
+// TS_NORM_COPY_OUT writes the new row of the stream to `out` without an opening norm (a block that norms only the
+// outputs of its sublayers: the next sublayer reads the stream itself, rounded to the activation dtype).
 #include "common.cuh"
 
-enum { TS_NORM_CENTERED = 1, TS_NORM_PLAIN_ADD = 2 };
+enum { TS_NORM_CENTERED = 1, TS_NORM_PLAIN_ADD = 2, TS_NORM_COPY_OUT = 4 };
+
+// Two branches of one sublayer, each under a norm of its own (null `branch2`: a single branch).
+struct BranchPair {
+    const void* branch2;
+    const float* w_branch;
+    const float* w_branch2;
+    float scale, scale2;
+};
 
 template <typename T>
 __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __restrict__ w_close, float* stream,
@@ -27,13 +41,44 @@ __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __
                                    const int* __restrict__ rows, int width, float eps, const T* __restrict__ table,
                                    const int* __restrict__ ids, int table_rows, float scale, int write_stream,
                                    int flags, const int* __restrict__ positions, const float* __restrict__ pos_freq,
-                                   const float* __restrict__ w_start) {
-    extern __shared__ float row[];                // width floats, then 32 of scratch
+                                   const float* __restrict__ w_start, BranchPair pair) {
+    extern __shared__ float row[];                // width floats, then 64 of scratch
     float* scratch = row + width;
     const int r = blockIdx.x;
     const int src = rows ? rows[r] : r;
     if (src < 0) return;                          // a padding row
     float* sr = stream + (long long)src * width;
+    T* o = out + (long long)r * width;
+    if (pair.branch2) {                           // the two branches' norms; their sum stands in for the branch from here on
+        const T* b1 = branch + (long long)src * width;
+        const T* b2 = (const T*)pair.branch2 + (long long)src * width;
+        float acc1 = 0.f, acc2 = 0.f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {
+            const float x1 = to_float<T>(b1[i]), x2 = to_float<T>(b2[i]);
+            acc1 += x1 * x1;
+            acc2 += x2 * x2;
+        }
+        const float inv1 = pair.scale / sqrtf(block_sum(acc1, scratch) / (float)width + eps);
+        const float inv2 = pair.scale2 / sqrtf(block_sum(acc2, scratch + 32) / (float)width + eps);
+        float acc = 0.f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {      // each thread reads back only the elements it wrote
+            const float b = to_float<T>(b1[i]) * inv1 * pair.w_branch[i] + to_float<T>(b2[i]) * inv2 * pair.w_branch2[i];
+            row[i] = b;
+            acc += b * b;
+        }
+        if (!stream) {
+            for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_float<T>(row[i]);
+            return;
+        }
+        __syncthreads();                          // scratch is used again below
+        if (flags & TS_NORM_PLAIN_ADD) {
+            for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] += sr[i];
+        } else {
+            const float inv = 1.f / sqrtf(block_sum(acc, scratch) / (float)width + eps);
+            __syncthreads();
+            for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] = sr[i] + row[i] * inv * w_close[i];
+        }
+    } else
     if (ids) {
         const int id = ids[src];
         const bool zeros = id < 0 || id >= table_rows;
@@ -80,7 +125,11 @@ __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __
     }
     if (write_stream && (ids || branch))
         for (int i = threadIdx.x; i < width; i += blockDim.x) sr[i] = row[i];
-    if (!w_open) return;
+    if (!w_open) {
+        if (flags & TS_NORM_COPY_OUT)
+            for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_float<T>(row[i]);
+        return;
+    }
     float mean = 0.f;
     if (flags & TS_NORM_CENTERED) {
         float sum = 0.f;
@@ -91,18 +140,20 @@ __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __
     float acc = 0.f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) acc += (row[i] - mean) * (row[i] - mean);
     const float inv = 1.f / sqrtf(block_sum(acc, scratch) / (float)width + eps);
-    T* o = out + (long long)r * width;
     for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_float<T>((row[i] - mean) * inv * w_open[i]);
 }
 
 TS_API int ts_stream_norm(const void* branch, const float* w_close, float* stream, const float* w_open, void* out,
                           const int* rows, int count, int width, float eps, const void* table, const int* ids,
                           int table_rows, float scale, int flags, int dtype, const int* positions, const float* pos_freq,
-                          const float* w_start, cudaStream_t stream_handle) {
+                          const float* w_start, const void* branch2, const float* w_branch, const float* w_branch2,
+                          float branch_scale, float branch_scale2, cudaStream_t stream_handle) {
     TS_REQUIRE(count >= 0 && width > 0, "stream_norm: bad sizes rows=%d width=%d", count, width);
-    TS_REQUIRE(stream != nullptr, "stream_norm: no residual stream");
-    TS_REQUIRE(!(branch && !w_close && !(flags & TS_NORM_PLAIN_ADD)), "stream_norm: a branch needs the weight of its closing norm");
-    TS_REQUIRE(!(w_open && !out), "stream_norm: an opening norm needs an output");
+    TS_REQUIRE(!branch2 || (branch && w_branch && w_branch2), "stream_norm: two branches need both their norms' weights");
+    TS_REQUIRE(stream != nullptr || (branch2 && out && !w_open), "stream_norm: no residual stream");
+    TS_REQUIRE(!(stream && branch && !w_close && !(flags & TS_NORM_PLAIN_ADD)),
+               "stream_norm: a branch needs the weight of its closing norm");
+    TS_REQUIRE(!((w_open || (flags & TS_NORM_COPY_OUT)) && !out), "stream_norm: an opening norm, or a copy of the stream, needs an output");
     TS_REQUIRE(!(ids && (!table || branch)), "stream_norm: token ids need the table and exclude a branch");
     TS_REQUIRE(!(pos_freq && (!ids || !positions)), "stream_norm: a position vector needs token ids and positions");
     TS_REQUIRE(!(w_start && !ids), "stream_norm: a norm on the embedding needs token ids");
@@ -112,7 +163,8 @@ TS_API int ts_stream_norm(const void* branch, const float* w_close, float* strea
     // many rows keep more CTAs on an SM instead
     const int wide = width >= 4096 ? 1024 : width >= 2048 ? 512 : width >= 1024 ? 256 : 128;
     const int threads = count <= 512 ? wide : (width >= 1024 ? 256 : 128);
-    const size_t smem = (size_t)(width + 32) * sizeof(float);
+    const size_t smem = (size_t)(width + 64) * sizeof(float);
+    const BranchPair pair{branch2, w_branch, w_branch2, branch_scale, branch_scale2};
     const int write = rows ? 0 : 1;
 #define TS_STREAM_NORM(TYPE)                                                                                      \
     do {                                                                                                          \
@@ -120,7 +172,7 @@ TS_API int ts_stream_norm(const void* branch, const float* w_close, float* strea
             cudaFuncSetAttribute(stream_norm_kernel<TYPE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         stream_norm_kernel<TYPE><<<count, threads, smem, stream_handle>>>(                                        \
             (const TYPE*)branch, w_close, stream, w_open, (TYPE*)out, rows, width, eps, (const TYPE*)table, ids,  \
-            table_rows, scale, write, flags, positions, pos_freq, w_start);                                             \
+            table_rows, scale, write, flags, positions, pos_freq, w_start, pair);                                       \
     } while (0)
     if (dtype == TS_F32) TS_STREAM_NORM(float);
     else if (dtype == TS_BF16) TS_STREAM_NORM(__nv_bfloat16);

@@ -3,14 +3,18 @@
 //
 //   q = y_q + b_q,  k = y_k + b_k,  v = y_v + b_v                      (biases optional)
 //   q = q / sqrt(mean(q^2) + eps) * w_q     over all heads' channels at once, likewise k   (optional);
-//       with `norm_per_head` every head is normed by itself and w_q, w_k hold one head's channels
+//       with `norm_per_head` every head is normed by itself and w_q, w_k hold one head's channels; `unweighted`
+//       norms every head of q and of k without a weight
 //   q = q * (1 + temp_coef * ln(floor((position + 1) / temp_every) + 1))             (temp_every > 0)
 //   rotate-half rotation of the first `rot` channels of every head of q and k: channel i pairs with
-//   i + rot/2, angle = position * freq[i], cos and sin both multiplied by `magnitude`
+//   i + rot/2, angle = position * freq[i], cos and sin both multiplied by `magnitude`; `interleaved` pairs channel
+//   2i with 2i + 1 instead.  (A rotation by pairs keeps a head's sum of squares, so a norm of a head without a
+//   weight is the same before the rotation and after it.)
 //   k and v go to the token's slot of the paged cache, q to a compact [tokens, heads * dim] tensor.
 //
 // Keys and values may differ in their head size and in their number of heads (`v_heads`: several key heads over
-// one value head), so the value pool has a geometry of its own.
+// one value head), so the value pool has a geometry of its own.  Values may also be the keys as projected: their
+// columns are then k's own (`v_off` = `k_off`), stored without norm and rotation.
 // One CTA a token; sums, angles and the rotation are float32, the stores round to the activation dtype.
 #include "common.cuh"
 
@@ -25,6 +29,7 @@ struct QKPrepareArgs {
     const int* block_table; int table_width; int writes;
     int heads, kv_heads, dim, vdim, v_heads;
     int norm_per_head; float temp_coef; int temp_every;
+    int unweighted, interleaved;
 };
 
 template <typename T>
@@ -48,7 +53,7 @@ __global__ void qk_norm_rope_store_kernel(QKPrepareArgs p) {
     const int page = p.writes ? p.block_table[(long long)seq * p.table_width + pos / p.k_geo.page_tokens] : -1;
     float inv_q = 1.f, inv_k = 1.f;
     extern __shared__ float inv_heads[];              // norm_per_head: 1 / rms of every q head, then of every k head
-    if (p.norm_per_head && (p.q_weight || p.k_weight)) {
+    if (p.norm_per_head && (p.q_weight || p.k_weight || p.unweighted)) {
         const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
         for (int hh = warp; hh < p.heads + p.kv_heads; hh += nwarps) {      // a warp a head
             const bool is_q = hh < p.heads;
@@ -56,7 +61,7 @@ __global__ void qk_norm_rope_store_kernel(QKPrepareArgs p) {
             const T* y = is_q ? yq : yk;
             const float* bias = is_q ? p.q_bias : p.k_bias;
             float acc = 0.f;
-            if (is_q ? p.q_weight != nullptr : p.k_weight != nullptr)
+            if (p.unweighted || (is_q ? p.q_weight != nullptr : p.k_weight != nullptr))
                 for (int i = lane; i < p.dim; i += 32) {
                     const float x = to_float<T>(y[e0 + i]) + (bias ? bias[e0 + i] : 0.f);
                     acc += x * x;
@@ -86,6 +91,7 @@ __global__ void qk_norm_rope_store_kernel(QKPrepareArgs p) {
     // `heads_at`: where this projection's heads start in inv_heads; `gain` multiplies every element (the query's temperature)
     auto element = [&](const T* y, const float* bias, const float* weight, float inv, int heads_at, float gain, int e) {
         const float x = to_float<T>(y[e]) + (bias ? bias[e] : 0.f);
+        if (p.unweighted) return x * inv_heads[heads_at + e / p.dim] * gain;
         if (!weight) return x * gain;
         if (p.norm_per_head) return x * inv_heads[heads_at + e / p.dim] * weight[e % p.dim] * gain;
         return x * inv * weight[e] * gain;
@@ -98,15 +104,16 @@ __global__ void qk_norm_rope_store_kernel(QKPrepareArgs p) {
         for (int e = threadIdx.x; e < n; e += blockDim.x) {
             const int i = e % p.dim;
             if (p.freq && i < p.rot) {
-                if (i >= half) continue;                   // written by the pair's first channel
+                if (p.interleaved ? (i & 1) : i >= half) continue;                 // written by the pair's first channel
+                const int other = p.interleaved ? e + 1 : e + half;
                 const float u = element(y, bias, weight, inv, heads_at, gain, e);
-                const float v = element(y, bias, weight, inv, heads_at, gain, e + half);
+                const float v = element(y, bias, weight, inv, heads_at, gain, other);
                 float sn, cs;
-                sincosf((float)pos * p.freq[i], &sn, &cs);
+                sincosf((float)pos * p.freq[p.interleaved ? i >> 1 : i], &sn, &cs);
                 sn *= p.magnitude;
                 cs *= p.magnitude;
                 store(e, u * cs - v * sn);
-                store(e + half, v * cs + u * sn);
+                store(other, v * cs + u * sn);
             } else {
                 store(e, element(y, bias, weight, inv, heads_at, gain, e));
             }
@@ -135,7 +142,9 @@ TS_API int ts_qk_norm_rope_store(const void* y, long long y_stride, int q_off, i
                                  long long k_entry_offset, long long v_page_stride, long long v_entry_offset,
                                  int page_tokens, int num_pages, const int* block_table, int table_width, int writes,
                                  int num_tokens, int heads, int kv_heads, int dim, int vdim, int dtype,
-                                 int norm_per_head, float temp_coef, int temp_every, int value_heads, cudaStream_t stream) {
+                                 int norm_per_head, float temp_coef, int temp_every, int value_heads, int unweighted,
+                                 int interleaved, cudaStream_t stream) {
+    TS_REQUIRE(!unweighted || (norm_per_head && !q_weight && !k_weight), "qk_norm_rope_store: an unweighted norm is one a head");
     TS_REQUIRE(value_heads >= 0, "qk_norm_rope_store: bad number of value heads");
     TS_REQUIRE(heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && num_tokens >= 0, "qk_norm_rope_store: bad sizes");
     TS_REQUIRE(rot >= 0 && rot <= dim && rot % 2 == 0, "qk_norm_rope_store: rotation over %d of %d channels", rot, dim);
@@ -145,7 +154,8 @@ TS_API int ts_qk_norm_rope_store(const void* y, long long y_stride, int q_off, i
                     rot > 0 ? freq : nullptr, rot, magnitude, positions, seq_of_token, q_out, k_pool, v_pool,
                     KVGeometry{k_page_stride, k_entry_offset, page_tokens, num_pages},
                     KVGeometry{v_page_stride, v_entry_offset, page_tokens, num_pages}, block_table, table_width, writes,
-                    heads, kv_heads, dim, vdim, value_heads > 0 ? value_heads : kv_heads, norm_per_head, temp_coef, temp_every};
+                    heads, kv_heads, dim, vdim, value_heads > 0 ? value_heads : kv_heads, norm_per_head, temp_coef, temp_every,
+                    unweighted, interleaved};
     const size_t smem = norm_per_head ? (size_t)(heads + kv_heads) * sizeof(float) : 0;
     TS_REQUIRE(smem <= 32 * 1024, "qk_norm_rope_store: %d heads are not supported", heads + kv_heads);
     // many tokens: small CTAs, many of them on an SM (a CTA's life is a chain of loads and two sums); few tokens: wide ones

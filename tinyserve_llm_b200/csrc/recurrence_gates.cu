@@ -1,11 +1,19 @@
-// What enters the scan of linear_recurrence.cu for two recurrences whose gates are computed from the
-// input: the gated delta rule and the matrix memory with exponential gates (mLSTM).  Everything here
-// is float32; the inputs are projections' outputs in the activation dtype (or float32).
+// What enters the scan of linear_recurrence.cu for recurrences whose gates are computed from the input:
+// the gated delta rule, the matrix memory with exponential gates (mLSTM), and time mixing with
+// decays per channel and a bonus for the current token (RWKV).  Everything here is float32; the
+// inputs are projections' outputs in the activation dtype (or float32).
 //
 // Gated delta rule.  q and k ([tokens, kv_heads * dim], float32, after their short convolution) become
 // unit vectors per head, x / sqrt(sum(x^2) + unit_eps), q also times q_scale; value head h uses q/k
 // head h / (heads / kv_heads).  The decay of head h, key channel i is
-//   a = exp(-exp(A_log[h]) * softplus(z[t, h, i] + dt_bias[h, i])),   beta[t, h] = sigmoid(b[t, h]).
+//   a = exp(-exp(A_log[h]) * softplus(z[t, h, i] + dt_bias[h, i])),   beta[t, h] = sigmoid(b[t, h]);
+// or, with one decay a head, z and dt_bias have no channel index and neither has a; q and k are then written once a
+// q/k head.
+//
+// Time mixing.  a[t, h, i] = exp(-exp(z[t, h, i] + w0[h, i])), r and k pass as they are, and what the current
+// token's write adds to the read-out under the bonus u is v times sum_i u[h, i] k[t, h, i] r[t, h, i].
+// The mixer's inputs are blends of the token's row and the one before it, h + (h' - h) mu, one for every mu;
+// the row before a step's first token comes from the request's state slot (zeros at the start).
 //
 // Matrix memory.  Per head (x_i, x_f: float32 projections), log input gate i = cap tanh((x_i + b_i) / cap), log forget gate
 // f = log_sigmoid(cap tanh((x_f + b_f) / cap)), running maximum m_t = max(f + m_(t-1), i) carried in the
@@ -61,6 +69,158 @@ TS_API int ts_delta_prepare(const float* q, const float* k, long long qk_stride,
     else
         return ts_fail("delta_prepare: unknown dtype code %d", dtype);
     TS_LAUNCH_CHECK("delta_prepare");
+    return 0;
+}
+
+// The same with one decay a head: one warp a (token, q/k head), which also takes its value heads' gates.  gates
+// [tokens, 2 heads] float32 holds the step sizes' logits, then the decays'; prepared is [2][tokens, kv_heads * dim],
+// beta and decay [tokens, heads].
+__global__ void delta_prepare_head_kernel(const float* __restrict__ q, const float* __restrict__ k, long long qk_stride,
+                                          const float* __restrict__ gates, const float* __restrict__ dt_bias,
+                                          const float* __restrict__ a_log, float* __restrict__ prepared,
+                                          float* __restrict__ beta, float* __restrict__ decay, long long items, int heads,
+                                          int kv_heads, int dim, float unit_eps, float q_scale) {
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= items) return;
+    const int lane = threadIdx.x & 31;
+    const long long t = item / kv_heads;
+    const int g = (int)(item % kv_heads), group = heads / kv_heads;
+    const float* qr = q + t * qk_stride + (long long)g * dim;
+    const float* kr = k + t * qk_stride + (long long)g * dim;
+    for (int i = lane; i < group; i += 32) {
+        const int h = g * group + i;
+        const float b = gates[t * 2 * heads + h], z = gates[t * 2 * heads + heads + h];
+        beta[t * heads + h] = 1.f / (1.f + expf(-b));
+        decay[t * heads + h] = expf(-expf(a_log[h]) * softplus(z + dt_bias[h]));
+    }
+    float sq = 0.f, sk = 0.f;
+    for (int i = lane; i < dim; i += 32) { sq += qr[i] * qr[i]; sk += kr[i] * kr[i]; }
+    const float inv_q = q_scale / sqrtf(warp_sum(sq) + unit_eps), inv_k = 1.f / sqrtf(warp_sum(sk) + unit_eps);
+    const long long at = item * dim, total = items * dim;
+    for (int i = lane; i < dim; i += 32) {
+        prepared[at + i] = qr[i] * inv_q;
+        prepared[total + at + i] = kr[i] * inv_k;
+    }
+}
+
+TS_API int ts_delta_prepare_head(const float* q, const float* k, long long qk_stride, const float* gates,
+                                 const float* dt_bias, const float* a_log, float* prepared, float* beta, float* decay,
+                                 int num_tokens, int heads, int kv_heads, int dim, float unit_eps, float q_scale,
+                                 cudaStream_t stream) {
+    TS_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0, "delta_prepare: %d heads over %d q/k heads",
+               heads, kv_heads);
+    if (num_tokens <= 0) return 0;
+    const long long items = (long long)num_tokens * kv_heads;
+    delta_prepare_head_kernel<<<(unsigned)((items + 3) / 4), 128, 0, stream>>>(q, k, qk_stride, gates, dt_bias, a_log, prepared,
+        beta, decay, items, heads, kv_heads, dim, unit_eps, q_scale);
+    TS_LAUNCH_CHECK("delta_prepare_head");
+    return 0;
+}
+
+// mixes[s][t] = x[t] + (x'[t] - x[t]) * mu[s], x' the request's row before t: of this step, or from its slot.
+// A thread takes a channel of a token and writes it for every s.
+template <typename T>
+__global__ void token_shift_kernel(const T* __restrict__ x, const float* __restrict__ mu, const int* __restrict__ seq_of_token,
+                                   const int* __restrict__ cu_q, const int* __restrict__ slots, const float* __restrict__ state,
+                                   long long slot_stride, T* __restrict__ mixes, int num_tokens, int width, int count) {
+    const long long total = (long long)num_tokens * width;
+    for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (long long)gridDim.x * blockDim.x) {
+        const int t = (int)(e / width), c = (int)(e % width);
+        const int seq = seq_of_token[t];
+        float now = 0.f, before = 0.f;                         // a padding row
+        if (seq >= 0) {
+            now = to_float<T>(x[e]);
+            const int slot = slots[seq];
+            if (t > cu_q[seq]) before = to_float<T>(x[e - width]);
+            else if (slot >= 0) before = state[(long long)slot * slot_stride + c];
+        }
+        for (int s = 0; s < count; ++s)
+            mixes[s * total + e] = from_float<T>(fmaf(before - now, mu[(long long)s * width + c], now));
+    }
+}
+
+// `state` points at the request slots' previous rows ([width] floats a slot, `slot_stride` floats apart); it is read
+// here and moved on by the kernel that prepares the scan's inputs.
+TS_API int ts_token_shift(const void* x, const float* mu, const int* seq_of_token, const int* cu_q, const int* slots,
+                          const float* state, long long slot_stride, void* mixes, int num_tokens, int width, int count,
+                          int dtype, cudaStream_t stream) {
+    TS_REQUIRE(width > 0 && count > 0 && slot_stride >= width, "token_shift: bad sizes");
+    if (num_tokens <= 0) return 0;
+    const long long total = (long long)num_tokens * width;
+    const unsigned blocks = (unsigned)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+    if (dtype == TS_F32)
+        token_shift_kernel<float><<<blocks, 256, 0, stream>>>((const float*)x, mu, seq_of_token, cu_q, slots, state, slot_stride,
+                                                              (float*)mixes, num_tokens, width, count);
+    else if (dtype == TS_BF16)
+        token_shift_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)x, mu, seq_of_token, cu_q, slots, state,
+                                                                      slot_stride, (__nv_bfloat16*)mixes, num_tokens, width, count);
+    else
+        return ts_fail("token_shift: unknown dtype code %d", dtype);
+    TS_LAUNCH_CHECK("token_shift");
+    return 0;
+}
+
+// One warp a (token, head); the blocks past `item_blocks` move the requests' previous rows on (a warp takes 32 x 4
+// channels of one request).
+template <typename T>
+__global__ void time_mix_prepare_kernel(const T* __restrict__ r, const T* __restrict__ k, long long rk_stride,
+                                        const float* __restrict__ z, const float* __restrict__ w0, const float* __restrict__ u,
+                                        float* __restrict__ prepared, float* __restrict__ bonus, long long items, int heads,
+                                        int dim, unsigned item_blocks, const T* __restrict__ x, int width,
+                                        const int* __restrict__ cu_q, const int* __restrict__ slots, int num_seqs,
+                                        float* __restrict__ state, long long slot_stride) {
+    const int lane = threadIdx.x & 31;
+    if (blockIdx.x >= item_blocks) {
+        const int stretches = (width + 127) / 128;
+        const long long w = (long long)(blockIdx.x - item_blocks) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+        const int seq = (int)(w / stretches), c0 = (int)(w % stretches) * 128;
+        if (seq >= num_seqs) return;
+        const int slot = slots[seq], last = cu_q[seq + 1] - 1;
+        if (slot < 0 || last < cu_q[seq]) return;              // a padding request, or one that feeds nothing
+        for (int c = c0 + lane; c < min(c0 + 128, width); c += 32)
+            state[(long long)slot * slot_stride + c] = to_float<T>(x[(long long)last * width + c]);
+        return;
+    }
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= items) return;
+    const long long t = item / heads;
+    const int h = (int)(item % heads);
+    const T* rr = r + t * rk_stride + (long long)h * dim;
+    const T* kr = k + t * rk_stride + (long long)h * dim;
+    const long long at = item * dim, total = items * dim, hc = (long long)h * dim;
+    float acc = 0.f;
+    for (int i = lane; i < dim; i += 32) {
+        const float rv = to_float<T>(rr[i]), kv = to_float<T>(kr[i]);
+        prepared[at + i] = rv;
+        prepared[total + at + i] = kv;
+        prepared[2 * total + at + i] = expf(-expf(z[at + i] + w0[hc + i]));
+        acc = fmaf(u[hc + i] * kv, rv, acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) bonus[item] = acc;
+}
+
+// r, k: [tokens, heads * dim] with one row stride; z float32 [tokens, heads * dim]; prepared [3][tokens, heads * dim],
+// bonus [tokens, heads].  `x` [tokens, width] is the mixer's input, whose last row of every request goes to its slot.
+TS_API int ts_time_mix_prepare(const void* r, const void* k, long long rk_stride, const float* z, const float* w0,
+                               const float* u, float* prepared, float* bonus, int num_tokens, int heads, int dim,
+                               const void* x, int width, const int* cu_q, const int* slots, int num_seqs, float* state,
+                               long long slot_stride, int dtype, cudaStream_t stream) {
+    TS_REQUIRE(heads > 0 && dim > 0 && width > 0 && slot_stride >= width, "time_mix_prepare: bad sizes");
+    if (num_tokens <= 0) return 0;
+    const long long items = (long long)num_tokens * heads;
+    const unsigned item_blocks = (unsigned)((items + 3) / 4);
+    const unsigned more = (unsigned)(((long long)num_seqs * ((width + 127) / 128) + 3) / 4);
+    if (dtype == TS_F32)
+        time_mix_prepare_kernel<float><<<item_blocks + more, 128, 0, stream>>>((const float*)r, (const float*)k, rk_stride, z, w0, u,
+            prepared, bonus, items, heads, dim, item_blocks, (const float*)x, width, cu_q, slots, num_seqs, state, slot_stride);
+    else if (dtype == TS_BF16)
+        time_mix_prepare_kernel<__nv_bfloat16><<<item_blocks + more, 128, 0, stream>>>((const __nv_bfloat16*)r, (const __nv_bfloat16*)k,
+            rk_stride, z, w0, u, prepared, bonus, items, heads, dim, item_blocks, (const __nv_bfloat16*)x, width, cu_q, slots,
+            num_seqs, state, slot_stride);
+    else
+        return ts_fail("time_mix_prepare: unknown dtype code %d", dtype);
+    TS_LAUNCH_CHECK("time_mix_prepare");
     return 0;
 }
 

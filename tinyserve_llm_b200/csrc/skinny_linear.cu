@@ -48,6 +48,8 @@ struct RopeArgs {
     float act_limit, act_alpha;
     int unary;                   // store epilogue: 1 + TS_UNARY_* of an activation of one argument (0: none), a, b below
     float unary_a, unary_b;
+    int group_tiles;             // store epilogue: CTAs of a group of output rows with an x and a y of its own (0: one group)
+    long long x_group, y_group;  // elements from a group's x, or y, to the next one's
 };
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
@@ -110,6 +112,8 @@ skinny_linear_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
     }
     const __nv_bfloat16* w_lo = W + row_lo * K + c * 8;
     const __nv_bfloat16* w_hi = W + row_hi * K + c * 8;
+    const int group = EPI == EPI_STORE && rope.group_tiles ? (int)blockIdx.x / rope.group_tiles : 0;
+    x += group * rope.x_group;
     const __nv_bfloat16* x_row[MT];
     bool x_ok[MT];
 #pragma unroll
@@ -273,6 +277,8 @@ skinny_linear_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
         }
     } else {
         constexpr int PER = 4;
+        const int col0 = ((int)blockIdx.x - group * rope.group_tiles) * ROWS;
+        y += group * rope.y_group;
         for (int i = threadIdx.x; i < MT * 32 * PER; i += WARPS * 32) {
             const int t = i / (32 * PER), l = (i / PER) % 32, e = i % PER;
             float v = 0.f;
@@ -281,7 +287,7 @@ skinny_linear_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* _
             const int row = (l >> 2) + ((e >> 1) << 3), token = t * 8 + ((l & 3) << 1) + (e & 1);
             // an activation of one argument reads the product as the separate kernel would: rounded to the output type
             if (rope.unary) v = ts_unary_activation(rope.unary - 1, round_to<OUT>(v), rope.unary_a, rope.unary_b);
-            if (row < rows_valid && token < M) store_out<OUT>(y + (long long)token * ldy + blockIdx.x * ROWS + row, v);
+            if (row < rows_valid && token < M) store_out<OUT>(y + (long long)token * ldy + col0 + row, v);
         }
     }
 }
@@ -371,7 +377,7 @@ TS_API int ts_skinny_linear_unary(const void* W, const void* x, void* y, int M, 
                ts_skinny_linear_max_rows());
     TS_REQUIRE(K % 32 == 0 && ldx % 8 == 0 && ((uintptr_t)W % 16 == 0) && ((uintptr_t)x % 16 == 0),
                "skinny_linear_unary: K a multiple of 32 and 16-byte aligned operands are needed");
-    TS_REQUIRE(kind == TS_UNARY_RELU2 || kind == TS_UNARY_XIELU, "skinny_linear_unary: unknown activation %d", kind);
+    TS_REQUIRE(kind >= TS_UNARY_RELU2 && kind <= TS_UNARY_LAST, "skinny_linear_unary: unknown activation %d", kind);
     if (M == 0) return 0;
     RopeArgs args{};
     args.unary = kind + 1;
@@ -380,6 +386,25 @@ TS_API int ts_skinny_linear_unary(const void* W, const void* x, void* y, int M, 
     if (out_dtype == TS_BF16) return dispatch_warps<EPI_STORE, __nv_bfloat16>(W, x, y, M, N, K, ldx, ldy, 0, stream, args);
     if (out_dtype == TS_F32) return dispatch_warps<EPI_STORE, float>(W, x, y, M, N, K, ldx, ldy, 0, stream, args);
     return ts_fail("skinny_linear_unary: unknown output dtype %d", out_dtype);
+}
+
+// `groups` products in one launch: y[g][M, N] = x[g][M, K] . W[g][N, K]^T, N a multiple of 16 (a CTA's 16 rows of W
+// belong to one group).  x and y of a group lie x_group and y_group elements behind those of the group before.
+TS_API int ts_skinny_linear_groups(const void* W, const void* x, void* y, int groups, int M, int N, int K, long long ldx,
+                                   long long x_group, long long ldy, long long y_group, int out_dtype, cudaStream_t stream) {
+    TS_REQUIRE(groups > 0 && M >= 0 && N > 0 && K > 0, "skinny_linear_groups: bad sizes M=%d N=%d K=%d", M, N, K);
+    TS_REQUIRE(M <= ts_skinny_linear_max_rows(), "skinny_linear_groups: %d rows of x; the kernel takes up to %d", M,
+               ts_skinny_linear_max_rows());
+    TS_REQUIRE(N % 16 == 0 && K % 32 == 0 && ldx % 8 == 0 && x_group % 8 == 0 && ((uintptr_t)W % 16 == 0) && ((uintptr_t)x % 16 == 0),
+               "skinny_linear_groups: N a multiple of 16, K of 32 and 16-byte aligned operands are needed");
+    if (M == 0) return 0;
+    RopeArgs args{};
+    args.group_tiles = N / 16;
+    args.x_group = x_group;
+    args.y_group = y_group;
+    if (out_dtype == TS_BF16) return dispatch_warps<EPI_STORE, __nv_bfloat16>(W, x, y, M, groups * N, K, ldx, ldy, 0, stream, args);
+    if (out_dtype == TS_F32) return dispatch_warps<EPI_STORE, float>(W, x, y, M, groups * N, K, ldx, ldy, 0, stream, args);
+    return ts_fail("skinny_linear_groups: unknown output dtype %d", out_dtype);
 }
 
 // y[M, N/2] = act(x Wgate^T, x Wup^T) with another gated activation than SiLU in the epilogue (TS_ACT_* of common.cuh).

@@ -7,6 +7,7 @@ attention: if the shared object cannot be built or loaded, constructing `Ops` ra
 from __future__ import annotations
 
 import ctypes
+import math
 import os
 
 import torch
@@ -30,10 +31,10 @@ _SIGNATURES = {
     "ts_paged_attention_bf16": ("int", "pppplliipippiiiiiiifiplpip"),
     "ts_paged_attention_generic": ("int", "pppplliipippiiiifiip"),
     "ts_paged_attention_bf16_sigmoid": ("int", "pl" "ppp" "lliipippiiiiiiifiplpi" "pppl" "p"),
-    "ts_paged_attention_bf16_masked": ("int", "pl" "ppp" "lllliipippiiiiiiifiifi" "plpi" "p"),
+    "ts_paged_attention_bf16_masked": ("int", "pl" "ppp" "lllliipippiiiiiiifiifi" "plpi" "fp"),
     "ts_attention_tcgen05_supported": ("int", "iiiii"),
     "ts_prefill_attention_tcgen05_dense": ("int", "pl" "ppp" "lpppiiiiiifpipp"),
-    "ts_prefill_attention_tcgen05_masked": ("int", "pl" "ppp" "iiiipippiiiiiifiifi" "pipp"),
+    "ts_prefill_attention_tcgen05_masked": ("int", "pl" "ppp" "iiiipippiiiiiifiifi" "pipfp"),
     "ts_prefill_attention_tcgen05": ("int", "ppppiiiipippiiiiiifpipp"),
     "ts_prefill_attention_tcgen05_sigmoid": ("int", "pl" "ppp" "iiiipippiiiiiifi" "pppl" "pipp"),
     "ts_embedding": ("int", "pppiiiip"),
@@ -55,8 +56,9 @@ _SIGNATURES = {
     "ts_skinny_qkv_rope_store": ("int", "pppiilpppiipipplliiiiiip"),
     "ts_skinny_linear_gated": ("int", "pppiiilliffp"),
     "ts_skinny_linear_unary": ("int", "pppiiilliffip"),
+    "ts_skinny_linear_groups": ("int", "pppiiiillllip"),
     "ts_gemm_tcgen05_gated": ("int", "pppiiilliffpp"),
-    "ts_stream_norm": ("int", "ppppppiifppifiipppp"),
+    "ts_stream_norm": ("int", "ppppppiifppifiippp" "pppff" "p"),
     "ts_linear_recurrence": ("int", "ppplllplppfffpipppiplpiiiipip"),
     "ts_head_norm_gate": ("int", "piplpippliiififip"),
     "ts_latent_prepare": ("int", "pliiippfppppplliipiiiip"),
@@ -68,16 +70,19 @@ _SIGNATURES = {
     "ts_moe_linear": ("int", "plpipipiipiiiffpiip"),
     "ts_moe_combine": ("int", "pppppiiiippp"),
     "ts_moe_route_grouped": ("int", "pppppppiiiiiiffp"),
-    "ts_paged_attention_scored": ("int", "plpppllllii" "pippiiiiifiiipppl" "fiii" "p"),
+    "ts_paged_attention_scored": ("int", "plpppllllii" "pippiiiiifiiipppl" "fiiif" "p"),
     "ts_mingru_scan": ("int", "pliiiippppiplpiiiip"),
     "ts_unary_activation_rows": ("int", "ppliffip"),
     "ts_gated_activation": ("int", "ppiiiffip"),
     "ts_sgemm_nt_batched": ("int", "pppiiilllilllp"),
-    "ts_qk_norm_rope_store": ("int", "pliiipppppfpifpppppllllii" "piiiiiiiiifiip"),
+    "ts_qk_norm_rope_store": ("int", "pliiipppppfpifpppppllllii" "piiiiiiiiifiiiip"),
     "ts_sigmoid_gate": ("int", "plplpliifip"),
     "ts_paged_attention_split": ("int", "plpppllllii" "pippiiiiifiip"),
     "ts_short_conv_silu": ("int", "plppppiplpiiiip"),
-    "ts_recurrence_scan": ("int", "ppliipppiplpiiiip"),
+    "ts_recurrence_scan": ("int", "pipi" "pliipppiplpiiiip"),
+    "ts_delta_prepare_head": ("int", "pplpppppp" "iiiiffp"),
+    "ts_token_shift": ("int", "pppppplp" "iiiip"),
+    "ts_time_mix_prepare": ("int", "pplppppp" "iiipippiplip"),
     "ts_delta_prepare": ("int", "pplppppl" "ppiiiiffip"),
     "ts_mlstm_prepare": ("int", "ppllpplppffppiplpppiiiip"),
     "ts_row_scaled_activation": ("int", "ppppiiiip"),
@@ -442,7 +447,8 @@ class Ops:
                     w_open: torch.Tensor | None, eps: float, dtype: torch.dtype, rows: torch.Tensor | None = None,
                     table: torch.Tensor | None = None, ids: torch.Tensor | None = None, scale: float = 1.0,
                     centered: bool = False, plain_add: bool = False, positions: torch.Tensor | None = None,
-                    position_frequencies: torch.Tensor | None = None, w_start: torch.Tensor | None = None) -> torch.Tensor | None:
+                    position_frequencies: torch.Tensor | None = None, w_start: torch.Tensor | None = None,
+                    copy_out: bool = False, pair: tuple | None = None) -> torch.Tensor | None:
         """
         stream (float32, in place) += closing norm of `branch` (if given; with `plain_add` the branch as
         it is); returns the opening norm of the sum in `dtype` (if `w_open` is given; with `centered` a
@@ -452,9 +458,16 @@ class Ops:
         [ceil(width / 2)]), the vector whose entry 2i is sin(position * frequency i) and entry 2i + 1 its cosine;
         with `w_start` the gathered rows are normed with that weight (as the opening norm norms: RMS, or centered)
         before they start the stream.  Weights are float32 and multiply as given.
+
+        `copy_out`: no opening norm; the new rows of the stream are returned in `dtype`.  `pair` (branch2, w1, w2,
+        scale1, scale2): two branches of one sublayer, each RMS-normed with a weight of its own, whose sum
+        scale1 * norm(branch) * w1 + scale2 * norm(branch2) * w2 takes the branch's place.
         """
         self._check(stream, "residual stream", torch.float32, 2)
         width = stream.shape[1]
+        if copy_out and (w_open is not None or rows is not None):
+            raise KernelError("stream_norm: a copy of the stream takes the place of the opening norm, for all rows")
+        branch2, w_branch, w_branch2, scale1, scale2 = self._branch_pair(branch, pair, width)
         if w_start is not None and ids is None:
             raise KernelError("stream_norm: a norm on the embedding rows needs token ids")
         for w, name in ((w_close, "closing weight"), (w_open, "opening weight"), (w_start, "embedding norm weight")):
@@ -481,13 +494,37 @@ class Ops:
             self._check(rows, "rows", torch.int32, 1)
             count = rows.shape[0]
         out = None
-        if w_open is not None:
+        if w_open is not None or copy_out:
             out = torch.empty((count, width), dtype=dtype, device=stream.device)
         self._call("ts_stream_norm", _ptr(branch), _ptr(w_close), _ptr(stream), _ptr(w_open), _ptr(out), _ptr(rows), count,
                    width, eps, _ptr(table), _ptr(ids), table.shape[0] if table is not None else 0, scale,
-                   (1 if centered else 0) | (2 if plain_add else 0), _DTYPE_CODE[dtype],
+                   (1 if centered else 0) | (2 if plain_add else 0) | (4 if copy_out else 0), _DTYPE_CODE[dtype],
                    _ptr(positions) if position_frequencies is not None else 0, _ptr(position_frequencies), _ptr(w_start),
-                   _stream())
+                   _ptr(branch2), _ptr(w_branch), _ptr(w_branch2), scale1, scale2, _stream())
+        return out
+
+    def _branch_pair(self, branch: torch.Tensor | None, pair: tuple | None, width: int) -> tuple:
+        if pair is None:
+            return None, None, None, 0.0, 0.0
+        branch2, w1, w2, scale1, scale2 = pair
+        if branch is None:
+            raise KernelError("a pair of branches needs both")
+        self._check(branch2, "second branch", branch.dtype, 2)
+        if branch2.shape != branch.shape:
+            raise KernelError(f"the branches differ: {tuple(branch.shape)} and {tuple(branch2.shape)}")
+        for w in (w1, w2):
+            self._check(w, "branch norm weight", torch.float32, 1)
+            if w.shape[0] != width:
+                raise KernelError(f"a branch norm weight has {w.shape[0]} elements for rows of {width}")
+        return branch2, w1, w2, float(scale1), float(scale2)
+
+    def normed_sum(self, branch: torch.Tensor, pair: tuple, eps: float) -> torch.Tensor:
+        """scale1 * norm(branch) * w1 + scale2 * norm(branch2) * w2 for `pair` (branch2, w1, w2, scale1, scale2), RMS norms of the rows."""
+        self._check(branch, "branch", tuple(_DTYPE_CODE), 2)
+        branch2, w1, w2, scale1, scale2 = self._branch_pair(branch, pair, branch.shape[1])
+        out = torch.empty_like(branch)
+        self._call("ts_stream_norm", _ptr(branch), 0, 0, 0, _ptr(out), 0, branch.shape[0], branch.shape[1], eps, 0, 0, 0, 1.0, 0,
+                   _DTYPE_CODE[branch.dtype], 0, 0, 0, _ptr(branch2), _ptr(w1), _ptr(w2), scale1, scale2, _stream())
         return out
 
     # ------------------------------------------------------------------ linear recurrences
@@ -558,14 +595,17 @@ class Ops:
     # ------------------------------------------------------------------ attention with normed queries and keys, gated recurrences
     def qk_norm_rope_store(self, y: torch.Tensor, offsets: tuple[int, int, int], biases, weights, eps: float, position,
                            ctx, binding, heads: int, kv_heads: int, dim: int, vdim: int, *, norm_per_head: bool = False,
-                           q_temperature: tuple[float, int] | None = None, value_heads: int = 0) -> torch.Tensor:
+                           q_temperature: tuple[float, int] | None = None, value_heads: int = 0,
+                           unweighted_norm: bool = False) -> torch.Tensor:
         """
         From the projection's output y (q, k, v at the column `offsets`): biases added (float32 tensors or
         None), q and k RMS-normed over the whole projection with `weights` (q's, k's; or None; with
         `norm_per_head` every head by itself, the weights [dim]), rotated by `position` (frequencies, dims,
         magnitude), q multiplied by 1 + coef * ln(floor((position + 1) / every) + 1) for `q_temperature`
         (coef, every), k and v stored into the token's cache slot.  `value_heads` (0: as many as key heads): v
-        holds that many heads of vdim channels.  Returns q [T, heads * dim].
+        holds that many heads of vdim channels.  `unweighted_norm`: every head of q and of k is RMS-normed by
+        itself without a weight.  The columns of v may be k's own: the value is then the key as projected.
+        Returns q [T, heads * dim].
         """
         if y.dtype not in _DTYPE_CODE or y.dim() != 2 or y.stride(1) != 1:
             raise KernelError("qk_norm_rope_store: y must be a [T, columns] stretch of an activation dtype")
@@ -588,14 +628,15 @@ class Ops:
                    _ptr(ctx.seq_of_token), _ptr(q), _ptr(binding.k_pool), _ptr(binding.v_pool), binding.page_stride,
                    binding.entry_offset, v_page_stride, v_entry_offset, binding.page_tokens, binding.num_pages,
                    _ptr(binding.block_table), binding.table_width, 1 if binding.writes else 0, T, heads, kv_heads, dim,
-                   vdim, _DTYPE_CODE[y.dtype], 1 if norm_per_head else 0, float(coef), int(every), int(value_heads), _stream())
+                   vdim, _DTYPE_CODE[y.dtype], 1 if norm_per_head or unweighted_norm else 0, float(coef), int(every),
+                   int(value_heads), 1 if unweighted_norm else 0, 1 if getattr(position, "interleaved", False) else 0, _stream())
         return q
 
     def paged_attention_split(self, q: torch.Tensor, ctx, binding, nh: int, nkv: int, hd: int, vd: int, scale: float,
                               window: int, *, weights: str = "softmax", slopes: torch.Tensor | None = None,
                               head_bias: torch.Tensor | None = None, head_gate: torch.Tensor | None = None,
                               softcap: float = 0.0, chunk: int = 0, value_heads: int = 0,
-                              out_dtype: torch.dtype | None = None) -> torch.Tensor:
+                              out_dtype: torch.dtype | None = None, sink: float | None = None) -> torch.Tensor:
         """
         [T, nh * vd]: causal attention of q [T, nh * hd] over the entry's cached keys (head size hd) and
         values (head size vd).  Equal head sizes of 64 or 128 in bfloat16 run on the tensor-core kernels
@@ -607,7 +648,7 @@ class Ops:
         the activation dtype) multiplies head h's output by sigmoid(head_gate[t, h]); `softcap` c > 0 turns the
         scaled product into c tanh(. / c); `chunk` n > 0 hides every key before floor(i / n) * n from query i;
         `value_heads` g > 0: the value pool holds g heads and head h reads value head h / (nh / g); `out_dtype`
-        float32 keeps the output unrounded.
+        float32 keeps the output unrounded; `sink` is a score that takes part in every softmax's sum without a key or a value.
         """
         self._check(q, "q", tuple(_DTYPE_CODE), 2)
         if q.shape[1] != nh * hd:
@@ -620,9 +661,12 @@ class Ops:
             raise KernelError(f"paged_attention_split: output dtype {out_dtype}")
         out_f32 = out_dtype == torch.float32 and q.dtype != torch.float32
         if (weights != "softmax" or slopes is not None or head_bias is not None or head_gate is not None or softcap > 0
-                or chunk > 0 or value_heads > 0 or out_f32):
+                or chunk > 0 or value_heads > 0 or out_f32 or sink is not None):
+            if sink is not None and (weights != "softmax" or not math.isfinite(sink)):
+                raise KernelError(f"paged_attention_split: a sink of {sink} with {weights} weights")
             return self._paged_attention_scored(q, ctx, binding, nh, nkv, hd, vd, scale, window, weights, slopes, head_bias,
-                                                head_gate, softcap, chunk, value_heads, out_f32)
+                                                head_gate, softcap, chunk, value_heads, out_f32,
+                                                -math.inf if sink is None else float(sink))
         if (hd == vd and q.dtype == torch.bfloat16 and getattr(ctx, "cu_q", None) is not None
                 and self.lib.ts_attention_bf16_supported(hd, binding.page_tokens, nh, nkv)):
             # the tensor-core kernels read q from the columns of a [q | k | v] row: q alone is such a row's first part
@@ -638,7 +682,7 @@ class Ops:
         return out
 
     def _paged_attention_scored(self, q, ctx, binding, nh, nkv, hd, vd, scale, window, weights, slopes, head_bias,
-                                head_gate, softcap=0.0, chunk=0, value_heads=0, out_f32=False) -> torch.Tensor:
+                                head_gate, softcap=0.0, chunk=0, value_heads=0, out_f32=False, sink=-math.inf) -> torch.Tensor:
         for t, name in ((slopes, "slopes"), (head_bias, "head bias")):
             if t is not None:
                 self._check(t, name, torch.float32, 1)
@@ -674,7 +718,7 @@ class Ops:
                            binding.entry_offset // per_entry, binding.page_tokens, _ptr(binding.block_table),
                            binding.table_width, _ptr(ctx.cu_q), _ptr(ctx.ctx_lens), num_seqs, q.shape[0], max_q_len, nh, nkv,
                            hd, scale, window, int(chunk), float(softcap), int(value_heads), _ptr(prefill_seqs), num_prefill,
-                           self.error_word().data_ptr(), _stream())
+                           self.error_word().data_ptr(), sink, _stream())
                 if ctx.min_q_len > 1:
                     return out
                 max_q_len = 1
@@ -684,7 +728,7 @@ class Ops:
                        binding.page_tokens, binding.num_pages, _ptr(binding.block_table), binding.table_width, _ptr(ctx.cu_q),
                        _ptr(ctx.ctx_lens), num_seqs, max_q_len, min(ctx.min_q_len, max_q_len), decode_ctx, nh, nkv, hd, scale, window,
                        int(chunk), float(softcap), int(value_heads), _ptr(scratch), floats, _ptr(prefill_seqs), num_prefill,
-                       _stream())
+                       sink, _stream())
             if ctx.min_q_len <= 1:
                 self.launches += 1 if max_q_len <= 1 else 2          # decode + combine (+ prefill) in one call
             return out
@@ -733,7 +777,7 @@ class Ops:
                    _ptr(ctx.seq_of_token), q.shape[0], nh, nkv, hd, vd, scale, window, _DTYPE_CODE[q.dtype],
                    1 if weights == "sigmoid" else 0, _ptr(slopes), _ptr(head_bias), _ptr(head_gate),
                    head_gate.stride(0) if head_gate is not None else 0, float(softcap), int(chunk), int(value_heads),
-                   1 if out_f32 else 0, _stream())
+                   1 if out_f32 else 0, sink, _stream())
         return out
 
     def dense_prompt_attention_supported(self, q: torch.Tensor, nh: int, nkv: int, hd: int) -> bool:
@@ -822,10 +866,10 @@ class Ops:
                    _DTYPE_CODE[dtype], _stream())
         return out
 
-    UNARY_ACTIVATIONS = {"relu2": 0, "xielu": 1}
+    UNARY_ACTIVATIONS = {"relu2": 0, "xielu": 1, "tanh": 2}
 
     def unary_activation(self, x: torch.Tensor, kind: str, a: float = 0.0, b: float = 0.0) -> torch.Tensor:
-        """act(x), in place: "relu2" relu(x)^2; "xielu" a x^2 + x/2 for x > 0 and b (exp(x) - 1 - x) + x/2 for x <= 0."""
+        """act(x), in place: "relu2" relu(x)^2; "xielu" a x^2 + x/2 for x > 0 and b (exp(x) - 1 - x) + x/2 for x <= 0; "tanh"."""
         self._check(x, "x", tuple(_DTYPE_CODE))
         if kind not in self.UNARY_ACTIVATIONS:
             raise KernelError(f"unary_activation: kind {kind!r} of {sorted(self.UNARY_ACTIVATIONS)}")
@@ -877,28 +921,39 @@ class Ops:
         return y
 
     def recurrence_scan(self, prepared: torch.Tensor, v: torch.Tensor, ctx, binding, *, heads: int, dim: int, vdim: int,
-                        v_cols: int | None = None, beta: torch.Tensor | None = None) -> torch.Tensor:
+                        v_cols: int | None = None, beta: torch.Tensor | None = None, head_decay: torch.Tensor | None = None,
+                        bonus: torch.Tensor | None = None, qk_group: int = 1) -> torch.Tensor:
         """
         float32 [T, heads * vdim]: the scan of `linear_recurrence` from inputs the caller prepared: prepared
         float32 [3, T, heads * dim] (q, k, decay), v [T, heads * v_cols] (float32 or an activation dtype; value
         columns from v_cols to vdim are the constant 1), `beta` float32 [T, heads] for the delta rule.
-        The state slot holds [heads, dim, vdim] floats.
+        With `head_decay` (float32 [T, heads], delta rule only) prepared is [2, T, heads / qk_group * dim]: q and k,
+        each q/k head serving `qk_group` heads.  `bonus` (float32 [T, heads], plain recurrence): the read-out is of
+        the state before the token's own write, plus bonus * v.  The state slot holds [heads, dim, vdim] floats.
         """
         T = prepared.shape[1]
         v_cols = vdim if v_cols is None else v_cols
         self._check(prepared, "prepared", torch.float32, 3)
-        if tuple(prepared.shape) != (3, T, heads * dim):
-            raise KernelError(f"recurrence_scan: prepared is {tuple(prepared.shape)}, expected {(3, T, heads * dim)}")
+        if heads % qk_group or (qk_group > 1 and head_decay is None) or (head_decay is not None) > (beta is not None) or (
+                bonus is not None and beta is not None):
+            raise KernelError(f"recurrence_scan: {heads} heads in groups of {qk_group}; a decay a head goes with the delta rule, "
+                              "a bonus with the plain recurrence")
+        expected = (3, T, heads * dim) if head_decay is None else (2, T, heads // qk_group * dim)
+        if tuple(prepared.shape) != expected:
+            raise KernelError(f"recurrence_scan: prepared is {tuple(prepared.shape)}, expected {expected}")
         if v.dtype not in _DTYPE_CODE or v.dim() != 2 or v.stride(1) != 1 or tuple(v.shape) != (T, heads * v_cols):
             raise KernelError(f"recurrence_scan: v must be a [T, {heads * v_cols}] stretch")
-        if beta is not None:
-            self._check(beta, "beta", torch.float32, 2)
-            if tuple(beta.shape) != (T, heads):
-                raise KernelError(f"recurrence_scan: beta is {tuple(beta.shape)}, expected {(T, heads)}")
+        for t, name in ((beta, "beta"), (head_decay, "decay"), (bonus, "bonus")):
+            if t is not None:
+                self._check(t, name, torch.float32, 2)
+                if tuple(t.shape) != (T, heads):
+                    raise KernelError(f"recurrence_scan: {name} is {tuple(t.shape)}, expected {(T, heads)}")
         state, stride = self._state_floats(binding, heads * dim * vdim, "recurrence_scan")
         out = torch.empty((T, heads * vdim), dtype=torch.float32, device=v.device)
-        self._call("ts_recurrence_scan", _ptr(prepared), _ptr(v), v.stride(0), v_cols, _DTYPE_CODE[v.dtype], _ptr(beta),
-                   _ptr(ctx.cu_q), _ptr(binding.state_slots), binding.state_slots.shape[0], state.data_ptr(), stride,
+        mode = 3 if bonus is not None else 0 if beta is None else 1 if head_decay is None else 2
+        decay = prepared[2] if head_decay is None else head_decay
+        self._call("ts_recurrence_scan", _ptr(prepared), qk_group, _ptr(decay), mode, _ptr(v), v.stride(0), v_cols,
+                   _DTYPE_CODE[v.dtype], _ptr(beta if bonus is None else bonus), _ptr(ctx.cu_q), _ptr(binding.state_slots), binding.state_slots.shape[0], state.data_ptr(), stride,
                    _ptr(out), heads, dim, vdim, T, _stream())
         return out
 
@@ -924,6 +979,66 @@ class Ops:
                    b.stride(0), _ptr(prepared), _ptr(beta), T, heads, kv_heads, dim, unit_eps, q_scale,
                    _DTYPE_CODE[b.dtype], _stream())
         return prepared, beta
+
+    def delta_prepare_head(self, q: torch.Tensor, k: torch.Tensor, gates: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+                           *, heads: int, kv_heads: int, dim: int, unit_eps: float, q_scale: float):
+        """
+        `delta_prepare` with one decay a head: (prepared [2, T, kv_heads * dim], beta [T, heads], decay [T, heads]),
+        float32.  gates float32 [T, 2 heads]: the step sizes' logits, then the decays'; dt_bias, a_log [heads].
+        """
+        T = q.shape[0]
+        for t, name in ((q, "q"), (k, "k")):
+            if t.dtype != torch.float32 or t.stride(1) != 1 or tuple(t.shape) != (T, kv_heads * dim) or t.stride(0) != q.stride(0):
+                raise KernelError(f"delta_prepare_head: {name} must be a float32 [T, {kv_heads * dim}] stretch, of q's row stride")
+        self._check(gates, "gates", torch.float32, 2)
+        if tuple(gates.shape) != (T, 2 * heads) or dt_bias.numel() != heads or a_log.numel() != heads:
+            raise KernelError("delta_prepare_head: gates [T, 2 heads] and a bias and a rate a head are needed")
+        prepared = torch.empty((2, T, kv_heads * dim), dtype=torch.float32, device=q.device)
+        beta = torch.empty((T, heads), dtype=torch.float32, device=q.device)
+        decay = torch.empty_like(beta)
+        self._call("ts_delta_prepare_head", _ptr(q), _ptr(k), q.stride(0), _ptr(gates), _ptr(dt_bias), _ptr(a_log), _ptr(prepared),
+                   _ptr(beta), _ptr(decay), T, heads, kv_heads, dim, unit_eps, q_scale, _stream())
+        return prepared, beta, decay
+
+    def token_shift(self, x: torch.Tensor, mu: torch.Tensor, ctx, binding) -> torch.Tensor:
+        """
+        [S, T, width] in x's dtype: x[t] + (x'[t] - x[t]) * mu[s] for the S rows of mu (float32 [S, width]), x' the
+        request's row before t.  The row before a step's first token comes from the request's state slot (float32
+        [width]); `time_mix_prepare` moves it on.
+        """
+        self._check(x, "x", tuple(_DTYPE_CODE), 2)
+        self._check(mu, "mu", torch.float32, 2)
+        T, width = x.shape
+        if mu.shape[1] != width:
+            raise KernelError(f"token_shift: mu has rows of {mu.shape[1]} for x of {width}")
+        state, stride = self._state_floats(binding, width, "token_shift")
+        mixes = torch.empty((mu.shape[0], T, width), dtype=x.dtype, device=x.device)
+        self._call("ts_token_shift", _ptr(x), _ptr(mu), _ptr(ctx.seq_of_token), _ptr(ctx.cu_q), _ptr(binding.state_slots),
+                   state.data_ptr(), stride, _ptr(mixes), T, width, mu.shape[0], _DTYPE_CODE[x.dtype], _stream())
+        return mixes
+
+    def time_mix_prepare(self, r: torch.Tensor, k: torch.Tensor, z: torch.Tensor, w0: torch.Tensor, u: torch.Tensor,
+                         x: torch.Tensor, ctx, binding, *, heads: int, dim: int):
+        """
+        (prepared [3, T, heads * dim], bonus [T, heads]), float32, for the scan's bonus form: r and k as they are,
+        decays exp(-exp(z + w0)), bonus = sum over a head's channels of u k r.  Each request's last row of x (the
+        mixer's input) goes to its state slot (`binding`: the slots' previous rows).
+        """
+        T = r.shape[0]
+        for t, name in ((r, "r"), (k, "k")):
+            if t.dtype != x.dtype or t.stride(1) != 1 or tuple(t.shape) != (T, heads * dim) or t.stride(0) != r.stride(0):
+                raise KernelError(f"time_mix_prepare: {name} must be a [T, {heads * dim}] stretch of x's dtype, of r's row stride")
+        self._check(x, "x", tuple(_DTYPE_CODE), 2)
+        self._check(z, "decay logits", torch.float32, 2)
+        if tuple(z.shape) != (T, heads * dim) or w0.numel() != heads * dim or u.numel() != heads * dim:
+            raise KernelError("time_mix_prepare: decay logits [T, heads * dim], w0 and u [heads * dim] are needed")
+        state, stride = self._state_floats(binding, x.shape[1], "time_mix_prepare")
+        prepared = torch.empty((3, T, heads * dim), dtype=torch.float32, device=x.device)
+        bonus = torch.empty((T, heads), dtype=torch.float32, device=x.device)
+        self._call("ts_time_mix_prepare", _ptr(r), _ptr(k), r.stride(0), _ptr(z), _ptr(w0), _ptr(u), _ptr(prepared), _ptr(bonus),
+                   T, heads, dim, _ptr(x), x.shape[1], _ptr(ctx.cu_q), _ptr(binding.state_slots), binding.state_slots.shape[0],
+                   state.data_ptr(), stride, _DTYPE_CODE[x.dtype], _stream())
+        return prepared, bonus
 
     def mlstm_prepare(self, q: torch.Tensor, k: torch.Tensor, gates: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor,
                       ctx, binding, *, heads: int, dim: int, cap: float, q_scale: float, max_offset_floats: int):
@@ -1215,6 +1330,33 @@ class Ops:
         if out_dtype != x.dtype:
             return torch.mm(x, weight.t(), out_dtype=out_dtype, out=out)
         return torch.mm(x, weight.t(), out=out)
+
+    def linear_groups(self, x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:
+        """
+        [G, M, N]: x[g] [M, K] . weight[g] [N, K]^T for every g, one launch.  float32: the engine's FFMA kernel;
+        bfloat16: a few rows on the weight-streaming kernel (N a multiple of 16), else the library's batched product.
+        """
+        self._check(x, "x", tuple(_DTYPE_CODE), 3)
+        self._check(weight, "weight", x.dtype, 3)
+        G, M, K = x.shape
+        N = weight.shape[1]
+        if weight.shape[0] != G or weight.shape[2] != K:
+            raise KernelError(f"linear_groups: x {tuple(x.shape)}, weight {tuple(weight.shape)}")
+        out_dtype = out_dtype or x.dtype
+        if x.dtype == torch.float32 and out_dtype != torch.float32:
+            raise KernelError("linear_groups: the float32 product has float32 output")
+        out = torch.empty((G, M, N), dtype=out_dtype, device=x.device)
+        if x.dtype == torch.float32:
+            self._call("ts_sgemm_nt_batched", _ptr(x), _ptr(weight), _ptr(out), M, N, K, K, K, N, G, M * K, N * K, M * N, _stream())
+            return out
+        if N % 16 == 0 and self._skinny(x[0], weight):
+            self._call("ts_skinny_linear_groups", _ptr(weight), _ptr(x), _ptr(out), G, M, N, K, K, M * K, N, M * N,
+                       _DTYPE_CODE[out_dtype], _stream())
+            return out
+        self.calls["library_bmm"] = self.calls.get("library_bmm", 0) + 1
+        if out_dtype != x.dtype:
+            return torch.bmm(x, weight.transpose(1, 2), out_dtype=out_dtype)
+        return torch.bmm(x, weight.transpose(1, 2), out=out)
 
     def gemm_tcgen05(self, x: torch.Tensor, weight: torch.Tensor, *, swiglu: bool = False,
                      out_dtype: torch.dtype | None = None) -> torch.Tensor:

@@ -4,7 +4,8 @@ Arrangements: how a block wires its mixer, feed-forward and norms.
 "pre_norm" is the reference's decoder layer (model/llama.py:238-253): the residual add is deferred
 into the following norm, so a block takes and returns (branch output, residual stream).
 "sandwich_norm" also norms each sublayer's output and keeps the stream in float32;
-"pre_norm_stream" is the pre-norm wiring around a float32 stream.
+"pre_norm_stream" is the pre-norm wiring around a float32 stream; "post_norm_stream" norms the
+sublayers' outputs only.
 """
 
 from __future__ import annotations
@@ -168,3 +169,64 @@ class PreNormStreamBlock(PreNormBlock):
             return branch, residual
         h, residual = self.feed_forward_norm.forward(branch, residual)
         return PendingBranch(self.feed_forward.forward(h, ctx), None), residual
+
+
+@register_arrangement("post_norm_stream")
+class PostNormStreamBlock:
+    """
+    x = x + norm_a(mixer(x)); x = x + norm_b(ffn(x)) around a residual stream kept in float32: the sublayers
+    read the stream itself, rounded to the activation dtype.  A branch's norm, its addition and the next
+    sublayer's rounded input are one kernel; the block hands its last branch on unclosed (`PendingBranch`) and the
+    next block, or the model's final norm, closes it.  A mixer of two branches with norms of their own
+    (`forward_branches`) leaves those to the same kernel.  A block without a feed-forward ends after its mixer.
+    """
+
+    takes_token_ids = True
+    takes_embedding_scale = True
+
+    @staticmethod
+    def _members(spec: BlockSpec):
+        members = [("mixer", spec.mixer, spec.mixer_prefix), ("norm", spec.mixer_post_norm, spec.mixer_post_norm_prefix)]
+        if spec.feed_forward is not None:
+            members += [("feed_forward", spec.feed_forward, spec.feed_forward_prefix),
+                        ("norm", spec.feed_forward_post_norm, spec.feed_forward_post_norm_prefix)]
+        return members
+
+    @classmethod
+    def declare(cls, spec: BlockSpec) -> dict[str, TensorDecl]:
+        if spec.mixer_post_norm is None or (spec.feed_forward is not None and spec.feed_forward_post_norm is None):
+            raise ValueError("a post_norm_stream block needs a norm after each of its sublayers")
+        out: dict[str, TensorDecl] = {}
+        for role, part, prefix in cls._members(spec):
+            for name, decl in part_class(role, part).declare(part).items():
+                out[prefix + name] = decl
+        return out
+
+    def __init__(self, spec: BlockSpec, tensors: dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.spec = spec
+        built = [part_class(role, part)(part, _sub(tensors, prefix), rt) for role, part, prefix in self._members(spec)]
+        self.mixer, self.mixer_post_norm = built[:2]
+        self.mixer_norm = self.feed_forward_norm = None
+        self.feed_forward = self.feed_forward_post_norm = None
+        if spec.feed_forward is not None:
+            self.feed_forward, self.feed_forward_post_norm = built[2:]
+        branches = getattr(self.mixer, "forward_branches", None) if getattr(self.mixer, "norm_weights", None) else None
+        same_eps = float(getattr(self.mixer.spec, "norm_eps", -1.0)) == self.mixer_post_norm.eps
+        self._mixer_branches = branches if same_eps else None      # the closing kernel norms all with one eps
+
+    def forward(self, x, residual: torch.Tensor | None, ctx, binding, embedding: torch.Tensor | None = None,
+                embedding_scale: float = 1.0):
+        from tinyserve_llm_b200.parts.norm import PendingBranch
+        if embedding is not None:
+            h, residual = self.mixer_post_norm.start_and_copy(embedding, x, embedding_scale)
+        else:
+            h = x.closing.close_and_copy(x, residual)
+        if self._mixer_branches is not None:
+            tensor, pair = self._mixer_branches(h, ctx, binding)
+            branch = PendingBranch(tensor, self.mixer_post_norm, pair)
+        else:
+            branch = PendingBranch(self.mixer.forward(h, ctx, binding), self.mixer_post_norm)
+        if self.feed_forward is None:
+            return branch, residual
+        h = self.mixer_post_norm.close_and_copy(branch, residual)
+        return PendingBranch(self.feed_forward.forward(h, ctx), self.feed_forward_post_norm), residual

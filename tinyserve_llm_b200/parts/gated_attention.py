@@ -14,8 +14,11 @@ p; a distance penalty slope_h (i - j) taken off the score with slope_h = 2^(-c (
 number per head added to every score; sigmoid weights instead of a softmax (a visible key's weight is
 sigmoid(score), nothing is normalised over the keys); an output gate of one number a head; chunks of n
 positions, counted from the request's first token, outside of which a query sees nothing (the cache keeps
-the last n keys, as for a window of n); scores capped as c tanh(score / c).  With any of the last six the
-attention runs on the kernels that carry them (`paged_attention_split`'s options).
+the last n keys, as for a window of n); scores capped as c tanh(score / c); a norm of every head of q and of k
+without a weight; values that are the keys as projected (no tensor `v`: the same columns of the
+projection go to the key pool normed and rotated and to the value pool as they are); a sink, a score
+without a key or a value in every softmax's sum.  With a distance penalty, a head bias, sigmoid weights, a gate
+a head, chunks, a cap or a sink the attention runs on the kernels that carry them (`paged_attention_split`'s options).
 
 Keys (rotated) and values live in the paged cache; one kernel norms, rotates and stores, one attends
 (the tensor-core kernels where keys and values share a head size they take, the generic one else),
@@ -53,6 +56,14 @@ class GatedAttention(Mixer):
                 raise ValueError(f"{name}={size} is not supported: the attention kernels take up to {MAX_HEAD_DIM}")
         if spec.qk_norm_scope not in ("projection", "head") or spec.output_gate_scope not in ("channel", "head"):
             raise NotImplementedError(f"attention: norm scope {spec.qk_norm_scope!r}, gate scope {spec.output_gate_scope!r}")
+        if spec.values not in ("projected", "keys") or (spec.values == "keys" and spec.value_dim != spec.head_dim):
+            raise ValueError(f"attention: values {spec.values!r} with key heads of {spec.head_dim} and value heads of {spec.value_dim}")
+        if not spec.qk_norm_weight and (not spec.qk_norm or spec.qk_norm_scope != "head"):
+            raise NotImplementedError("attention: a norm of q and k without a weight is one a head")
+        if spec.values == "keys" and spec.bias:
+            raise NotImplementedError("attention: values that are the keys have no bias of their own")
+        if spec.sink is not None and spec.weights != "softmax":
+            raise NotImplementedError("attention: a sink belongs to the softmax")
         if spec.weights not in ("softmax", "sigmoid"):
             raise NotImplementedError(f"attention: weights {spec.weights!r}; have softmax and sigmoid")
         if spec.q_temperature_every < 0 or spec.distance_slope_exponent < 0 or spec.window < 0 or spec.chunk < 0 or spec.softcap < 0:
@@ -64,10 +75,12 @@ class GatedAttention(Mixer):
         nq, nk, nv = spec.num_heads * spec.head_dim, spec.num_kv_heads * spec.head_dim, spec.num_kv_heads * spec.value_dim
         no = spec.num_heads * spec.value_dim
         out = {"q": TensorDecl((nq, spec.hidden_size)), "k": TensorDecl((nk, spec.hidden_size)),
-               "v": TensorDecl((nv, spec.hidden_size)), "o": TensorDecl((spec.hidden_size, no))}
+               "o": TensorDecl((spec.hidden_size, no))}
+        if spec.values == "projected":
+            out["v"] = TensorDecl((nv, spec.hidden_size))
         if spec.bias:
             out.update({"q.b": TensorDecl((nq,)), "k.b": TensorDecl((nk,)), "v.b": TensorDecl((nv,))})
-        if spec.qk_norm:
+        if spec.qk_norm and spec.qk_norm_weight:
             per_head = spec.qk_norm_scope == "head"
             out.update({"q.norm": TensorDecl((spec.head_dim if per_head else nq,), init="unit"),
                         "k.norm": TensorDecl((spec.head_dim if per_head else nk,), init="unit")})
@@ -81,12 +94,12 @@ class GatedAttention(Mixer):
         super().__init__(spec, tensors, rt)
         self.validate(spec)
         f32 = dict(device=rt.device, dtype=torch.float32)
-        rows = [tensors["q"], tensors["k"], tensors["v"]] + ([tensors["g"]] if spec.output_gate else [])
+        rows = [tensors[n] for n in ["q", "k"] + (["v"] if spec.values == "projected" else []) + (["g"] if spec.output_gate else [])]
         self.input_rows = fuse_rows(rows)
         self.out_weight = tensors["o"]
         self.inner_width = spec.num_heads * spec.value_dim
         self.biases = tuple(tensors[n].to(**f32).contiguous() for n in ("q.b", "k.b", "v.b")) if spec.bias else None
-        self.norm_weights = tuple(tensors[n].to(**f32).contiguous() for n in ("q.norm", "k.norm")) if spec.qk_norm else None
+        self.norm_weights = tuple(tensors[n].to(**f32).contiguous() for n in ("q.norm", "k.norm")) if spec.qk_norm and spec.qk_norm_weight else None
         self.head_bias = tensors["pb"].to(**f32).contiguous() if spec.head_bias else None
         self.slopes = None
         if spec.distance_slope_exponent > 0:
@@ -110,17 +123,22 @@ class GatedAttention(Mixer):
 
     def inner(self, y: torch.Tensor, x: torch.Tensor, ctx, binding, scale: float = 1.0,
               out: torch.Tensor | None = None) -> torch.Tensor:
-        """y: this mixer's columns of the projection of x, [q | k | v | g].  Returns [T, heads * value_dim] * scale."""
+        """y: this mixer's columns of the projection of x, [q | k | v | g] (no v where the keys are the values).  Returns [T, heads * value_dim] * scale."""
         s, ops = self.spec, self.rt.ops
         nq, nk, nv = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim, s.num_kv_heads * s.value_dim
-        q = ops.qk_norm_rope_store(y, (0, nq, nq + nk), self.biases, self.norm_weights, s.qk_norm_eps, self.position,
+        v_at = nq + nk
+        if s.values == "keys":
+            v_at, nv = nq, 0
+        q = ops.qk_norm_rope_store(y, (0, nq, v_at), self.biases, self.norm_weights, s.qk_norm_eps, self.position,
                                    ctx, binding, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim,
-                                   norm_per_head=s.qk_norm_scope == "head", q_temperature=self.q_temperature)
+                                   norm_per_head=s.qk_norm_scope == "head", q_temperature=self.q_temperature,
+                                   unweighted_norm=s.qk_norm and not s.qk_norm_weight)
         gate = y[:, nq + nk + nv:nq + nk + nv + self.gate_width] if s.output_gate else None
         per_head_gate = s.output_gate and s.output_gate_scope == "head"
         o = ops.paged_attention_split(q, ctx, binding, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, s.scale, s.window,
                                       weights=s.weights, slopes=self.slopes, head_bias=self.head_bias,
-                                      head_gate=gate if per_head_gate else None, softcap=s.softcap, chunk=s.chunk)
+                                      head_gate=gate if per_head_gate else None, softcap=s.softcap, chunk=s.chunk,
+                                      sink=s.sink)
         if per_head_gate:                               # the gate went into the attention kernel's last step
             if scale != 1.0:
                 o = o * scale

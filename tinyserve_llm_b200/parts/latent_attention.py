@@ -94,6 +94,8 @@ class LatentAttention(Mixer):
             if getattr(self.position, "frequencies", None) is None or self.position.dims != spec.rot_dim:
                 raise NotImplementedError("latent attention rotates inside its kernels: it takes a position part with "
                                           "`frequencies` over exactly rot_dim channels")
+            if getattr(self.position, "interleaved", False):
+                raise NotImplementedError("latent attention rotates by halves, not by neighbouring channels")
             self.frequencies = self.position.frequencies
 
     def kv_need(self) -> KVNeed:

@@ -13,7 +13,7 @@ import torch
 
 from tinyserve_llm_b200.config.spec import ModelSpec
 from tinyserve_llm_b200.parts import (attention, delta_rule, differential_attention, gated_attention, latent_attention,  # noqa: F401  (registration)
-                                      mingru, mlp, mlstm, norm, parallel, recurrence, rotary, routed_experts)
+                                      mingru, mlp, mlstm, norm, parallel, recurrence, rotary, routed_experts, time_mixing)
 from tinyserve_llm_b200.parts.base import KVNeed, Runtime, TensorDecl, arrangement_class, part_class
 from tinyserve_llm_b200.parts.block import _sub
 from tinyserve_llm_b200.parts.linear import Linear

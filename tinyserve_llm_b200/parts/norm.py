@@ -48,11 +48,12 @@ class PendingBranch:
     their sublayers hand this on as `x`, the next block's first norm (or the model's final norm) takes it.
     """
 
-    __slots__ = ("tensor", "closing")
+    __slots__ = ("tensor", "closing", "pair")
 
-    def __init__(self, tensor: torch.Tensor, closing: "StreamRMSNorm | None") -> None:
+    def __init__(self, tensor: torch.Tensor, closing: "StreamRMSNorm | None", pair: tuple | None = None) -> None:
         self.tensor = tensor
         self.closing = closing
+        self.pair = pair          # a sublayer of two normed branches: the second one and the norms (see `Ops.stream_norm`)
 
 
 @register_part("norm", "rmsnorm_stream")
@@ -80,13 +81,28 @@ class StreamRMSNorm(Norm):
     def forward(self, x, residual: torch.Tensor | None, rows: torch.Tensor | None = None):
         if residual is None:
             raise ValueError("a stream norm needs the residual stream (the first norm starts it from the embedding)")
-        branch = closing = None
+        branch = closing = pair = None
         if isinstance(x, PendingBranch):
-            branch, closing = x.tensor, (x.closing.weight if x.closing is not None else None)
+            branch, closing, pair = x.tensor, (x.closing.weight if x.closing is not None else None), x.pair
+            if pair is not None and self.centered:
+                raise NotImplementedError("the branches of a pair are RMS-normed")
         elif x is not None:
             raise ValueError("a stream norm takes a PendingBranch (a sublayer's output and its closing norm) or nothing")
         out = self.rt.ops.stream_norm(branch, closing, residual, self.weight, self.eps, self.rt.dtype, rows=rows,
-                                      centered=self.centered, plain_add=branch is not None and closing is None)
+                                      centered=self.centered, plain_add=branch is not None and closing is None, pair=pair)
+        return out, residual
+
+    def close_and_copy(self, x: PendingBranch, residual: torch.Tensor) -> torch.Tensor:
+        """stream += closing(branch) with this norm as the closing one; returns the new stream in the activation dtype, unnormed."""
+        if self.centered:
+            raise NotImplementedError("a branch is closed by an RMS norm")
+        return self.rt.ops.stream_norm(x.tensor, self.weight, residual, None, self.eps, self.rt.dtype, copy_out=True, pair=x.pair)
+
+    def start_and_copy(self, table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
+        """(the rows table[ids] * scale in the activation dtype, the stream they start): a stream whose sublayers read it unnormed."""
+        residual = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.float32, device=table.device)
+        out = self.rt.ops.stream_norm(None, None, residual, None, self.eps, self.rt.dtype, table=table, ids=ids, scale=scale,
+                                      copy_out=True)
         return out, residual
 
     def close(self, branch: torch.Tensor, residual: torch.Tensor) -> None:

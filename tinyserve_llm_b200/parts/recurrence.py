@@ -85,6 +85,8 @@ class LinearRecurrence(Mixer):
             self.position = part_class("position", spec.position)(spec.position, {}, rt)
             if getattr(self.position, "frequencies", None) is None:
                 raise NotImplementedError("the recurrence rotates q and k itself: it takes a position part with `frequencies`")
+            if getattr(self.position, "interleaved", False):
+                raise NotImplementedError("the recurrence rotates by halves of a head, not by neighbouring channels")
 
     def state_bytes(self) -> int:
         return self.spec.num_heads * self.spec.key_dim * self.spec.value_dim * 4

@@ -87,7 +87,8 @@ class InlineRotary(PositionEncoding):
     """
     Rotate-half rotation whose angles the kernels compute themselves, position * frequencies[i] in
     float32 with frequencies[i] = base^(-2i/dims) (rescaled by the spec's `yarn` or `bands`): no table,
-    so no longest position.  Mixers that rotate inside their own kernels read `dims` and `frequencies`.
+    so no longest position.  Mixers that rotate inside their own kernels read `dims` and `frequencies`, and
+    `interleaved` (channel 2i paired with 2i + 1); one whose kernel pairs halves only must refuse the latter.
     """
 
     def __init__(self, spec, tensors: dict[str, torch.Tensor], rt: Runtime) -> None:
@@ -104,6 +105,7 @@ class InlineRotary(PositionEncoding):
                 freq = yarn_frequencies(spec.dims, float(spec.base), spec.yarn)
             rt.shared[key] = freq.to(torch.float32).to(rt.device)
         self.dims = spec.dims
+        self.interleaved = bool(getattr(spec, "interleaved", False))
         self.frequencies = rt.shared[key]
         # cos and sin are multiplied by this (1 without YaRN); a kernel that rotates with a YaRN rescaling has to apply it
         self.magnitude = 1.0 if spec.yarn is None else 0.1 * math.log(spec.yarn.factor) + 1.0
