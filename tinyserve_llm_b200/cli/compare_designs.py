@@ -1,9 +1,9 @@
 """
 Prefill and decode throughput of a design at layer sizes that resemble a real model's, beside the
 engine's closest other design at equal width and depth (Duduvik beside Llama, Nipizen beside
-Duduvik, Lugipel beside Nipizen, Folavik beside Llama), both with random weights through the engine's own step function:
+Duduvik, Lugipel beside Nipizen, Folavik beside Llama, Fuvipel beside Nipizen), both with random weights through the engine's own step function:
 
-    python bench.py --design duduvik|nipizen|lugipel|folavik [--size small|medium|large] [--steps K] [--warmup W]
+    python bench.py --design duduvik|nipizen|lugipel|folavik|fuvipel [--size small|medium|large] [--steps K] [--warmup W]
 
 For each design: a prompt of `prefill` tokens in one step (launched kernel by kernel), and decode
 steps of `batch` requests at `context` tokens each (replayed from a CUDA graph), timed on the device
@@ -117,6 +117,26 @@ def folavik_config(s: dict) -> dict:
     mixers = (diff, lat, att)
     return {"architecture": "Folavik", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
             "logit_softcap": 30.0, "layers": [dict(mixers[i % 3], mlp=dense) for i in range(s["layers"])]}
+
+
+def fuvipel_config(s: dict) -> dict:
+    """
+    Layers in the order delta rule / parallel (attention beside time mixing) / delta rule, every one with a dense
+    squared-relu feed-forward.  Attention heads of 128 channels (keys as values), so that the tensor-core attention
+    kernels take them, 4 query heads a key/value head; delta rules of `heads` value heads over a quarter as many q/k
+    heads; time mixing of `heads` heads; recurrent heads of 128 channels throughout.
+    """
+    width, heads = s["width"], s["heads"]
+    dim = width // heads                                   # 128 at every size
+    rule = {"type": "delta", "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "conv": 4}}
+    par = {"type": "parallel",
+           "mixer": {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                              "rot": {"base": 500000.0, "dims": dim}},
+                     "right": {"heads": heads, "dim": dim, "decay_rank": 64}}}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    mixers = (rule, par, rule)
+    return {"architecture": "Fuvipel", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6},
+            "layers": [dict(mixers[i % 3], mlp=dense) for i in range(s["layers"])]}
 
 
 def llama_config(s: dict) -> dict:
@@ -252,8 +272,10 @@ def run(design: str, size: str, steps: int, warmup: int, peaks: dict) -> int:
         pair = (("nipizen", nipizen_config(s), True), ("lugipel", lugipel_config(s), True))
     elif design == "folavik":
         pair = (("llama", llama_config(s), True), ("folavik", folavik_config(s), True))
+    elif design == "fuvipel":
+        pair = (("nipizen", nipizen_config(s), True), ("fuvipel", fuvipel_config(s), True))
     else:
-        raise SystemExit(f"--design {design!r}: have ['duduvik', 'nipizen', 'lugipel', 'folavik']")
+        raise SystemExit(f"--design {design!r}: have ['duduvik', 'nipizen', 'lugipel', 'folavik', 'fuvipel']")
     for name, cfg, profile in pair:
         record = {"design": name, "size": size, "width": s["width"], "layers": s["layers"], "dtype": "bf16",
                   "data": "synthetic", "timing": "CUDA events, median, L2 flushed between timed steps", "peaks": peaks}
