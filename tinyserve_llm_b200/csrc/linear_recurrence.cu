@@ -91,6 +91,7 @@ struct RecurrenceArgs {
     float* state; long long slot_stride;              // floats between slots; a slot holds [heads, dim, vdim]
     float* out;                                       // [tokens, heads * vdim] float32
     int heads, dim, vdim;
+    int singles;                                      // 1: only requests that feed one token (prompt portions: recurrence_tiles.cu)
 };
 
 // COLS: value channels of a CTA (16; the delta rule, whose tokens are a chain of dependent steps, runs 8 a CTA so that
@@ -115,6 +116,7 @@ linear_recurrence_kernel(RecurrenceArgs p) {
     const int slot = p.slots[seq];
     const int begin = p.cu_q[seq], end = p.cu_q[seq + 1];
     if (slot < 0 || end <= begin) return;                // a padding request, or one that feeds nothing
+    if (p.singles && end - begin > 1) return;
     // plain: the threads of a row group are neighbours (their loads of a state row coalesce); delta rule: the
     // sixteen row groups of a column are the lanes of half a warp
     const int r = DELTA ? threadIdx.x % LR_ROWGROUPS : threadIdx.x / COLS;
@@ -333,10 +335,11 @@ static int launch_recurrence(const RecurrenceArgs& p, int mode, int num_seqs, cu
 // (q and k as they enter the recurrence), decay [tokens, heads * dim], v [tokens, heads * v_cols] in float32 or the
 // activation dtype.  `mode` 0: plain; 1: delta rule with the step sizes `coef` [tokens, heads]; 2: the same with the
 // decay [tokens, heads]; 3: bonus form with `coef` [tokens, heads].  A slot holds [heads, dim, vdim] floats.
+// `singles` 1: only requests that feed one token are walked.
 TS_API int ts_recurrence_scan(const float* qk, int qk_group, const float* decay, int mode, const void* v,
                               long long v_stride, int v_cols, int v_dtype, const float* coef, const int* cu_q,
                               const int* slots, int num_seqs, float* state, long long slot_stride, float* out, int heads,
-                              int dim, int vdim, int num_tokens, cudaStream_t stream) {
+                              int dim, int vdim, int num_tokens, int singles, cudaStream_t stream) {
     TS_REQUIRE(heads > 0 && dim > 0 && vdim > 0 && num_seqs >= 0 && num_tokens >= 0, "recurrence_scan: bad sizes");
     TS_REQUIRE(dim <= 16 * LR_ROWGROUPS, "recurrence_scan: %d key channels a head are not supported (up to %d)", dim,
                16 * LR_ROWGROUPS);
@@ -347,7 +350,7 @@ TS_API int ts_recurrence_scan(const float* qk, int qk_group, const float* decay,
     TS_REQUIRE(num_seqs <= 65535 && heads <= 65535, "recurrence_scan: grid too large");
     if (num_seqs == 0 || num_tokens == 0) return 0;
     RecurrenceArgs p{qk, (long long)num_tokens * (heads / qk_group) * dim, qk_group, decay, v, v_stride, v_cols, coef, cu_q,
-                     slots, state, slot_stride, out, heads, dim, vdim};
+                     slots, state, slot_stride, out, heads, dim, vdim, singles};
     if (v_dtype == TS_F32) return launch_recurrence<float>(p, mode, num_seqs, stream);
     if (v_dtype == TS_BF16) return launch_recurrence<__nv_bfloat16>(p, mode, num_seqs, stream);
     return ts_fail("recurrence_scan: unknown dtype code %d", v_dtype);
@@ -383,7 +386,7 @@ TS_API int ts_linear_recurrence(const void* q, const void* k, const void* v, lon
         return ts_fail("linear_recurrence: unknown dtype code %d", dtype);
     TS_LAUNCH_CHECK("linear_recurrence (prepare)");
     RecurrenceArgs p{prepared, total, 1, prepared + 2 * total, v, v_stride, vdim, nullptr, cu_q, slots, state, slot_stride, out,
-                     heads, dim, vdim};
+                     heads, dim, vdim, 0};
     if (dtype == TS_F32) return launch_recurrence<float>(p, LR_PLAIN, num_seqs, stream);
     return launch_recurrence<__nv_bfloat16>(p, LR_PLAIN, num_seqs, stream);
 }

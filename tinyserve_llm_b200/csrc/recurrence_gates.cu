@@ -72,18 +72,27 @@ TS_API int ts_delta_prepare(const float* q, const float* k, long long qk_stride,
     return 0;
 }
 
+// With `single_of` (the request of every token): whether the token's request feeds it alone (a padding row does not).
+__device__ __forceinline__ bool feeds_one(const int* single_of, const int* cu_q, long long t) {
+    if (!single_of) return true;
+    const int seq = single_of[t];
+    return seq >= 0 && cu_q[seq + 1] - cu_q[seq] == 1;
+}
+
 // The same with one decay a head: one warp a (token, q/k head), which also takes its value heads' gates.  gates
 // [tokens, 2 heads] float32 holds the step sizes' logits, then the decays'; prepared is [2][tokens, kv_heads * dim],
-// beta and decay [tokens, heads].
+// beta and decay [tokens, heads].  `single_of` (optional): only tokens of requests that feed one are prepared.
 __global__ void delta_prepare_head_kernel(const float* __restrict__ q, const float* __restrict__ k, long long qk_stride,
                                           const float* __restrict__ gates, const float* __restrict__ dt_bias,
                                           const float* __restrict__ a_log, float* __restrict__ prepared,
                                           float* __restrict__ beta, float* __restrict__ decay, long long items, int heads,
-                                          int kv_heads, int dim, float unit_eps, float q_scale) {
+                                          int kv_heads, int dim, float unit_eps, float q_scale,
+                                          const int* __restrict__ single_of, const int* __restrict__ cu_q) {
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (item >= items) return;
     const int lane = threadIdx.x & 31;
     const long long t = item / kv_heads;
+    if (!feeds_one(single_of, cu_q, t)) return;
     const int g = (int)(item % kv_heads), group = heads / kv_heads;
     const float* qr = q + t * qk_stride + (long long)g * dim;
     const float* kr = k + t * qk_stride + (long long)g * dim;
@@ -106,13 +115,13 @@ __global__ void delta_prepare_head_kernel(const float* __restrict__ q, const flo
 TS_API int ts_delta_prepare_head(const float* q, const float* k, long long qk_stride, const float* gates,
                                  const float* dt_bias, const float* a_log, float* prepared, float* beta, float* decay,
                                  int num_tokens, int heads, int kv_heads, int dim, float unit_eps, float q_scale,
-                                 cudaStream_t stream) {
+                                 const int* single_of, const int* cu_q, cudaStream_t stream) {
     TS_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0, "delta_prepare: %d heads over %d q/k heads",
                heads, kv_heads);
     if (num_tokens <= 0) return 0;
     const long long items = (long long)num_tokens * kv_heads;
     delta_prepare_head_kernel<<<(unsigned)((items + 3) / 4), 128, 0, stream>>>(q, k, qk_stride, gates, dt_bias, a_log, prepared,
-        beta, decay, items, heads, kv_heads, dim, unit_eps, q_scale);
+        beta, decay, items, heads, kv_heads, dim, unit_eps, q_scale, single_of, cu_q);
     TS_LAUNCH_CHECK("delta_prepare_head");
     return 0;
 }
@@ -168,7 +177,7 @@ __global__ void time_mix_prepare_kernel(const T* __restrict__ r, const T* __rest
                                         float* __restrict__ prepared, float* __restrict__ bonus, long long items, int heads,
                                         int dim, unsigned item_blocks, const T* __restrict__ x, int width,
                                         const int* __restrict__ cu_q, const int* __restrict__ slots, int num_seqs,
-                                        float* __restrict__ state, long long slot_stride) {
+                                        float* __restrict__ state, long long slot_stride, const int* __restrict__ single_of) {
     const int lane = threadIdx.x & 31;
     if (blockIdx.x >= item_blocks) {
         const int stretches = (width + 127) / 128;
@@ -184,6 +193,7 @@ __global__ void time_mix_prepare_kernel(const T* __restrict__ r, const T* __rest
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (item >= items) return;
     const long long t = item / heads;
+    if (!feeds_one(single_of, cu_q, t)) return;
     const int h = (int)(item % heads);
     const T* rr = r + t * rk_stride + (long long)h * dim;
     const T* kr = k + t * rk_stride + (long long)h * dim;
@@ -202,22 +212,26 @@ __global__ void time_mix_prepare_kernel(const T* __restrict__ r, const T* __rest
 
 // r, k: [tokens, heads * dim] with one row stride; z float32 [tokens, heads * dim]; prepared [3][tokens, heads * dim],
 // bonus [tokens, heads].  `x` [tokens, width] is the mixer's input, whose last row of every request goes to its slot.
+// `portions_only` 1: no token is prepared, the rows move on all the same; `single_of` (optional): only tokens of
+// requests that feed one are prepared.
 TS_API int ts_time_mix_prepare(const void* r, const void* k, long long rk_stride, const float* z, const float* w0,
                                const float* u, float* prepared, float* bonus, int num_tokens, int heads, int dim,
                                const void* x, int width, const int* cu_q, const int* slots, int num_seqs, float* state,
-                               long long slot_stride, int dtype, cudaStream_t stream) {
+                               long long slot_stride, int portions_only, const int* single_of, int dtype,
+                               cudaStream_t stream) {
     TS_REQUIRE(heads > 0 && dim > 0 && width > 0 && slot_stride >= width, "time_mix_prepare: bad sizes");
-    if (num_tokens <= 0) return 0;
-    const long long items = (long long)num_tokens * heads;
+    if (num_tokens <= 0 || num_seqs <= 0) return 0;
+    const long long items = portions_only ? 0 : (long long)num_tokens * heads;
     const unsigned item_blocks = (unsigned)((items + 3) / 4);
     const unsigned more = (unsigned)(((long long)num_seqs * ((width + 127) / 128) + 3) / 4);
     if (dtype == TS_F32)
         time_mix_prepare_kernel<float><<<item_blocks + more, 128, 0, stream>>>((const float*)r, (const float*)k, rk_stride, z, w0, u,
-            prepared, bonus, items, heads, dim, item_blocks, (const float*)x, width, cu_q, slots, num_seqs, state, slot_stride);
+            prepared, bonus, items, heads, dim, item_blocks, (const float*)x, width, cu_q, slots, num_seqs, state, slot_stride,
+            single_of);
     else if (dtype == TS_BF16)
         time_mix_prepare_kernel<__nv_bfloat16><<<item_blocks + more, 128, 0, stream>>>((const __nv_bfloat16*)r, (const __nv_bfloat16*)k,
             rk_stride, z, w0, u, prepared, bonus, items, heads, dim, item_blocks, (const __nv_bfloat16*)x, width, cu_q, slots,
-            num_seqs, state, slot_stride);
+            num_seqs, state, slot_stride, single_of);
     else
         return ts_fail("time_mix_prepare: unknown dtype code %d", dtype);
     TS_LAUNCH_CHECK("time_mix_prepare");

@@ -79,10 +79,14 @@ _SIGNATURES = {
     "ts_sigmoid_gate": ("int", "plplpliifip"),
     "ts_paged_attention_split": ("int", "plpppllllii" "pippiiiiifiip"),
     "ts_short_conv_silu": ("int", "plppppiplpiiiip"),
-    "ts_recurrence_scan": ("int", "pipi" "pliipppiplpiiiip"),
-    "ts_delta_prepare_head": ("int", "pplpppppp" "iiiiffp"),
+    "ts_recurrence_scan": ("int", "pipi" "pliipppiplpiiiiip"),
+    "ts_delta_prepare_head": ("int", "pplpppppp" "iiiiffppp"),
     "ts_token_shift": ("int", "pppppplp" "iiiip"),
-    "ts_time_mix_prepare": ("int", "pplppppp" "iiipippiplip"),
+    "ts_time_mix_prepare": ("int", "pplppppp" "iiipippiplipip"),
+    "ts_recurrence_tiles_pack_floats": ("long long", "iiii"),
+    "ts_recurrence_tiles_coef_floats": ("long long", "iii"),
+    "ts_delta_tiles": ("int", "pplppppl" "pppii" "plppp" "iiiiffp"),
+    "ts_mix_tiles": ("int", "pplppppl" "pppii" "plppp" "iiip"),
     "ts_delta_prepare": ("int", "pplppppl" "ppiiiiffip"),
     "ts_mlstm_prepare": ("int", "ppllpplppffppiplpppiiiip"),
     "ts_row_scaled_activation": ("int", "ppppiiiip"),
@@ -178,6 +182,8 @@ class Ops:
         # 3.2 1B's sizes, whole decode steps: 4 to 6 % faster than the library product plus the activation kernel at 12,
         # 16, 24 and 32 rows, since the weights go through the cp.async ring)
         self.swiglu_skinny_rows = self.skinny_max_rows
+        # TINYSERVE_B200_TILES=0 keeps the recurrences that have a form of sixteen tokens at a time on the scan token by token
+        self.recurrence_tiles = os.environ.get("TINYSERVE_B200_TILES", "1") != "0"
         # from this many (token, expert) pairs a routed feed-forward's bfloat16 products go to the library's grouped product
         self.grouped_mm_min_pairs = int(os.environ.get("TINYSERVE_B200_GROUPED_PAIRS", "256"))
 
@@ -922,14 +928,16 @@ class Ops:
 
     def recurrence_scan(self, prepared: torch.Tensor, v: torch.Tensor, ctx, binding, *, heads: int, dim: int, vdim: int,
                         v_cols: int | None = None, beta: torch.Tensor | None = None, head_decay: torch.Tensor | None = None,
-                        bonus: torch.Tensor | None = None, qk_group: int = 1) -> torch.Tensor:
+                        bonus: torch.Tensor | None = None, qk_group: int = 1, singles: bool = False,
+                        out: torch.Tensor | None = None) -> torch.Tensor:
         """
         float32 [T, heads * vdim]: the scan of `linear_recurrence` from inputs the caller prepared: prepared
         float32 [3, T, heads * dim] (q, k, decay), v [T, heads * v_cols] (float32 or an activation dtype; value
         columns from v_cols to vdim are the constant 1), `beta` float32 [T, heads] for the delta rule.
         With `head_decay` (float32 [T, heads], delta rule only) prepared is [2, T, heads / qk_group * dim]: q and k,
         each q/k head serving `qk_group` heads.  `bonus` (float32 [T, heads], plain recurrence): the read-out is of
-        the state before the token's own write, plus bonus * v.  The state slot holds [heads, dim, vdim] floats.
+        the state before the token's own write, plus bonus * v.  `singles`: only requests that feed one token are
+        walked, the other rows of `out` are left alone.  The state slot holds [heads, dim, vdim] floats.
         """
         T = prepared.shape[1]
         v_cols = vdim if v_cols is None else v_cols
@@ -949,12 +957,78 @@ class Ops:
                 if tuple(t.shape) != (T, heads):
                     raise KernelError(f"recurrence_scan: {name} is {tuple(t.shape)}, expected {(T, heads)}")
         state, stride = self._state_floats(binding, heads * dim * vdim, "recurrence_scan")
-        out = torch.empty((T, heads * vdim), dtype=torch.float32, device=v.device)
+        out = self._scan_out(out, T, heads * vdim, v.device)
         mode = 3 if bonus is not None else 0 if beta is None else 1 if head_decay is None else 2
         decay = prepared[2] if head_decay is None else head_decay
         self._call("ts_recurrence_scan", _ptr(prepared), qk_group, _ptr(decay), mode, _ptr(v), v.stride(0), v_cols,
                    _DTYPE_CODE[v.dtype], _ptr(beta if bonus is None else bonus), _ptr(ctx.cu_q), _ptr(binding.state_slots), binding.state_slots.shape[0], state.data_ptr(), stride,
-                   _ptr(out), heads, dim, vdim, T, _stream())
+                   _ptr(out), heads, dim, vdim, T, 1 if singles else 0, _stream())
+        return out
+
+    def _scan_out(self, out: torch.Tensor | None, rows: int, cols: int, device) -> torch.Tensor:
+        if out is None:
+            return torch.empty((rows, cols), dtype=torch.float32, device=device)
+        self._check(out, "out", torch.float32, 2)
+        if tuple(out.shape) != (rows, cols):
+            raise KernelError(f"a scan's out is {tuple(out.shape)}, expected {(rows, cols)}")
+        return out
+
+    def portions_by_tiles(self, ctx) -> bool:
+        """Whether the step holds prompt portions that the kernels of `delta_tiles` and `mix_tiles` take (a bare context may not list them)."""
+        return bool(self.recurrence_tiles and ctx.max_q_len > 1 and getattr(ctx, "prefill_seqs", None) is not None
+                    and ctx.prefill_seqs.shape[0] > 0)
+
+    def _tile_buffers(self, ctx, T: int, qk_heads: int, heads: int, dim: int, device) -> tuple[torch.Tensor, torch.Tensor]:
+        seqs = ctx.cu_q.shape[0] - 1
+        floats = (int(self.lib.ts_recurrence_tiles_pack_floats(T, seqs, qk_heads, dim)),
+                  int(self.lib.ts_recurrence_tiles_coef_floats(T, seqs, heads)))
+        return tuple(torch.empty((n,), dtype=torch.float32, device=device) for n in floats)
+
+    def delta_tiles(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.Tensor, dt_bias: torch.Tensor,
+                    a_log: torch.Tensor, ctx, binding, *, heads: int, kv_heads: int, dim: int, vdim: int, unit_eps: float,
+                    q_scale: float) -> torch.Tensor:
+        """
+        `delta_prepare_head` and its scan for the step's prompt portions, sixteen tokens at a time: float32
+        [T, heads * vdim], of which the rows of requests that feed one token are left unwritten.  q, k, v float32
+        stretches after the convolution, gates [T, 2 heads].
+        """
+        T = q.shape[0]
+        for t, name, cols in ((q, "q", kv_heads * dim), (k, "k", kv_heads * dim), (v, "v", heads * vdim)):
+            if t.dtype != torch.float32 or t.stride(1) != 1 or tuple(t.shape) != (T, cols) or (name == "k" and t.stride(0) != q.stride(0)):
+                raise KernelError(f"delta_tiles: {name} must be a float32 [T, {cols}] stretch (q and k of one row stride)")
+        self._check(gates, "gates", torch.float32, 2)
+        if tuple(gates.shape) != (T, 2 * heads) or dt_bias.numel() != heads or a_log.numel() != heads:
+            raise KernelError("delta_tiles: gates [T, 2 heads] and a bias and a rate a head are needed")
+        state, stride = self._state_floats(binding, heads * dim * vdim, "delta_tiles")
+        pack, coef = self._tile_buffers(ctx, T, kv_heads, heads, dim, q.device)
+        out = torch.empty((T, heads * vdim), dtype=torch.float32, device=q.device)
+        self._call("ts_delta_tiles", _ptr(q), _ptr(k), q.stride(0), _ptr(gates), _ptr(dt_bias), _ptr(a_log), _ptr(v), v.stride(0),
+                   _ptr(ctx.cu_q), _ptr(binding.state_slots), _ptr(ctx.prefill_seqs), ctx.prefill_seqs.shape[0], ctx.max_q_len,
+                   state.data_ptr(), stride, _ptr(pack), _ptr(coef), _ptr(out), heads, kv_heads, dim, vdim, unit_eps, q_scale, _stream())
+        self.launches += 1                                   # what the columns of a tile share, then the scan
+        return out
+
+    def mix_tiles(self, r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, w0: torch.Tensor, u: torch.Tensor,
+                  ctx, binding, *, heads: int, dim: int) -> torch.Tensor:
+        """
+        The scan's bonus form (see `time_mix_prepare`) for the step's prompt portions, sixteen tokens at a time: float32
+        [T, heads * dim], of which the rows of requests that feed one token are left unwritten.
+        """
+        T = r.shape[0]
+        for t, name in ((r, "r"), (k, "k"), (v, "v")):
+            if t.dtype != r.dtype or t.dtype not in _DTYPE_CODE or t.stride(1) != 1 or tuple(t.shape) != (T, heads * dim) or (
+                    name == "k" and t.stride(0) != r.stride(0)):
+                raise KernelError(f"mix_tiles: {name} must be a [T, {heads * dim}] stretch of an activation dtype (r and k of one row stride)")
+        self._check(z, "decay logits", torch.float32, 2)
+        if tuple(z.shape) != (T, heads * dim) or w0.numel() != heads * dim or u.numel() != heads * dim:
+            raise KernelError("mix_tiles: decay logits [T, heads * dim], w0 and u [heads * dim] are needed")
+        state, stride = self._state_floats(binding, heads * dim * dim, "mix_tiles")
+        pack, coef = self._tile_buffers(ctx, T, heads, heads, dim, r.device)
+        out = torch.empty((T, heads * dim), dtype=torch.float32, device=r.device)
+        self._call("ts_mix_tiles", _ptr(r), _ptr(k), r.stride(0), _ptr(z), _ptr(w0), _ptr(u), _ptr(v), v.stride(0), _ptr(ctx.cu_q),
+                   _ptr(binding.state_slots), _ptr(ctx.prefill_seqs), ctx.prefill_seqs.shape[0], ctx.max_q_len, state.data_ptr(),
+                   stride, _ptr(pack), _ptr(coef), _ptr(out), heads, dim, _DTYPE_CODE[r.dtype], _stream())
+        self.launches += 1
         return out
 
     def delta_prepare(self, q: torch.Tensor, k: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
@@ -981,10 +1055,11 @@ class Ops:
         return prepared, beta
 
     def delta_prepare_head(self, q: torch.Tensor, k: torch.Tensor, gates: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
-                           *, heads: int, kv_heads: int, dim: int, unit_eps: float, q_scale: float):
+                           *, heads: int, kv_heads: int, dim: int, unit_eps: float, q_scale: float, singles=None):
         """
         `delta_prepare` with one decay a head: (prepared [2, T, kv_heads * dim], beta [T, heads], decay [T, heads]),
         float32.  gates float32 [T, 2 heads]: the step sizes' logits, then the decays'; dt_bias, a_log [heads].
+        `singles` (a step context): only the rows of requests that feed one token are prepared.
         """
         T = q.shape[0]
         for t, name in ((q, "q"), (k, "k")):
@@ -997,7 +1072,8 @@ class Ops:
         beta = torch.empty((T, heads), dtype=torch.float32, device=q.device)
         decay = torch.empty_like(beta)
         self._call("ts_delta_prepare_head", _ptr(q), _ptr(k), q.stride(0), _ptr(gates), _ptr(dt_bias), _ptr(a_log), _ptr(prepared),
-                   _ptr(beta), _ptr(decay), T, heads, kv_heads, dim, unit_eps, q_scale, _stream())
+                   _ptr(beta), _ptr(decay), T, heads, kv_heads, dim, unit_eps, q_scale,
+                   0 if singles is None else _ptr(singles.seq_of_token), 0 if singles is None else _ptr(singles.cu_q), _stream())
         return prepared, beta, decay
 
     def token_shift(self, x: torch.Tensor, mu: torch.Tensor, ctx, binding) -> torch.Tensor:
@@ -1018,13 +1094,16 @@ class Ops:
         return mixes
 
     def time_mix_prepare(self, r: torch.Tensor, k: torch.Tensor, z: torch.Tensor, w0: torch.Tensor, u: torch.Tensor,
-                         x: torch.Tensor, ctx, binding, *, heads: int, dim: int):
+                         x: torch.Tensor, ctx, binding, *, heads: int, dim: int, rows: str = "all"):
         """
         (prepared [3, T, heads * dim], bonus [T, heads]), float32, for the scan's bonus form: r and k as they are,
         decays exp(-exp(z + w0)), bonus = sum over a head's channels of u k r.  Each request's last row of x (the
-        mixer's input) goes to its state slot (`binding`: the slots' previous rows).
+        mixer's input) goes to its state slot (`binding`: the slots' previous rows).  `rows` "singles": only the rows of
+        requests that feed one token are prepared; "none": none, the slots move on all the same.
         """
         T = r.shape[0]
+        if rows not in ("all", "singles", "none"):
+            raise KernelError(f"time_mix_prepare: rows {rows!r}")
         for t, name in ((r, "r"), (k, "k")):
             if t.dtype != x.dtype or t.stride(1) != 1 or tuple(t.shape) != (T, heads * dim) or t.stride(0) != r.stride(0):
                 raise KernelError(f"time_mix_prepare: {name} must be a [T, {heads * dim}] stretch of x's dtype, of r's row stride")
@@ -1033,11 +1112,12 @@ class Ops:
         if tuple(z.shape) != (T, heads * dim) or w0.numel() != heads * dim or u.numel() != heads * dim:
             raise KernelError("time_mix_prepare: decay logits [T, heads * dim], w0 and u [heads * dim] are needed")
         state, stride = self._state_floats(binding, x.shape[1], "time_mix_prepare")
-        prepared = torch.empty((3, T, heads * dim), dtype=torch.float32, device=x.device)
+        prepared = torch.empty((3, T if rows != "none" else 0, heads * dim), dtype=torch.float32, device=x.device)
         bonus = torch.empty((T, heads), dtype=torch.float32, device=x.device)
         self._call("ts_time_mix_prepare", _ptr(r), _ptr(k), r.stride(0), _ptr(z), _ptr(w0), _ptr(u), _ptr(prepared), _ptr(bonus),
                    T, heads, dim, _ptr(x), x.shape[1], _ptr(ctx.cu_q), _ptr(binding.state_slots), binding.state_slots.shape[0],
-                   state.data_ptr(), stride, _DTYPE_CODE[x.dtype], _stream())
+                   state.data_ptr(), stride, 1 if rows == "none" else 0, _ptr(ctx.seq_of_token) if rows == "singles" else 0,
+                   _DTYPE_CODE[x.dtype], _stream())
         return prepared, bonus
 
     def mlstm_prepare(self, q: torch.Tensor, k: torch.Tensor, gates: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor,

@@ -125,8 +125,13 @@ class GatedDeltaRule(Mixer):
         q, k, v = conv[:, :G * D], conv[:, G * D:2 * G * D], conv[:, 2 * G * D:]
         sizes = dict(heads=H, kv_heads=G, dim=D, unit_eps=s.unit_eps, q_scale=s.q_scale)
         if self.head_decay:
-            prepared, beta, decay = ops.delta_prepare_head(q, k, b, self.dt_bias, self.a_log, **sizes)
-            o = ops.recurrence_scan(prepared, v, ctx, matrices, heads=H, dim=D, vdim=V, beta=beta, head_decay=decay, qk_group=H // G)
+            o, tiles = None, ops.portions_by_tiles(ctx)
+            if tiles:                                   # prompt portions sixteen tokens at a time
+                o = ops.delta_tiles(q, k, v, b, self.dt_bias, self.a_log, ctx, matrices, vdim=V, **sizes)
+            if not tiles or ctx.min_q_len <= 1:         # single tokens (or every request) by the scan
+                prepared, beta, decay = ops.delta_prepare_head(q, k, b, self.dt_bias, self.a_log, singles=ctx if tiles else None, **sizes)
+                o = ops.recurrence_scan(prepared, v, ctx, matrices, heads=H, dim=D, vdim=V, beta=beta, head_decay=decay,
+                                        qk_group=H // G, singles=tiles, out=o)
         else:
             z = self.decay_up(y[:, C:C + self.decay_rank].contiguous(), out_dtype=torch.float32)  # decay logits, float32 from here on
             prepared, beta = ops.delta_prepare(q, k, z, self.dt_bias, self.a_log, b, **sizes)

@@ -9,7 +9,7 @@ token under a bonus, and whose inputs are blends of the token's row and the one 
 
 One kernel makes the five blends, one grouped product the four projections of equal shape, a small
 one with tanh in its epilogue and a second one (float32 out) the decays' logits; then the scan of
-`linear_recurrence.cu` in its bonus form.  The state (float32: the matrices, then the last h) lives in
+`linear_recurrence.cu` in its bonus form (prompt portions: `recurrence_tiles.cu`).  The state (float32: the matrices, then the last h) lives in
 the request's slot of the cache manager, so prompts in portions, decoding and mixed batches are one
 code path.  Since every projection reads a blend of its own, none of them can join a projection
 of h: inside a `ParallelMixer` this branch exposes no input rows and reads h itself.
@@ -80,8 +80,14 @@ class TimeMixing(Mixer):
         r, k, v, g = ops.linear_groups(mixes[:4], self.rkvg)
         low = ops.linear_unary(mixes[4], self.decay_down.weight, "tanh")
         z = self.decay_up(low, out_dtype=torch.float32)                   # decay logits, float32 from here on
-        prepared, bonus = ops.time_mix_prepare(r, k, z, self.w0, self.u, x, ctx, previous, heads=H, dim=D)
-        o = ops.recurrence_scan(prepared, v, ctx, matrices, heads=H, dim=D, vdim=D, bonus=bonus)
+        o, tiles = None, ops.portions_by_tiles(ctx)
+        if tiles:                                        # prompt portions sixteen tokens at a time
+            o = ops.mix_tiles(r, k, v, z, self.w0, self.u, ctx, matrices, heads=H, dim=D)
+        singles = not tiles or ctx.min_q_len <= 1        # single tokens (or every request) by the scan
+        prepared, bonus = ops.time_mix_prepare(r, k, z, self.w0, self.u, x, ctx, previous, heads=H, dim=D,
+                                               rows="all" if not tiles else "singles" if singles else "none")
+        if singles:
+            o = ops.recurrence_scan(prepared, v, ctx, matrices, heads=H, dim=D, vdim=D, bonus=bonus, singles=tiles, out=o)
         return ops.head_norm_gate(o, g, self.norm_weight, H, D, s.out_norm_eps, x.dtype, gate_kind="silu", weight_per_head=True,
                                   scale=scale, out=out)
 
