@@ -14,25 +14,38 @@
 //   o_t = sum_i r_(t,i) d_(t-1,i) S_0[i] + sum_{j<t} P[t][j] v_j + bonus_t v_t,
 //   P[t][j] = sum_i r_(t,i) k_(j,i) a_(j+1,i) ... a_(t-1,i),   S_B = d_B S_0 + sum_j (k_j a_(j+1) ... a_B) v_j^T
 //
-// No decay is ever divided by another: products of decays are taken as they are needed.  Everything is float32.
-// A first kernel works out, per tile and q/k head (time mixing: head), what all columns of the state share:
-// the "pack", a row per key channel [16 q-side entries | 16 k-side entries | the row's decay over the tile], and
-// the coefficients (W = M diag(b), P, c, G[B]).  The second kernel walks the tiles: a CTA owns one request, one
-// head and 16 columns of the state and does three small products a tile,
-//   S_0^T [q-side | k-side]  (rows of S split over the warps, 4 x 4 outputs a thread, partial sums added up in order)
-//   U and O from the 16 x 16 coefficients,  S_B  (the state's own 4 columns x R rows a thread in registers)
-// with the next tile's pack and coefficients on their way by cp.async.  A tile cut short by the portion's end is
-// filled up with tokens that change nothing (k = 0, decay 1).  Requests that feed one token are left to the
-// other scan.  Tiles count from the portion's first token, so where a prompt was cut moves sums inside
-// rounding only.
+// No decay is ever divided by another: products of decays are taken as they are needed.
+//
+// A first kernel works out, per tile and q/k head (time mixing: head), what all columns of the state share: the
+// "pack" (16 rows for the q side, 16 for the k side, one with the channels' decays over the tile) and the coefficients
+// (W = M diag(b); P W, so that O = diag(c) S_0^T Q + (P W) (V - diag(c) R) does not wait for U; c; G[B]).  The second
+// kernel walks the tiles: a CTA owns one request, one head and 16 columns of the state and does three small
+// products a tile on tensor cores,
+//   [q side | k side] S_0   (each warp its own rows of S, the partial sums meet in shared memory in warp order)
+//   U (two warps) and O (two warps) from the 16 x 16 coefficients
+//   K^T U, by which the state moves on
+// with the next tile's pack and coefficients on their way by cp.async.  The products are float32 to rounding: every
+// factor is split into two TF32 numbers, x = hi + lo, and hi hi + hi lo + lo hi is summed in float32 (what is
+// left out is 2^-22 of a term).  The state stays in registers, in the layout in which the third product
+// leaves it (its transpose) and the first one takes it; the update is added to it by an ordinary fused
+// multiply-add, so that what the tensor cores round is the update and not the state.
+//
+// A tile cut short by the portion's end is filled up with tokens that change nothing (k = 0, decay 1).  Requests that
+// feed one token are left to the other scan.  Tiles count from the portion's first token, so where a prompt was cut
+// moves sums inside rounding only.
 #include "common.cuh"
 
 namespace {
 
 constexpr int B = 16;              // tokens a tile
 constexpr int COLS = 16;           // value channels a CTA
-constexpr int ROW = 36;            // floats a pack row: 16 + 16 entries, the row's decay, 3 unused (rows start 16-byte aligned)
-constexpr int COEF = 2 * B * B + 2 * B;   // W [16][16], P [16][16], c [16], g [16]
+constexpr int WARPS = 4, THREADS = WARPS * 32;   // of the scan
+constexpr int CP = 20;             // pitch of a coefficient matrix: a warp's fragment loads fall into different banks
+constexpr int COEF = 2 * B * CP + 2 * B;   // W [16][20], P W (time mixing: P) [16][20], c [16], g [16]
+constexpr int RP = 24;             // pitch of the partial sums and of U: likewise
+// A pack: 33 rows (16 q-side, 16 k-side, the channels' decays) of `rows` floats and a pad that does the same for it.
+__host__ __device__ constexpr int pack_pitch(int rows) { return rows + 8; }
+__host__ __device__ constexpr int pack_floats(int rows) { return (2 * B + 1) * pack_pitch(rows); }
 enum { DELTA = 0, MIX = 1 };
 
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
@@ -83,10 +96,11 @@ __global__ void __launch_bounds__(128) delta_tile_prepare_kernel(PrepareArgs p) 
     }
     __syncthreads();
     const long long slot = tile_slot(seq, begin, tile);
-    float* pack = p.pack + (slot * p.kv_heads + g) * p.rows * ROW;
-    for (int e = threadIdx.x; e < p.rows * 32; e += 128) {
-        const int i = e >> 5, t = e & 31;
-        pack[i * ROW + t] = t < B ? qs[t * pitch + i] : ks[(t - B) * pitch + i];
+    float* pack = p.pack + (slot * p.kv_heads + g) * pack_floats(p.rows);
+    for (int e = threadIdx.x; e < B * p.rows; e += 128) {
+        const int t = e / p.rows, i = e % p.rows;
+        pack[t * pack_pitch(p.rows) + i] = qs[t * pitch + i];
+        pack[(B + t) * pack_pitch(p.rows) + i] = ks[t * pitch + i];
     }
     {   // the dot products: thread (t, pair of j)
         const int t = threadIdx.x >> 3, j = (threadIdx.x & 7) * 2;
@@ -111,7 +125,7 @@ __global__ void __launch_bounds__(128) delta_tile_prepare_kernel(PrepareArgs p) 
             a = expf(-expf(p.rate[h]) * softplus(gr[p.heads + h] + p.bias[h]));
         }
         float* out = p.coef + (slot * p.heads + h) * COEF;
-        float M[B];
+        float M[B], P[B];
         float decay = 1.f, c = 1.f, c_own = 1.f;         // G[t][j] as t runs; c_t; c_j
 #pragma unroll
         for (int t = 0; t < B; ++t) {
@@ -120,19 +134,25 @@ __global__ void __launch_bounds__(128) delta_tile_prepare_kernel(PrepareArgs p) 
             if (t == j) c_own = c;
             if (t > j) decay *= at;
             const float A = t > j ? bt * decay * kk[t * (B + 1) + j] : 0.f;
-            const float P = t >= j ? decay * qk[t * (B + 1) + j] : 0.f;
+            P[t] = t >= j ? decay * qk[t * (B + 1) + j] : 0.f;
             float row = t == j ? 1.f : 0.f;              // M[t][j] = delta - sum_s A[t][s] M[s][j]
 #pragma unroll
             for (int s = 0; s < t; ++s) row = fmaf(-__shfl_sync(0xffffffffu, A, s), M[s], row);
             M[t] = row;
+        }
+#pragma unroll
+        for (int t = 0; t < B; ++t) {
+            float pw = 0.f;
+#pragma unroll
+            for (int s = 0; s <= t; ++s) pw = fmaf(__shfl_sync(0xffffffffu, P[t], s), M[s] * b, pw);
             if (lane < B) {
-                out[t * B + j] = row * b;
-                out[B * B + t * B + j] = P;
+                out[t * CP + j] = M[t] * b;
+                out[B * CP + t * CP + j] = pw;
             }
         }
         if (lane < B) {
-            out[2 * B * B + j] = c_own;
-            out[2 * B * B + B + j] = decay;
+            out[2 * B * CP + j] = c_own;
+            out[2 * B * CP + B + j] = decay;
         }
     }
 }
@@ -151,7 +171,7 @@ __global__ void __launch_bounds__(128) mix_tile_prepare_kernel(PrepareArgs p) {
     float* ks = rs + B * pitch;
     float* as = ks + B * pitch;
     const long long slot = tile_slot(seq, begin, tile);
-    float* pack = p.pack + (slot * p.heads + h) * p.rows * ROW;
+    float* pack = p.pack + (slot * p.heads + h) * pack_floats(p.rows);
     const long long width = (long long)p.heads * p.dim, hc = (long long)h * p.dim;
     for (int e = threadIdx.x; e < B * p.rows; e += 128) {
         const int t = e / p.rows, i = e % p.rows;
@@ -184,32 +204,28 @@ __global__ void __launch_bounds__(128) mix_tile_prepare_kernel(PrepareArgs p) {
                 }
             }
         }
-        float* out = p.coef + (slot * p.heads + h) * COEF + B * B;
+        float* out = p.coef + (slot * p.heads + h) * COEF + B * CP;
 #pragma unroll
         for (int t = 0; t < B; ++t) {
             float s = sum[t];
 #pragma unroll
             for (int o = 4; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-            if (part == 0) out[t * B + j] = s;                                          // 0 where t < j
+            if (part == 0) out[t * CP + j] = s;                                         // 0 where t < j
         }
     }
     __syncthreads();
     for (int i = threadIdx.x; i < p.rows; i += 128) {    // a thread a channel: products from the left and from the right
+        const int pp = pack_pitch(p.rows);
         float left = 1.f, right = 1.f;
         for (int t = 0; t < B; ++t) {
-            rs[t * pitch + i] *= left;
+            pack[t * pp + i] = rs[t * pitch + i] * left;
             left *= as[t * pitch + i];
         }
         for (int t = B - 1; t >= 0; --t) {
-            ks[t * pitch + i] *= right;
+            pack[(B + t) * pp + i] = ks[t * pitch + i] * right;
             right *= as[t * pitch + i];
         }
-        pack[i * ROW + 2 * B] = left;
-    }
-    __syncthreads();
-    for (int e = threadIdx.x; e < p.rows * 32; e += 128) {
-        const int i = e >> 5, t = e & 31;
-        pack[i * ROW + t] = t < B ? rs[t * pitch + i] : ks[(t - B) * pitch + i];
+        pack[2 * B * pp + i] = left;
     }
 }
 
@@ -226,195 +242,221 @@ __device__ __forceinline__ void cp16(void* smem, const void* gmem) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
 }
 
-// R: rows of the state a thread holds (32 R rows in all)
-template <typename T, int R, int MODE>
-__global__ void __launch_bounds__(128) recurrence_tiles_kernel(ScanArgs p) {
-    constexpr int ROWS = 32 * R, WROWS = 8 * R;          // rows of the state; rows of a warp
-    constexpr int STAGE = ROWS * ROW + COEF;             // floats a stage
-    constexpr int RP = COLS + 4;                         // pitch of the partial sums
-    constexpr int TQ = MODE == DELTA ? 32 : 16;          // entries of a pack row that meet S_0
+// A float32 number as the sum of two TF32 numbers (11 significant bits each): hi is x to the nearest (half of its last
+// place added before the low 13 bits go), lo what is left, of which the tensor cores read the leading bits: 2^-23 of x is lost.
+struct Split { uint32_t hi, lo; };
+__device__ __forceinline__ Split split_tf32(float x) {
+    Split s;
+    s.hi = (__float_as_uint(x) + 0x1000u) & 0xffffe000u;
+    s.lo = __float_as_uint(x - __uint_as_float(s.hi));
+    return s;
+}
+__device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+struct SplitA { uint32_t hi[4], lo[4]; };
+__device__ __forceinline__ SplitA split_a(float a0, float a1, float a2, float a3) {
+    const Split s0 = split_tf32(a0), s1 = split_tf32(a1), s2 = split_tf32(a2), s3 = split_tf32(a3);
+    return SplitA{{s0.hi, s1.hi, s2.hi, s3.hi}, {s0.lo, s1.lo, s2.lo, s3.lo}};
+}
+// The two large and the small parts of a product of split factors, each in an accumulator of its own (no long chain).
+__device__ __forceinline__ void mma_split(float (&big)[4], float (&small)[4], const SplitA& a, Split b0, Split b1) {
+    mma_tf32(big, a.hi, b0.hi, b1.hi);
+    mma_tf32(small, a.hi, b0.lo, b1.lo);
+    mma_tf32(small, a.lo, b0.hi, b1.hi);
+}
+
+// NT: eights of rows of the state a warp holds.  Fragments of mma.m16n8k8, lane = 4 r + c (r 0..7, c 0..3):
+//   A (16 x 8): (r, c), (r + 8, c), (r, c + 4), (r + 8, c + 4);   B (8 x 8): (c, r), (c + 4, r);
+//   C (16 x 8): (r, 2c), (r, 2c + 1), (r + 8, 2c), (r + 8, 2c + 1).
+// The state is held as C fragments of S^T (16 columns x 8 rows of S).  Read as B fragments of S they hold rows 2c and
+// 2c + 1 where the product counts k = c and c + 4: the A side takes its k in the same order.
+template <typename T, int NT, int MODE>
+__global__ void __launch_bounds__(THREADS) recurrence_tiles_kernel(ScanArgs p) {
+    constexpr int WROWS = 8 * NT, ROWS = WARPS * WROWS;  // rows of a warp; rows of the state
+    constexpr int PP = pack_pitch(ROWS);
+    constexpr int PACK = pack_floats(ROWS), STAGE = PACK + COEF;
+    constexpr int TQ = MODE == DELTA ? 2 * B : B;        // rows of the pack that meet S_0
     extern __shared__ __align__(16) float smem[];
-    float* S_s = smem + 2 * STAGE;                       // [ROWS][COLS]
-    float* red = S_s + ROWS * COLS;                      // [4][TQ][RP]
-    float* X_s = red + 4 * TQ * RP;                      // [B][COLS]: V - c R; mixing: V
-    float* U_s = X_s + B * COLS;                         // [B][COLS]: U (delta)
-    float* G_s = U_s + B * COLS;                         // [B][COLS]: G[B] U (delta)
+    float* red = smem + 2 * STAGE;                       // [WARPS][TQ][RP]
+    float* G_s = red + WARPS * TQ * RP;                  // [B][RP]: what the state's update takes, G[B] U or V
     const int seq = p.prefill_seqs[blockIdx.z], h = blockIdx.y, j0 = blockIdx.x * COLS;
     if (seq < 0) return;
     const int begin = p.cu_q[seq], n = p.cu_q[seq + 1] - begin, slot = p.slots[seq];
     if (n <= 1 || slot < 0) return;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int tg = lane >> 2, cg = lane & 3;             // product 1: entries of group tg, columns 4 cg ..; product 3: rows tg + 8 e
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane >> 2, c = lane & 3;
     const int qk_heads = p.heads / p.qk_group, qh = h / p.qk_group;
     float* st = p.state + (long long)slot * p.slot_stride + (long long)h * p.dim * p.vdim;
 
-    float S[R][4];
+    auto element = [&](int nt, int e, int& i, int& j) {  // row and column of S of register e of tile nt
+        i = warp * WROWS + 8 * nt + 2 * c + (e & 1);
+        j = j0 + r + 8 * (e >> 1);
+        return i < p.dim && j < p.vdim;
+    };
+    float S[NT][4];
 #pragma unroll
-    for (int e = 0; e < R; ++e) {
-        const int i = warp * WROWS + tg + 8 * e;
+    for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-            const int j = j0 + 4 * cg + c;
-            S[e][c] = i < p.dim && j < p.vdim ? st[(long long)i * p.vdim + j] : 0.f;
+        for (int e = 0; e < 4; ++e) {
+            int i, j;
+            S[nt][e] = element(nt, e, i, j) ? st[(long long)i * p.vdim + j] : 0.f;
         }
-        *reinterpret_cast<float4*>(S_s + i * COLS + 4 * cg) = make_float4(S[e][0], S[e][1], S[e][2], S[e][3]);
-    }
     const int tiles = (n + B - 1) / B;
     const long long first = tile_slot(seq, begin, 0);
     auto issue = [&](int tile) {
         float* stage = smem + (tile & 1) * STAGE;
-        const float* pack = p.pack + ((first + tile) * qk_heads + qh) * (long long)(ROWS * ROW);
+        const float* pack = p.pack + ((first + tile) * qk_heads + qh) * (long long)PACK;
         const float* coef = p.coef + ((first + tile) * p.heads + h) * (long long)COEF;
-        for (int e = tid; e < ROWS * ROW / 4; e += 128) cp16(stage + 4 * e, pack + 4 * e);
-        for (int e = tid; e < COEF / 4; e += 128) cp16(stage + ROWS * ROW + 4 * e, coef + 4 * e);
+#pragma unroll
+        for (int e = 0; e < PACK / 4; e += THREADS)
+            if (e + tid < PACK / 4) cp16(stage + 4 * (e + tid), pack + 4 * (e + tid));
+#pragma unroll
+        for (int e = 0; e < COEF / 4; e += THREADS)
+            if (e + tid < COEF / 4) cp16(stage + PACK + 4 * (e + tid), coef + 4 * (e + tid));
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
-    // thread (t, two columns) for the values, U and O
-    const int vt = tid >> 3, vj = (tid & 7) * 2;
-    const T* v = (const T*)p.v;
-    auto fetch_v = [&](int tile, float (&x)[2]) {
-        const int t = tile * B + vt;
+    // Warps 0 and 1 make U (time mixing: hand the values on), warps 2 and 3 O, for columns 8 (warp & 1) .. + 7 each.
+    // Their values, as B fragments: tokens c, c + 4, c + 8, c + 12 of column r.
+    const int nt_uo = warp & 1, col = 8 * nt_uo + r;
+    const bool makes_o = warp >= 2;
+    static_assert(WARPS == 4, "two warps make U, two make O");
+    const T* v = (const T*)p.v + (long long)(begin + c) * p.v_stride + (long long)h * p.vdim + j0 + col;
+    T vnow[4], vnext[4];
+    auto fetch_v = [&](int tile, T (&x)[4]) {            // as loaded: converting would wait for the load
 #pragma unroll
-        for (int c = 0; c < 2; ++c)
-            x[c] = t < n && j0 + vj + c < p.vdim ? to_float<T>(v[(long long)(begin + t) * p.v_stride + (long long)h * p.vdim + j0 + vj + c]) : 0.f;
+        for (int k = 0; k < 4; ++k)
+            x[k] = tile * B + c + 4 * k < n && j0 + col < p.vdim ? v[(long long)(tile * B + 4 * k) * p.v_stride] : from_float<T>(0.f);
     };
     issue(0);
-    float vnow[2], vnext[2] = {0.f, 0.f};
     fetch_v(0, vnow);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) vnext[k] = vnow[k];
     for (int tile = 0; tile < tiles; ++tile) {
         asm volatile("cp.async.wait_all;\n" ::: "memory");
-        __syncthreads();                                 // the tile's inputs and the state are in; the other stage has been read
+        __syncthreads();                                 // the tile's inputs are in; the other stage, U and the sums have been read
         if (tile + 1 < tiles) {
             issue(tile + 1);
             fetch_v(tile + 1, vnext);
         }
         const float* pack = smem + (tile & 1) * STAGE;
-        const float* coef = pack + ROWS * ROW;
-        // product 1: this warp's rows of S against the pack's entries
+        const float* coef = pack + PACK;
+        // product 1: the pack's rows against this warp's rows of S
         {
-            constexpr int TT = TQ / 8;                   // entries a thread: 4 (delta) or 2
-            float acc[TT][4];
+            float big[TQ / B][2][4] = {}, small[TQ / B][2][4] = {};
 #pragma unroll
-            for (int x = 0; x < TT; ++x)
+            for (int nt = 0; nt < NT; ++nt) {
+                Split b[4];
 #pragma unroll
-                for (int c = 0; c < 4; ++c) acc[x][c] = 0.f;
-            const float* pk = pack + warp * WROWS * ROW + TT * tg;
-            const float* sr = S_s + warp * WROWS * COLS + 4 * cg;
+                for (int e = 0; e < 4; ++e) b[e] = split_tf32(S[nt][e]);
 #pragma unroll
-            for (int i = 0; i < WROWS; ++i) {
-                __align__(16) float kq[TT];
-                if constexpr (TT == 4) *reinterpret_cast<float4*>(kq) = *reinterpret_cast<const float4*>(pk + i * ROW);
-                else *reinterpret_cast<float2*>(kq) = *reinterpret_cast<const float2*>(pk + i * ROW);
-                const float4 s = *reinterpret_cast<const float4*>(sr + i * COLS);
-#pragma unroll
-                for (int x = 0; x < TT; ++x) {
-                    acc[x][0] = fmaf(kq[x], s.x, acc[x][0]);
-                    acc[x][1] = fmaf(kq[x], s.y, acc[x][1]);
-                    acc[x][2] = fmaf(kq[x], s.z, acc[x][2]);
-                    acc[x][3] = fmaf(kq[x], s.w, acc[x][3]);
+                for (int mt = 0; mt < TQ / B; ++mt) {
+                    const float* row = pack + (mt * B + r) * PP + warp * WROWS + 8 * nt + 2 * c;
+                    const float2 lo = *reinterpret_cast<const float2*>(row), hi = *reinterpret_cast<const float2*>(row + 8 * PP);
+                    const SplitA a = split_a(lo.x, hi.x, lo.y, hi.y);
+                    mma_split(big[mt][0], small[mt][0], a, b[0], b[1]);
+                    mma_split(big[mt][1], small[mt][1], a, b[2], b[3]);
                 }
             }
 #pragma unroll
-            for (int x = 0; x < TT; ++x)
-                *reinterpret_cast<float4*>(red + (warp * TQ + TT * tg + x) * RP + 4 * cg) = make_float4(acc[x][0], acc[x][1], acc[x][2], acc[x][3]);
+            for (int mt = 0; mt < TQ / B; ++mt)
+#pragma unroll
+                for (int nj = 0; nj < 2; ++nj)
+#pragma unroll
+                    for (int half = 0; half < 2; ++half)
+                        *reinterpret_cast<float2*>(red + (warp * TQ + mt * B + r + 8 * half) * RP + 8 * nj + 2 * c) =
+                            make_float2(big[mt][nj][2 * half] + small[mt][nj][2 * half],
+                                        big[mt][nj][2 * half + 1] + small[mt][nj][2 * half + 1]);
         }
-        if (MODE == MIX) *reinterpret_cast<float2*>(X_s + vt * COLS + vj) = make_float2(vnow[0], vnow[1]);
-        __syncthreads();                                 // partial sums (and, mixing, the values) are in
-        float o[2] = {0.f, 0.f}, rd[2] = {0.f, 0.f};
+        __syncthreads();                                 // the partial sums are in
+        {
+            float x[4];                                  // V - c R (time mixing: V) at tokens c + 4 k of column `col`
 #pragma unroll
-        for (int w = 0; w < 4; ++w) {
-            const float2 x = *reinterpret_cast<const float2*>(red + (w * TQ + vt) * RP + vj);
-            o[0] += x.x; o[1] += x.y;
-            if (MODE == DELTA) {
-                const float2 y = *reinterpret_cast<const float2*>(red + (w * TQ + B + vt) * RP + vj);
-                rd[0] += y.x; rd[1] += y.y;
-            }
-        }
-        const float* in_s = X_s;                         // what O and the state's update take: U, or the values
-        const float* up_s = X_s;
-        if constexpr (MODE == DELTA) {
-            const float c = coef[2 * B * B + vt];
-            o[0] *= c; o[1] *= c;
-            *reinterpret_cast<float2*>(X_s + vt * COLS + vj) = make_float2(fmaf(-c, rd[0], vnow[0]), fmaf(-c, rd[1], vnow[1]));
-            __syncthreads();
-            float u[2] = {0.f, 0.f};
+            for (int k = 0; k < 4; ++k) {
+                x[k] = to_float<T>(vnow[k]);
+                if (MODE == DELTA) {
+                    float sum = 0.f;
 #pragma unroll
-            for (int s4 = 0; s4 < B; s4 += 4) {
-                const float4 w = *reinterpret_cast<const float4*>(coef + vt * B + s4);
-                const float ww[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-                for (int s = 0; s < 4; ++s) {
-                    const float2 x = *reinterpret_cast<const float2*>(X_s + (s4 + s) * COLS + vj);
-                    u[0] = fmaf(ww[s], x.x, u[0]);
-                    u[1] = fmaf(ww[s], x.y, u[1]);
+                    for (int w = 0; w < WARPS; ++w) sum += red[(w * TQ + B + c + 4 * k) * RP + col];
+                    x[k] = fmaf(-coef[2 * B * CP + c + 4 * k], sum, x[k]);
                 }
             }
-            const float gt = coef[2 * B * B + B + vt];
-            *reinterpret_cast<float2*>(U_s + vt * COLS + vj) = make_float2(u[0], u[1]);
-            *reinterpret_cast<float2*>(G_s + vt * COLS + vj) = make_float2(gt * u[0], gt * u[1]);
-            __syncthreads();
-            in_s = U_s;
-            up_s = G_s;
-        }
-        // O
+            if (MODE == MIX && !makes_o) {
 #pragma unroll
-        for (int s4 = 0; s4 < B; s4 += 4) {
-            const float4 w = *reinterpret_cast<const float4*>(coef + B * B + vt * B + s4);
-            const float ww[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-            for (int s = 0; s < 4; ++s) {
-                const float2 x = *reinterpret_cast<const float2*>(in_s + (s4 + s) * COLS + vj);
-                o[0] = fmaf(ww[s], x.x, o[0]);
-                o[1] = fmaf(ww[s], x.y, o[1]);
+                for (int k = 0; k < 4; ++k) G_s[(c + 4 * k) * RP + col] = x[k];
             }
-        }
-        if (tile * B + vt < n) {
-            float* dst = p.out + ((long long)(begin + tile * B + vt) * p.heads + h) * p.vdim + j0 + vj;
-            if (j0 + vj < p.vdim) dst[0] = o[0];
-            if (j0 + vj + 1 < p.vdim) dst[1] = o[1];
-        }
-        // the state after the tile
-        const float cB = coef[2 * B * B + B - 1];
+            if (MODE == DELTA || makes_o) {
+                const float* m = coef + (makes_o ? B * CP : 0);
+                float big[4] = {}, small[4] = {};
 #pragma unroll
-        for (int e = 0; e < R; ++e) {
-            const float d = MODE == DELTA ? cB : pack[(warp * WROWS + tg + 8 * e) * ROW + 2 * B];
+                for (int ks = 0; ks < 2; ++ks) {
+                    const float* a = m + r * CP + 8 * ks + c;
+                    mma_split(big, small, split_a(a[0], a[8 * CP], a[4], a[8 * CP + 4]), split_tf32(x[2 * ks]), split_tf32(x[2 * ks + 1]));
+                }
 #pragma unroll
-            for (int c = 0; c < 4; ++c) S[e][c] *= d;
-        }
+                for (int half = 0; half < 2; ++half) {
+                    const int t = r + 8 * half;
+                    float y0 = big[2 * half] + small[2 * half], y1 = big[2 * half + 1] + small[2 * half + 1];
+                    if (!makes_o) {
+                        const float g = coef[2 * B * CP + B + t];
+                        *reinterpret_cast<float2*>(G_s + t * RP + 8 * nt_uo + 2 * c) = make_float2(g * y0, g * y1);
+                    } else {
+                        float q0 = 0.f, q1 = 0.f;
 #pragma unroll
-        for (int t4 = 0; t4 < B; t4 += 4) {
-            float4 u4[4];
-#pragma unroll
-            for (int t = 0; t < 4; ++t) u4[t] = *reinterpret_cast<const float4*>(up_s + (t4 + t) * COLS + 4 * cg);
-#pragma unroll
-            for (int e = 0; e < R; ++e) {
-                const float4 k4 = *reinterpret_cast<const float4*>(pack + (warp * WROWS + tg + 8 * e) * ROW + B + t4);
-                const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
-#pragma unroll
-                for (int t = 0; t < 4; ++t) {
-                    S[e][0] = fmaf(kk[t], u4[t].x, S[e][0]);
-                    S[e][1] = fmaf(kk[t], u4[t].y, S[e][1]);
-                    S[e][2] = fmaf(kk[t], u4[t].z, S[e][2]);
-                    S[e][3] = fmaf(kk[t], u4[t].w, S[e][3]);
+                        for (int w = 0; w < WARPS; ++w) {
+                            const float2 q = *reinterpret_cast<const float2*>(red + (w * TQ + t) * RP + 8 * nt_uo + 2 * c);
+                            q0 += q.x;
+                            q1 += q.y;
+                        }
+                        const float ct = MODE == DELTA ? coef[2 * B * CP + t] : 1.f;
+                        y0 = fmaf(ct, q0, y0);
+                        y1 = fmaf(ct, q1, y1);
+                        const int j = j0 + 8 * nt_uo + 2 * c;
+                        if (tile * B + t < n) {
+                            float* dst = p.out + ((long long)(begin + tile * B + t) * p.heads + h) * p.vdim + j;
+                            if (j < p.vdim) dst[0] = y0;
+                            if (j + 1 < p.vdim) dst[1] = y1;
+                        }
+                    }
                 }
             }
         }
-        // a warp's rows of S_s are read by that warp alone, and it has read them: no barrier before they change
+        __syncthreads();                                 // what the update takes is in
+        // product 3, S^T <- decay S^T + G^T K, and the state after the tile
+        {
+            SplitA a[2];
 #pragma unroll
-        for (int e = 0; e < R; ++e)
-            *reinterpret_cast<float4*>(S_s + (warp * WROWS + tg + 8 * e) * COLS + 4 * cg) = make_float4(S[e][0], S[e][1], S[e][2], S[e][3]);
-        vnow[0] = vnext[0];
-        vnow[1] = vnext[1];
+            for (int ks = 0; ks < 2; ++ks) {
+                const float* g = G_s + (8 * ks + c) * RP + r;
+                a[ks] = split_a(g[0], g[8], g[4 * RP], g[4 * RP + 8]);
+            }
+            const float cB = MODE == DELTA ? coef[2 * B * CP + B - 1] : 1.f;
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt) {
+                float big[4] = {}, small[4] = {};
+                const float* k = pack + (B + c) * PP + warp * WROWS + 8 * nt + r;
+#pragma unroll
+                for (int ks = 0; ks < 2; ++ks)
+                    mma_split(big, small, a[ks], split_tf32(k[8 * ks * PP]), split_tf32(k[(8 * ks + 4) * PP]));
+                float2 d = make_float2(cB, cB);
+                if (MODE == MIX) d = *reinterpret_cast<const float2*>(pack + 2 * B * PP + warp * WROWS + 8 * nt + 2 * c);
+                S[nt][0] = fmaf(d.x, S[nt][0], big[0] + small[0]);
+                S[nt][1] = fmaf(d.y, S[nt][1], big[1] + small[1]);
+                S[nt][2] = fmaf(d.x, S[nt][2], big[2] + small[2]);
+                S[nt][3] = fmaf(d.y, S[nt][3], big[3] + small[3]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) vnow[k] = vnext[k];
     }
 #pragma unroll
-    for (int e = 0; e < R; ++e) {
-        const int i = warp * WROWS + tg + 8 * e;
+    for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-            const int j = j0 + 4 * cg + c;
-            if (i < p.dim && j < p.vdim) st[(long long)i * p.vdim + j] = S[e][c];
+        for (int e = 0; e < 4; ++e) {
+            int i, j;
+            if (element(nt, e, i, j)) st[(long long)i * p.vdim + j] = S[nt][e];
         }
-    }
 }
 
 int padded_rows(int dim) { return dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
@@ -422,13 +464,13 @@ int padded_rows(int dim) { return dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
 template <typename T, int MODE>
 int launch_scan(const ScanArgs& p, int portions, cudaStream_t stream) {
     const dim3 grid((p.vdim + COLS - 1) / COLS, p.heads, portions);
-#define TS_TILES(R)                                                                                                  \
+#define TS_TILES(NT)                                                                                                 \
     do {                                                                                                             \
-        constexpr int TQ = MODE == DELTA ? 32 : 16;                                                                  \
-        const size_t smem = sizeof(float) * (2 * (32 * R * ROW + COEF) + 32 * R * COLS + 4 * TQ * (COLS + 4) + 3 * B * COLS); \
-        auto kernel = recurrence_tiles_kernel<T, R, MODE>;                                                           \
+        constexpr int TQ = MODE == DELTA ? 2 * B : B;                                                                \
+        const size_t smem = sizeof(float) * (2 * (pack_floats(WARPS * 8 * NT) + COEF) + (WARPS * TQ + B) * RP);      \
+        auto kernel = recurrence_tiles_kernel<T, NT, MODE>;                                                          \
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                        \
-        kernel<<<grid, 128, smem, stream>>>(p);                                                                      \
+        kernel<<<grid, THREADS, smem, stream>>>(p);                                                                  \
     } while (0)
     const int rows = padded_rows(p.dim);
     if (rows == 64) TS_TILES(2);
@@ -443,7 +485,7 @@ int launch_scan(const ScanArgs& p, int portions, cudaStream_t stream) {
 
 // Floats of the two buffers the tile kernels need: packs (`heads`: the q/k heads) and coefficients (`heads`: the value heads).
 TS_API long long ts_recurrence_tiles_pack_floats(int num_tokens, int num_seqs, int heads, int dim) {
-    return ((long long)num_tokens / B + num_seqs + 1) * heads * padded_rows(dim) * ROW;
+    return ((long long)num_tokens / B + num_seqs + 1) * heads * pack_floats(padded_rows(dim));
 }
 TS_API long long ts_recurrence_tiles_coef_floats(int num_tokens, int num_seqs, int heads) {
     return ((long long)num_tokens / B + num_seqs + 1) * heads * COEF;
