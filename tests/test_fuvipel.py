@@ -417,6 +417,50 @@ def test_time_mixing_reads_the_first_token_far_later():
     torch.testing.assert_close(got, want, **TOL[torch.float32])
 
 
+# ---------------------------------------------------------------------------------------------- tiles of tokens
+@pytest.mark.parametrize("kind", ["delta", "mixing"])
+@pytest.mark.parametrize("tiles", [True, False])
+def test_portions_by_tiles_and_token_by_token_agree_with_the_plain_recurrence(monkeypatch, kind, tiles):
+    """
+    Three requests in one launch: a long portion (several tiles, the last one cut short), one of exactly a tile, and a
+    single token beside them, then portions of two tokens and up that start inside what would be a tile; decays near one, so
+    that sums over hundreds of tokens show, and a head whose decays are zero in float32.
+    """
+    from tinyserve_llm_b200.ops import get_ops
+    monkeypatch.setattr(get_ops(), "recurrence_tiles", tiles)
+    width, H, D = 48, 3, 72
+    if kind == "delta":
+        spec, m = _delta_spec(width, H, 1, D, 40, 3), {"heads": H, "kv_heads": 1, "dim": D, "vdim": 40, "conv": 3}
+        want_of = lambda x, w: plain.gated_delta_rule(x, w, m, 1e-5)  # noqa: E731
+
+        def edit(t):
+            t["A_log"] = torch.tensor([-8.0, -2.0, 6.0]).to(t["A_log"].dtype)
+            t["q"] = t["k"] + t["q"] / 4
+            t["q.conv"] = t["k.conv"]
+    else:
+        spec, m = _mixing_spec(width, H, D, 4), {"heads": H, "dim": D}
+        want_of = lambda x, w: plain.time_mixing(x, w, m, 1e-5)  # noqa: E731
+
+        def edit(t):
+            t["w0"] = torch.tensor([-8.0, -2.0, 6.0]).repeat_interleave(D).to(t["w0"].dtype)
+            t["r"] = t["k"] + t["r"] / 4
+            t["u"] = t["u"] + 1
+
+    mixer, w = _mixer(spec, torch.float32, 31, edit)
+    g = torch.Generator().manual_seed(8)
+    lens = [420, 60, 45]
+    x_of = [torch.randn(n, width, generator=g) for n in lens]
+    cuts = [[(0, 333), (0, 16), (0, 1)], [(333, 335), (16, 17), (1, 18)], [(335, 418), (17, 49), (18, 45)], [(418, 420), (49, 60), (45, 45)]]
+    before = dict(get_ops().calls)
+    got = _in_steps(_Slots(mixer, torch.float32, lens), x_of, cuts)
+    name = "ts_delta_tiles" if kind == "delta" else "ts_mix_tiles"
+    assert (get_ops().calls.get(name, 0) > before.get(name, 0)) == tiles
+    for a, x in zip(got, x_of):
+        want = want_of(x.double(), w)
+        err = (a - want).norm(dim=-1) / want.norm(dim=-1)
+        assert float(err.max()) < 2e-4 and float(err.median()) < 5e-6, f"worst {float(err.max()):.2e}, median {float(err.median()):.2e}"
+
+
 # ---------------------------------------------------------------------------------------------- both halves, norms, products
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("layer", [0, 3])
