@@ -159,6 +159,30 @@ def test_long_decoding_keeps_its_state(folders):
     close(got, plain_logits(folders[name], ids), dtype)
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_layer_sizes_of_a_real_model(tmp_path, dtype):
+    """
+    Heads of 128 channels, a width of 1,024: a prompt of 600 tokens in one step, a portion over it, single tokens from
+    graphs.
+    """
+    from tinyserve_llm_b200.weights import write_random_model
+    from tinyserve_llm_b200.weights.safetensors_io import write_safetensors
+    raw = C.model(1000, 1024, 1e-6, [
+        (C.delta(8, 2, 128, 128, 4), None),
+        (C.parallel(C.attention(8, 2, 128, 0.08, 128, base=500000.0), C.mixing(8, 128, 64)), C.dense(2048)),
+    ])
+    folder = str(tmp_path / "model")
+    write_random_model(folder, raw, 77, std=0.03, unit_std=0.2)
+    tensors = read_tensors(folder)
+    C.steady_reads(tensors)
+    write_safetensors(os.path.join(folder, "model.safetensors"), tensors)
+    ids = ids_of(raw["vocab"], 660, 5)
+    eng = Engine(folder, dtype, page=64, pages=12, cuda_graphs=True)
+    got = eng.run("a", ids, [600, 50, 1, 1, 1, 1, 1, 5])
+    assert eng.runner.graph_replays > 0
+    close(got, plain_logits(folder, ids), dtype)
+
+
 # ---------------------------------------------------------------------------------------------- attention alone
 def _attention_spec(width, heads, kv_heads, dim, scale, rot, base=300.0, gate=True):
     from tinyserve_llm_b200.config.spec import GatedAttentionSpec, InlineRotarySpec
