@@ -77,12 +77,12 @@ def test_what_cannot_be_served_is_refused_with_the_key(edit, message):
 
 
 def test_other_mixers_refuse_a_rotation_of_neighbouring_channels():
-    from tinyserve_llm_b200.config.spec import InlineRotarySpec, LatentAttentionSpec
+    from tinyserve_llm_b200.config.spec import InlineRotarySpec, LinearRecurrenceSpec
     from tinyserve_llm_b200.parts.base import Runtime, part_class
-    spec = LatentAttentionSpec(hidden_size=8, num_heads=1, head_dim=4, rot_dim=4, value_dim=4, kv_rank=4, scale=1.0,
-                               position=InlineRotarySpec(dims=4, interleaved=True))
+    spec = LinearRecurrenceSpec(hidden_size=8, num_heads=1, key_dim=4, value_dim=4, head_decays=(0.5,),
+                                position=InlineRotarySpec(dims=4, interleaved=True))
     cls = part_class("mixer", spec)
-    tensors = {n: torch.zeros([max(s, 1) for s in d.shape]) for n, d in cls.declare(spec).items()}
+    tensors = {n: torch.zeros(d.shape) for n, d in cls.declare(spec).items()}
     with pytest.raises(NotImplementedError, match="neighbouring"):
         cls(spec, tensors, Runtime(dtype=torch.float32, device=torch.device("cpu"), ops=None))
 

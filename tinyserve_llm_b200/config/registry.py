@@ -16,6 +16,7 @@ from typing import Any, Callable, Mapping
 from tinyserve_llm_b200.config.duduvik import DuduvikConfig, duduvik_model_spec
 from tinyserve_llm_b200.config.folavik import FolavikConfig, folavik_model_spec
 from tinyserve_llm_b200.config.fuvipel import FuvipelConfig, fuvipel_model_spec
+from tinyserve_llm_b200.config.gimotar import GimotarConfig, gimotar_model_spec
 from tinyserve_llm_b200.config.llama import ConfigError, LlamaConfig, llama_model_spec
 from tinyserve_llm_b200.config.lugipel import LugipelConfig, lugipel_model_spec
 from tinyserve_llm_b200.config.nipizen import NipizenConfig, nipizen_model_spec
@@ -44,6 +45,7 @@ register_architecture(Architecture("Nipizen", "nipizen", NipizenConfig.from_dict
 register_architecture(Architecture("Lugipel", "lugipel", LugipelConfig.from_dict, lugipel_model_spec))
 register_architecture(Architecture("Folavik", "folavik", FolavikConfig.from_dict, folavik_model_spec))
 register_architecture(Architecture("Fuvipel", "fuvipel", FuvipelConfig.from_dict, fuvipel_model_spec))
+register_architecture(Architecture("Gimotar", "gimotar", GimotarConfig.from_dict, gimotar_model_spec))
 
 
 def resolve_architecture(raw: Mapping[str, Any]) -> Architecture:

@@ -130,7 +130,8 @@ class LatentAttentionSpec(PartSpec):
     Softmax attention whose per-head keys and values are up-projections of one cached latent per
     token; queries go through a normed latent of their own (`q_rank` 0: they are a projection of the input,
     tensor `q`); one rotated key part is shared by the heads (`rot_dim` 0: none, and no `position`);
-    `output_gate`: the concatenated heads are multiplied by sigmoid(W_g h) before the output projection.
+    `output_gate`: the concatenated heads are multiplied by sigmoid(W_g h) before the output projection;
+    `sink`: the number `sink`[h] takes part in every softmax of head h as a score without a key or a value.
     """
 
     kind: str = field(init=False, default="latent_attention")
@@ -146,6 +147,7 @@ class LatentAttentionSpec(PartSpec):
     norm_eps: float = 1e-6
     position: PartSpec | None = None
     output_gate: bool = False
+    sink: bool = False
 
 
 @dataclass(frozen=True)
@@ -173,6 +175,40 @@ class SinusoidSpec(PartSpec):
     kind: str = field(init=False, default="sinusoid")
     size: int = 0
     base: float = 10000.0
+
+
+@dataclass(frozen=True)
+class PairEmbeddingSpec(PartSpec):
+    """
+    A second embedding by the pair (previous token, token), added to the token embedding as it starts the
+    residual stream: row (previous * mul_prev + token * mul_cur) mod buckets of a table of buckets + 1 rows of
+    `size` entries; a request's first token takes the last row.  `name` is the table's tensor.
+    """
+
+    kind: str = field(init=False, default="pair_embedding")
+    size: int = 0
+    buckets: int = 0
+    mul_prev: int = 0
+    mul_cur: int = 0
+    name: str = "bigram"
+
+
+@dataclass(frozen=True)
+class GatedLRUSpec(PartSpec):
+    """
+    Griffin's recurrent block around a real-gated linear recurrent unit, `width` channels:
+    y = gelu_tanh(W_y h + b_y), u = conv(W_x h + b_x) (causal, one filter of `conv_taps` taps and a bias a channel);
+    with u in `blocks` equal parts, r = sigmoid(R_b u_b + c_b) and i = sigmoid(I_b u_b + d_b) part by part;
+    log a = -decay_rate * r * softplus(lam), S_t = a S_(t-1) + sqrt(1 - a^2) i u, output W_o (S * y).
+    State and convolution inputs start at zero.
+    """
+
+    kind: str = field(init=False, default="gated_lru")
+    hidden_size: int = 0
+    width: int = 0
+    blocks: int = 1
+    conv_taps: int = 1
+    decay_rate: float = 8.0
 
 
 @dataclass(frozen=True)
@@ -224,7 +260,9 @@ class GatedAttentionSpec(PartSpec):
     `qk_norm_weight` False (scope "head" only): the norm of every head of q and k has no weight (such a norm is the
     same before the rotation and after it); `values` "keys": the values are the keys as projected, before norm and
     rotation, and there is no tensor `v`; `sink` s: a score s without a key or a value takes part in every softmax's
-    sum, so that the weights add up to less than one.
+    sum, so that the weights add up to less than one; `value_mix` "mixed": the values that are cached and attended to
+    are (1 - vmix) v + vmix v_source, with `vmix` a number of the layer and v_source the values, as projected, that the
+    model's layer with `value_mix` "source" made of the same token (an earlier layer of equal value sizes).
     """
 
     kind: str = field(init=False, default="gated_attention")
@@ -252,6 +290,7 @@ class GatedAttentionSpec(PartSpec):
     qk_norm_weight: bool = True
     values: str = "projected"            # "projected": by the tensor `v`; "keys": the keys as projected
     sink: float | None = None            # None: no sink
+    value_mix: str = "none"              # "none", "source" (this layer's values are mixed into later layers'), "mixed"
 
 
 @dataclass(frozen=True)
@@ -447,7 +486,8 @@ class BlockSpec:
     x + mixer(norm(x)) followed by x + ffn(norm(x)) with the adds deferred into the next norm;
     "sandwich_norm" norms each sublayer's output as well, x + norm_b(mixer(norm(x))), around a
     float32 residual stream; "pre_norm_stream" is "pre_norm" around a float32 residual stream;
-    "post_norm_stream" norms the sublayers' outputs only, x + norm(mixer(x)), around a float32 stream.
+    "post_norm_stream" norms the sublayers' outputs only, x + norm(mixer(x)), around a float32 stream;
+    "parallel_stream" is x + branch_scale * (mixer(h) + ffn(h)) with one norm h = norm(x), around a float32 stream.
     """
 
     arrangement: str
@@ -465,6 +505,7 @@ class BlockSpec:
     feed_forward_post_norm: PartSpec | None = None
     mixer_post_norm_prefix: str = ""
     feed_forward_post_norm_prefix: str = ""
+    branch_scale: float = 1.0        # multiplies what the sublayers add to the stream ("parallel_stream")
 
 
 @dataclass(frozen=True)
@@ -501,6 +542,7 @@ class ModelSpec:
     embedding_position: PartSpec | None = None  # a position vector added to the scaled embedding rows (`SinusoidSpec`)
     embedding_norm: PartSpec | None = None     # a norm of the embedding rows before they start the stream (a stream norm's spec)
     embedding_norm_prefix: str = ""            # where its tensors live
+    embedding_pairs: PairEmbeddingSpec | None = None   # rows by (previous token, token) added to the scaled embedding rows
     logit_scale: float = 1.0                   # multiplies the logits
     logit_softcap: float = 0.0                 # c > 0: logits <- c tanh(logits / c), after the scale
 

@@ -20,12 +20,14 @@
 // depends on the query's position only.  In a step of few tokens (decoding) a token's keys are split over
 // several CTAs, 128 keys each counted from the window's first key, and a second kernel merges the
 // partial results in key order: again nothing depends on the rest of the batch.
+// With `sink` (a number a head), exp(sink[h]) takes part in the sum of head h's softmax without a key or a value: it
+// is added once, where the output is divided by the sum (the merging kernel of a split step).
 #include "common.cuh"
 
 bool ts_latent_mma_supported(int rank, int rot);
 int ts_latent_attention_mma_launch(const float* q_lat, long long ql_t, long long ql_h, const void* q, long long q_stride,
-                                   int q_head_width, int q_rot_offset, const float* freq, const void* k_pool,
-                                   KVGeometry geo, const int* block_table, int table_width, const int* positions,
+                                   int q_head_width, int q_rot_offset, const float* freq, float magnitude,
+                                   const float* sink, const void* k_pool, KVGeometry geo, const int* block_table, int table_width, const int* positions,
                                    const int* seq_of_token, void* out, int num_tokens, int heads, int rank, int rot,
                                    float scale, int window, int split_keys, int splits, float* partial, cudaStream_t stream);
 
@@ -36,7 +38,7 @@ constexpr int LA_SPLIT = 128;       // keys of one CTA when a small step's keys 
 template <typename T>
 __global__ void latent_prepare_kernel(const T* __restrict__ y, long long y_stride, int q_rank, int rank, int rot,
                                       const float* __restrict__ wq, const float* __restrict__ wkv, float eps,
-                                      const float* __restrict__ freq, const int* __restrict__ positions,
+                                      const float* __restrict__ freq, float magnitude, const int* __restrict__ positions,
                                       const int* __restrict__ seq_of_token, T* __restrict__ cq, T* k_pool, KVGeometry geo,
                                       const int* __restrict__ block_table, int table_width, int writes) {
     __shared__ float scratch[32];
@@ -67,6 +69,8 @@ __global__ void latent_prepare_kernel(const T* __restrict__ y, long long y_strid
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float sn, cs;
         sincosf((float)pos * freq[i], &sn, &cs);
+        sn *= magnitude;
+        cs *= magnitude;
         const float u = to_float<T>(kr[i]), v = to_float<T>(kr[i + half]);
         dst[rank + i] = from_float<T>(u * cs - v * sn);
         dst[rank + i + half] = from_float<T>(v * cs + u * sn);
@@ -74,7 +78,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ y, long long y_strid
 }
 
 TS_API int ts_latent_prepare(const void* y, long long y_stride, int q_rank, int rank, int rot, const float* wq,
-                             const float* wkv, float eps, const float* freq, const int* positions,
+                             const float* wkv, float eps, const float* freq, float magnitude, const int* positions,
                              const int* seq_of_token, void* cq, void* k_pool, long long page_stride, long long entry_offset,
                              int page_tokens, int num_pages, const int* block_table, int table_width, int writes,
                              int num_tokens, int dtype, cudaStream_t stream) {
@@ -84,10 +88,10 @@ TS_API int ts_latent_prepare(const void* y, long long y_stride, int q_rank, int 
     KVGeometry geo{page_stride, entry_offset, page_tokens, num_pages};
     if (dtype == TS_F32)
         latent_prepare_kernel<float><<<num_tokens, 128, 0, stream>>>((const float*)y, y_stride, q_rank, rank, rot, wq, wkv,
-            eps, freq, positions, seq_of_token, (float*)cq, (float*)k_pool, geo, block_table, table_width, writes);
+            eps, freq, magnitude, positions, seq_of_token, (float*)cq, (float*)k_pool, geo, block_table, table_width, writes);
     else if (dtype == TS_BF16)
         latent_prepare_kernel<__nv_bfloat16><<<num_tokens, 128, 0, stream>>>((const __nv_bfloat16*)y, y_stride, q_rank, rank,
-            rot, wq, wkv, eps, freq, positions, seq_of_token, (__nv_bfloat16*)cq, (__nv_bfloat16*)k_pool, geo, block_table,
+            rot, wq, wkv, eps, freq, magnitude, positions, seq_of_token, (__nv_bfloat16*)cq, (__nv_bfloat16*)k_pool, geo, block_table,
             table_width, writes);
     else
         return ts_fail("latent_prepare: unknown dtype code %d", dtype);
@@ -95,11 +99,21 @@ TS_API int ts_latent_prepare(const void* y, long long y_stride, int q_rank, int 
     return 0;
 }
 
+// What the unscaled output (maximum mx taken off its exponents, sum l) is multiplied by: 1 / (l + exp(sink - mx)); where
+// the sink is above the maximum, in the form that cannot overflow.  l = 0: no key, output 0.
+__device__ __forceinline__ float latent_inverse_sum(float mx, float l, float sink) {
+    if (!(l > 0.f)) return 0.f;
+    if (sink <= mx) return 1.f / (l + expf(sink - mx));
+    const float e = expf(mx - sink);
+    return e / (l * e + 1.f);
+}
+
 template <typename T, int MAXR>
 __global__ void __launch_bounds__(LA_WARPS * 32)
 latent_attention_kernel(const float* __restrict__ q_lat, long long ql_token_stride, long long ql_head_stride,
                         const T* __restrict__ q, long long q_stride, int q_head_width, int q_rot_offset,
-                        const float* __restrict__ freq, const T* __restrict__ k_pool, KVGeometry geo,
+                        const float* __restrict__ freq, float magnitude, const float* __restrict__ sink,
+                        const T* __restrict__ k_pool, KVGeometry geo,
                         const int* __restrict__ block_table, int table_width, const int* __restrict__ positions,
                         const int* __restrict__ seq_of_token, T* __restrict__ out, int heads, int rank, int rot, float scale,
                         int window, int split_keys, float* __restrict__ partial) {
@@ -123,6 +137,8 @@ latent_attention_kernel(const float* __restrict__ q_lat, long long ql_token_stri
         for (int i = lane; i < half; i += 32) {
             float sn, cs;
             sincosf((float)pos * freq[i], &sn, &cs);
+            sn *= magnitude;
+            cs *= magnitude;
             const float u = to_float<T>(qr[i]), v = to_float<T>(qr[i + half]);
             mine[rank + i] = u * cs - v * sn;
             mine[rank + i + half] = v * cs + u * sn;
@@ -208,7 +224,7 @@ latent_attention_kernel(const float* __restrict__ q_lat, long long ql_token_stri
         }
         return;
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    const float inv = latent_inverse_sum(mx, l, sink ? sink[h] : -INFINITY);
     T* dst = out + ((long long)t * heads + h) * rank;
 #pragma unroll
     for (int m = 0; m < MAXR; ++m) {
@@ -224,7 +240,8 @@ constexpr int LC_MAX_SPLITS = 1024;
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, long long items, int splits, int rank) {
+latent_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, long long items, int splits, int rank,
+                      int heads, const float* __restrict__ sink) {
     __shared__ float weight[LC_MAX_SPLITS];
     const long long item = blockIdx.x;
     const float* p = partial + item * splits * (rank + 2);
@@ -242,7 +259,7 @@ latent_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, lo
             total += l * w;
         }
         total = warp_sum(total);
-        const float inv = total > 0.f ? 1.f / total : 0.f;
+        const float inv = latent_inverse_sum(mx, total, sink ? sink[(int)(item % heads)] : -INFINITY);
         for (int z = lane; z < splits; z += 32) weight[z] *= inv;
     }
     __syncthreads();
@@ -255,7 +272,8 @@ latent_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, lo
 
 template <typename T>
 static int launch_latent(const float* q_lat, long long ql_t, long long ql_h, const void* q, long long q_stride,
-                         int q_head_width, int q_rot_offset, const float* freq, const void* k_pool, KVGeometry geo,
+                         int q_head_width, int q_rot_offset, const float* freq, float magnitude, const float* sink,
+                         const void* k_pool, KVGeometry geo,
                          const int* block_table, int table_width, const int* positions, const int* seq_of_token, void* out,
                          int num_tokens, int heads, int rank, int rot, float scale, int window, int split_keys, int splits,
                          float* partial, cudaStream_t stream) {
@@ -268,7 +286,8 @@ static int launch_latent(const float* q_lat, long long ql_t, long long ql_h, con
             cudaFuncSetAttribute(latent_attention_kernel<T, MAXR>, cudaFuncAttributeMaxDynamicSharedMemorySize,      \
                                  (int)smem);                                                                         \
         latent_attention_kernel<T, MAXR><<<grid, LA_WARPS * 32, smem, stream>>>(                                     \
-            q_lat, ql_t, ql_h, (const T*)q, q_stride, q_head_width, q_rot_offset, freq, (const T*)k_pool, geo,       \
+            q_lat, ql_t, ql_h, (const T*)q, q_stride, q_head_width, q_rot_offset, freq, magnitude, sink,             \
+            (const T*)k_pool, geo,                                                                                   \
             block_table, table_width, positions, seq_of_token, (T*)out, heads, rank, rot, scale, window, split_keys, \
             partial);                                                                                                \
     } while (0)
@@ -279,7 +298,8 @@ static int launch_latent(const float* q_lat, long long ql_t, long long ql_h, con
     TS_LAUNCH_CHECK("latent_attention");
     if (split_keys > 0) {
         const long long items = (long long)num_tokens * heads;
-        latent_combine_kernel<T><<<(unsigned)items, 128, 0, stream>>>(partial, (T*)out, items, splits, rank);
+        latent_combine_kernel<T><<<(unsigned)items, 128, 0, stream>>>(partial, (T*)out, items, splits, rank,
+                                                                        heads, sink);
         TS_LAUNCH_CHECK("latent_attention (combine)");
     }
     return 0;
@@ -295,7 +315,7 @@ TS_API long long ts_latent_attention_scratch_floats(int num_tokens, int heads, i
 
 TS_API int ts_latent_attention(const float* q_lat, long long ql_token_stride, long long ql_head_stride, const void* q,
                                long long q_stride, int q_head_width, int q_rot_offset, const float* freq,
-                               const void* k_pool, long long page_stride, long long entry_offset, int page_tokens,
+                               float magnitude, const float* sink, const void* k_pool, long long page_stride, long long entry_offset, int page_tokens,
                                int num_pages, const int* block_table, int table_width, const int* positions,
                                const int* seq_of_token, void* out, int num_tokens, int heads, int rank, int rot,
                                float scale, int window, int max_keys, float* scratch, long long scratch_floats, int dtype,
@@ -322,24 +342,24 @@ TS_API int ts_latent_attention(const float* q_lat, long long ql_token_stride, lo
         (uintptr_t)k_pool % 16 == 0) {
         // bfloat16 with sizes the tensor-core kernel takes: heads as the rows of mma.sync products
         if (ts_latent_attention_mma_launch(q_lat, ql_token_stride, ql_head_stride, q, q_stride, q_head_width, q_rot_offset,
-                                           freq, k_pool, geo, block_table, table_width, positions, seq_of_token, out,
+                                           freq, magnitude, sink, k_pool, geo, block_table, table_width, positions, seq_of_token, out,
                                            num_tokens, heads, rank, rot, scale, window, split_keys, splits, scratch, stream))
             return 1;
         if (split_keys > 0) {
             const long long items = (long long)num_tokens * heads;
             latent_combine_kernel<__nv_bfloat16><<<(unsigned)items, 128, 0, stream>>>(
-                scratch, (__nv_bfloat16*)out, items, splits, rank);
+                scratch, (__nv_bfloat16*)out, items, splits, rank, heads, sink);
             TS_LAUNCH_CHECK("latent_attention (combine)");
         }
         return 0;
     }
     if (dtype == TS_F32)
         return launch_latent<float>(q_lat, ql_token_stride, ql_head_stride, q, q_stride, q_head_width, q_rot_offset, freq,
-                                    k_pool, geo, block_table, table_width, positions, seq_of_token, out, num_tokens, heads,
+                                    magnitude, sink, k_pool, geo, block_table, table_width, positions, seq_of_token, out, num_tokens, heads,
                                     rank, rot, scale, window, split_keys, splits, scratch, stream);
     if (dtype == TS_BF16)
         return launch_latent<__nv_bfloat16>(q_lat, ql_token_stride, ql_head_stride, q, q_stride, q_head_width, q_rot_offset,
-                                            freq, k_pool, geo, block_table, table_width, positions, seq_of_token, out,
+                                            freq, magnitude, sink, k_pool, geo, block_table, table_width, positions, seq_of_token, out,
                                             num_tokens, heads, rank, rot, scale, window, split_keys, splits, scratch, stream);
     return ts_fail("latent_attention: unknown dtype code %d", dtype);
 }

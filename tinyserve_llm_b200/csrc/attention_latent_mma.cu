@@ -13,6 +13,7 @@
 // latent part, whose rounding the unfolded form of the attention does not have, and the probabilities; the
 // logits then differ from the float32 kernel's no more than that kernel's from the plain model (measured: the
 // largest error of a replay fell from 0.5 to 0.3 of its bound, for 15 % of the kernel's time).
+// A sink (a number a head) joins a head's sum where the output is divided by it.
 // A small step's keys may be split over CTAs exactly as in the FFMA kernel; the partial results have the
 // same form and the same kernel merges them.
 #include "common.cuh"
@@ -45,7 +46,8 @@ template <int NT>
 __global__ void __launch_bounds__(LM_WARPS * 32)
 latent_attention_mma_kernel(const float* __restrict__ q_lat, long long ql_token_stride, long long ql_head_stride,
                             const __nv_bfloat16* __restrict__ q, long long q_stride, int q_head_width, int q_rot_offset,
-                            const float* __restrict__ freq, const __nv_bfloat16* __restrict__ k_pool, KVGeometry geo,
+                            const float* __restrict__ freq, float magnitude, const float* __restrict__ sink,
+                            const __nv_bfloat16* __restrict__ k_pool, KVGeometry geo,
                             const int* __restrict__ block_table, int table_width, const int* __restrict__ positions,
                             const int* __restrict__ seq_of_token, __nv_bfloat16* __restrict__ out, int heads, int rot,
                             float scale, int window, int split_keys, float* __restrict__ partial) {
@@ -82,6 +84,8 @@ latent_attention_mma_kernel(const float* __restrict__ q_lat, long long ql_token_
             const __nv_bfloat16* qr = q + (long long)t * q_stride + (long long)(h0 + r) * q_head_width + q_rot_offset;
             float sn, cs;
             sincosf((float)pos * freq[i], &sn, &cs);
+            sn *= magnitude;
+            cs *= magnitude;
             const float u = __bfloat162float(qr[i]), v = __bfloat162float(qr[i + half]);
             a = u * cs - v * sn;
             b = v * cs + u * sn;
@@ -248,7 +252,11 @@ latent_attention_mma_kernel(const float* __restrict__ q_lat, long long ql_token_
                 dst[2 + ch0 + nt * 8 + 2 * quad + 1] = o[nt][2 * r2 + 1];
             }
         } else {
-            const float inv = l > 0.f ? 1.f / l : 0.f;
+            float inv = l > 0.f ? 1.f / l : 0.f;
+            if (sink && l > 0.f) {                         // exp(sink) joins the sum; above the maximum in the form that cannot overflow
+                const float d = sink[h] - m_run[r2], e = expf(-fabsf(d));
+                inv = d <= 0.f ? 1.f / (l + e) : e / (l * e + 1.f);
+            }
             __nv_bfloat16* dst = out + ((long long)t * heads + h) * RANK;
 #pragma unroll
             for (int nt = 0; nt < NT; ++nt)
@@ -269,8 +277,8 @@ bool ts_latent_mma_supported(int rank, int rot) {
 }
 
 int ts_latent_attention_mma_launch(const float* q_lat, long long ql_t, long long ql_h, const void* q, long long q_stride,
-                                   int q_head_width, int q_rot_offset, const float* freq, const void* k_pool,
-                                   KVGeometry geo, const int* block_table, int table_width, const int* positions,
+                                   int q_head_width, int q_rot_offset, const float* freq, float magnitude,
+                                   const float* sink, const void* k_pool, KVGeometry geo, const int* block_table, int table_width, const int* positions,
                                    const int* seq_of_token, void* out, int num_tokens, int heads, int rank, int rot,
                                    float scale, int window, int split_keys, int splits, float* partial,
                                    cudaStream_t stream) {
@@ -284,7 +292,7 @@ int ts_latent_attention_mma_launch(const float* q_lat, long long ql_t, long long
         if (smem > 48 * 1024)                                                                                          \
             cudaFuncSetAttribute(latent_attention_mma_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         latent_attention_mma_kernel<NT><<<grid, LM_WARPS * 32, smem, stream>>>(                                        \
-            q_lat, ql_t, ql_h, (const __nv_bfloat16*)q, q_stride, q_head_width, q_rot_offset, freq,                    \
+            q_lat, ql_t, ql_h, (const __nv_bfloat16*)q, q_stride, q_head_width, q_rot_offset, freq, magnitude, sink,   \
             (const __nv_bfloat16*)k_pool, geo, block_table, table_width, positions, seq_of_token, (__nv_bfloat16*)out, \
             heads, rot, scale, window, split_keys, partial);                                                           \
     } while (0)

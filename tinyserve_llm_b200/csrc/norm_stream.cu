@@ -17,6 +17,11 @@
 // With a second branch (`branch2`) the sublayer is two mixers side by side whose outputs are normed one by one:
 //   b = branch_scale * branch / sqrt(mean(branch^2) + eps) * w_branch + branch_scale2 * (the same of branch2 with w_branch2)
 // takes the place of the branch; with a closing weight of null and no plain add, b itself goes to `out` (no stream).
+// Branches without norms of their own (null `w_branch`, TS_NORM_PLAIN_ADD) are added as they are, each times its scale.
+//
+// With `pairs.table` the gathered embedding row (times `scale`) gets a second row added, of a table of buckets + 1 rows
+// picked by (previous token, token): (previous * mul_prev + token * mul_cur) mod buckets, the last row where there is no
+// previous token.  The previous token is the one before in the batch, or prev_tokens[request] for a request's first row.
 //
 // `flags`: TS_NORM_CENTERED makes the opening norm a layer norm without bias,
 //   opening(s) = (s - mean(s)) / sqrt(mean((s - mean(s))^2) + eps) * w_open;
@@ -35,13 +40,30 @@ struct BranchPair {
     float scale, scale2;
 };
 
+// A second embedding by (previous token, token); null `table`: none.
+struct PairTable {
+    const void* table;
+    const int* prev_tokens; const int* cu_q; const int* seq_of_token;
+    int buckets;
+    long long mul_prev, mul_cur;
+};
+
+// The row of the pair table for batch row `r` (a padding row: -1).
+__device__ __forceinline__ long long pair_row(const PairTable& p, const int* ids, int r) {
+    const int seq = p.seq_of_token[r];
+    if (seq < 0) return -1;
+    const int prev = r > p.cu_q[seq] ? ids[r - 1] : p.prev_tokens[seq];
+    if (prev < 0) return p.buckets;
+    return (prev * p.mul_prev + ids[r] * p.mul_cur) % p.buckets;
+}
+
 template <typename T>
 __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __restrict__ w_close, float* stream,
                                    const float* __restrict__ w_open, T* __restrict__ out,
                                    const int* __restrict__ rows, int width, float eps, const T* __restrict__ table,
                                    const int* __restrict__ ids, int table_rows, float scale, int write_stream,
                                    int flags, const int* __restrict__ positions, const float* __restrict__ pos_freq,
-                                   const float* __restrict__ w_start, BranchPair pair) {
+                                   const float* __restrict__ w_start, BranchPair pair, PairTable pairs) {
     extern __shared__ float row[];                // width floats, then 64 of scratch
     float* scratch = row + width;
     const int r = blockIdx.x;
@@ -49,7 +71,7 @@ __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __
     if (src < 0) return;                          // a padding row
     float* sr = stream + (long long)src * width;
     T* o = out + (long long)r * width;
-    if (pair.branch2) {                           // the two branches' norms; their sum stands in for the branch from here on
+    if (pair.branch2 && pair.w_branch) {          // the two branches' norms; their sum stands in for the branch from here on
         const T* b1 = branch + (long long)src * width;
         const T* b2 = (const T*)pair.branch2 + (long long)src * width;
         float acc1 = 0.f, acc2 = 0.f;
@@ -89,6 +111,11 @@ __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __
                 const float angle = pos * pos_freq[i >> 1];
                 row[i] = (zeros ? 0.f : to_float<T>(tr[i]) * scale) + ((i & 1) ? cosf(angle) : sinf(angle));
             }
+        } else if (pairs.table && !zeros) {
+            const long long pr = pair_row(pairs, ids, src);
+            const T* second = (const T*)pairs.table + (pr < 0 ? 0 : pr) * width;
+            for (int i = threadIdx.x; i < width; i += blockDim.x)
+                row[i] = to_float<T>(tr[i]) * scale + (pr < 0 ? 0.f : to_float<T>(second[i]));
         } else {
             for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] = zeros ? 0.f : to_float<T>(tr[i]) * scale;
         }
@@ -108,7 +135,13 @@ __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __
         }
     } else if (branch && (flags & TS_NORM_PLAIN_ADD)) {
         const T* br = branch + (long long)src * width;
-        for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] = sr[i] + to_float<T>(br[i]);
+        if (pair.branch2) {
+            const T* b2 = (const T*)pair.branch2 + (long long)src * width;
+            for (int i = threadIdx.x; i < width; i += blockDim.x)
+                row[i] = sr[i] + (pair.scale * to_float<T>(br[i]) + pair.scale2 * to_float<T>(b2[i]));
+        } else {
+            for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] = sr[i] + pair.scale * to_float<T>(br[i]);
+        }
     } else if (branch) {
         const T* br = branch + (long long)src * width;
         float acc = 0.f;
@@ -147,9 +180,15 @@ TS_API int ts_stream_norm(const void* branch, const float* w_close, float* strea
                           const int* rows, int count, int width, float eps, const void* table, const int* ids,
                           int table_rows, float scale, int flags, int dtype, const int* positions, const float* pos_freq,
                           const float* w_start, const void* branch2, const float* w_branch, const float* w_branch2,
-                          float branch_scale, float branch_scale2, cudaStream_t stream_handle) {
+                          float branch_scale, float branch_scale2, const void* pair_table, const int* prev_tokens,
+                          const int* cu_q, const int* seq_of_token, int buckets, long long mul_prev, long long mul_cur,
+                          cudaStream_t stream_handle) {
     TS_REQUIRE(count >= 0 && width > 0, "stream_norm: bad sizes rows=%d width=%d", count, width);
-    TS_REQUIRE(!branch2 || (branch && w_branch && w_branch2), "stream_norm: two branches need both their norms' weights");
+    TS_REQUIRE(!branch2 || (branch && (w_branch != nullptr) == (w_branch2 != nullptr)),
+               "stream_norm: two branches need both their norms' weights, or neither");
+    TS_REQUIRE(!branch2 || w_branch || (flags & TS_NORM_PLAIN_ADD), "stream_norm: branches without norms are added as they are");
+    TS_REQUIRE(!pair_table || (ids && !pos_freq && prev_tokens && cu_q && seq_of_token && buckets > 0 && mul_prev >= 0 && mul_cur >= 0),
+               "stream_norm: a pair table needs token ids, the previous tokens and the requests' rows, and no position vector");
     TS_REQUIRE(stream != nullptr || (branch2 && out && !w_open), "stream_norm: no residual stream");
     TS_REQUIRE(!(stream && branch && !w_close && !(flags & TS_NORM_PLAIN_ADD)),
                "stream_norm: a branch needs the weight of its closing norm");
@@ -165,6 +204,7 @@ TS_API int ts_stream_norm(const void* branch, const float* w_close, float* strea
     const int threads = count <= 512 ? wide : (width >= 1024 ? 256 : 128);
     const size_t smem = (size_t)(width + 64) * sizeof(float);
     const BranchPair pair{branch2, w_branch, w_branch2, branch_scale, branch_scale2};
+    const PairTable pairs{pair_table, prev_tokens, cu_q, seq_of_token, buckets, mul_prev, mul_cur};
     const int write = rows ? 0 : 1;
 #define TS_STREAM_NORM(TYPE)                                                                                      \
     do {                                                                                                          \
@@ -172,7 +212,7 @@ TS_API int ts_stream_norm(const void* branch, const float* w_close, float* strea
             cudaFuncSetAttribute(stream_norm_kernel<TYPE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         stream_norm_kernel<TYPE><<<count, threads, smem, stream_handle>>>(                                        \
             (const TYPE*)branch, w_close, stream, w_open, (TYPE*)out, rows, width, eps, (const TYPE*)table, ids,  \
-            table_rows, scale, write, flags, positions, pos_freq, w_start, pair);                                       \
+            table_rows, scale, write, flags, positions, pos_freq, w_start, pair, pairs);                                       \
     } while (0)
     if (dtype == TS_F32) TS_STREAM_NORM(float);
     else if (dtype == TS_BF16) TS_STREAM_NORM(__nv_bfloat16);

@@ -15,6 +15,7 @@
 // Keys and values may differ in their head size and in their number of heads (`v_heads`: several key heads over
 // one value head), so the value pool has a geometry of its own.  Values may also be the keys as projected: their
 // columns are then k's own (`v_off` = `k_off`), stored without norm and rotation.
+// With `v_mix` (a stretch of rows like v's own, of another layer) the stored value is (1 - v_lambda) v + v_lambda v_mix.
 // One CTA a token; sums, angles and the rotation are float32, the stores round to the activation dtype.
 #include "common.cuh"
 
@@ -30,6 +31,7 @@ struct QKPrepareArgs {
     int heads, kv_heads, dim, vdim, v_heads;
     int norm_per_head; float temp_coef; int temp_every;
     int unweighted, interleaved;
+    const void* v_mix; long long v_mix_stride; float v_lambda;
 };
 
 template <typename T>
@@ -128,10 +130,12 @@ __global__ void qk_norm_rope_store_kernel(QKPrepareArgs p) {
         const int h = e / p.dim, i = e % p.dim;
         kp[((long long)h * p.k_geo.page_tokens + slot) * p.dim + i] = from_float<T>(x);
     });
+    const T* mix = p.v_mix ? (const T*)p.v_mix + (long long)t * p.v_mix_stride : nullptr;
     for (int e = threadIdx.x; e < nv; e += blockDim.x) {
         const int h = e / p.vdim, i = e % p.vdim;
-        vp[((long long)h * p.v_geo.page_tokens + slot) * p.vdim + i] =
-            from_float<T>(to_float<T>(yv[e]) + (p.v_bias ? p.v_bias[e] : 0.f));
+        float v = to_float<T>(yv[e]) + (p.v_bias ? p.v_bias[e] : 0.f);
+        if (mix) v = (1.f - p.v_lambda) * v + p.v_lambda * to_float<T>(mix[e]);
+        vp[((long long)h * p.v_geo.page_tokens + slot) * p.vdim + i] = from_float<T>(v);
     }
 }
 
@@ -143,7 +147,8 @@ TS_API int ts_qk_norm_rope_store(const void* y, long long y_stride, int q_off, i
                                  int page_tokens, int num_pages, const int* block_table, int table_width, int writes,
                                  int num_tokens, int heads, int kv_heads, int dim, int vdim, int dtype,
                                  int norm_per_head, float temp_coef, int temp_every, int value_heads, int unweighted,
-                                 int interleaved, cudaStream_t stream) {
+                                 int interleaved, const void* v_mix, long long v_mix_stride, float v_lambda,
+                                 cudaStream_t stream) {
     TS_REQUIRE(!unweighted || (norm_per_head && !q_weight && !k_weight), "qk_norm_rope_store: an unweighted norm is one a head");
     TS_REQUIRE(value_heads >= 0, "qk_norm_rope_store: bad number of value heads");
     TS_REQUIRE(heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && num_tokens >= 0, "qk_norm_rope_store: bad sizes");
@@ -155,7 +160,7 @@ TS_API int ts_qk_norm_rope_store(const void* y, long long y_stride, int q_off, i
                     KVGeometry{k_page_stride, k_entry_offset, page_tokens, num_pages},
                     KVGeometry{v_page_stride, v_entry_offset, page_tokens, num_pages}, block_table, table_width, writes,
                     heads, kv_heads, dim, vdim, value_heads > 0 ? value_heads : kv_heads, norm_per_head, temp_coef, temp_every,
-                    unweighted, interleaved};
+                    unweighted, interleaved, v_mix, v_mix_stride, v_lambda};
     const size_t smem = norm_per_head ? (size_t)(heads + kv_heads) * sizeof(float) : 0;
     TS_REQUIRE(smem <= 32 * 1024, "qk_norm_rope_store: %d heads are not supported", heads + kv_heads);
     // many tokens: small CTAs, many of them on an SM (a CTA's life is a chain of loads and two sums); few tokens: wide ones

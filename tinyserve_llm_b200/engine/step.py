@@ -62,6 +62,8 @@ class StepContext:
         self.state_slots: torch.Tensor = None     # int32 [S]
         self.rows: torch.Tensor = None            # int32 [R] flat rows whose logits are wanted
         self.prefill_seqs: torch.Tensor = None    # int32 [P] requests that feed more than one token (prompt portions)
+        self.prev_tokens: torch.Tensor = None     # int32 [S] the token before each request's first one of the step (-1: none);
+                                                  # empty unless the model embeds token pairs
         self.tables: list[torch.Tensor] = []      # per pool of the cache manager int32 [S, width]
         lens = [b - a for a, b in zip(host.cu_q, host.cu_q[1:])]
         self.max_q_len = max(lens, default=0)     # which attention kernels a step needs is decided on the host
@@ -164,6 +166,7 @@ class StepRunner:
         self.manager = manager
         self.storage = storage
         self.device = model.rt.device
+        self._pairs = model.embedding_pairs is not None
         self.bindings = [storage.entry_binding(e) for e in range(model.spec.num_cache_entries)]
         self._staging: torch.Tensor | None = None       # pinned int32 buffer for the step's index data
         self._staged = torch.cuda.Event()
@@ -225,8 +228,9 @@ class StepRunner:
         """
         The step's index data as one list of int32 words in sections (each padded to 16 bytes):
         token ids, positions, request of each token, offsets of the requests' tokens, lengths after
-        this step, wanted rows, state slots, one block table per pool of the cache manager, and the requests
-        that feed more than one token.  With `shape`, every section is padded to the shape's size.
+        this step, wanted rows, state slots, one block table per pool of the cache manager, the requests
+        that feed more than one token, and (for models that embed token pairs) the token before each
+        request's first one.  With `shape`, every section is padded to the shape's size.
         Returns (words, offset of each section, sizes).
         """
         seqs = self.manager.seqs
@@ -257,6 +261,8 @@ class StepRunner:
                 if k > 1:
                     portions.append(s)
         slots = [st.state_slot for st in states]
+        # a committed token is never pending: the host has seen the sample before it committed it
+        previous = [st.tokens[st.committed - 1] if st.committed else -1 for st in states] if self._pairs else []
         T, R, P = len(ids), len(rows), len(portions)
         if shape is None:
             widths = [max(1, max(len(st.tables[g]) for st in states)) for g in range(groups)]
@@ -274,6 +280,8 @@ class StepRunner:
             slots = slots + [-1] * (S - n)
             rows = rows + [0] * (S - R)
             portions = portions + [-1] * (shape.portions - P)
+            if self._pairs:
+                previous = previous + [-1] * (S - n)
         sections = [ids, positions, seq_of_token, cu_q, ctx_lens, rows, slots]
         for g in range(groups):
             flat: list[int] = []
@@ -289,6 +297,7 @@ class StepRunner:
                 flat.extend([-1] * (width * (S - n)))
             sections.append(flat)
         sections.append(portions)
+        sections.append(previous)
         offsets, words = [], []
         for sec in sections:
             offsets.append(len(words))
@@ -341,6 +350,7 @@ class StepRunner:
         groups = len(widths)
         ctx.tables = [view(7 + g, S * widths[g]).view(S, widths[g]) for g in range(groups)]
         ctx.prefill_seqs = view(7 + groups, P)
+        ctx.prev_tokens = view(8 + groups, S if self._pairs else 0)
         return ctx
 
     # ------------------------------------------------------------------ the step

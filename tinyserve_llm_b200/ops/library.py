@@ -58,11 +58,11 @@ _SIGNATURES = {
     "ts_skinny_linear_unary": ("int", "pppiiilliffip"),
     "ts_skinny_linear_groups": ("int", "pppiiiillllip"),
     "ts_gemm_tcgen05_gated": ("int", "pppiiilliffpp"),
-    "ts_stream_norm": ("int", "ppppppiifppifiippp" "pppff" "p"),
+    "ts_stream_norm": ("int", "ppppppiifppifiippp" "pppff" "ppppill" "p"),
     "ts_linear_recurrence": ("int", "ppplllplppfffpipppiplpiiiipip"),
     "ts_head_norm_gate": ("int", "piplpippliiififip"),
-    "ts_latent_prepare": ("int", "pliiippfppppplliipiiiip"),
-    "ts_latent_attention": ("int", "pllpliipplliipipppiiiifiiplip"),
+    "ts_latent_prepare": ("int", "pliiippfp" "f" "pppplliipiiiip"),
+    "ts_latent_attention": ("int", "pllpliip" "fp" "plliipipppiiiifiiplip"),
     "ts_latent_attention_scratch_floats": ("long long", "iiii"),
     "ts_set_latent_mma": ("void", "i"),
     "ts_moe_route": ("int", "ppppppiiiip"),
@@ -72,10 +72,15 @@ _SIGNATURES = {
     "ts_moe_route_grouped": ("int", "pppppppiiiiiiffp"),
     "ts_paged_attention_scored": ("int", "plpppllllii" "pippiiiiifiiipppl" "fiiif" "p"),
     "ts_mingru_scan": ("int", "pliiiippppiplpiiiip"),
+    "ts_lru_decode_supported": ("int", "iiili"),
+    "ts_lru_decode": ("int", "pliipppppppppp" "ipl" "piiii" "pp"),
+    "ts_lru_conv": ("int", "pliipppppppppp" "ipl" "piiii" "ip"),
+    "ts_lru_scan_scratch_floats": ("long long", "iii"),
+    "ts_lru_scan": ("int", "pliipppppppppp" "ipl" "piiii" "ppllpii" "plip"),
     "ts_unary_activation_rows": ("int", "ppliffip"),
     "ts_gated_activation": ("int", "ppiiiffip"),
     "ts_sgemm_nt_batched": ("int", "pppiiilllilllp"),
-    "ts_qk_norm_rope_store": ("int", "pliiipppppfpifpppppllllii" "piiiiiiiiifiiiip"),
+    "ts_qk_norm_rope_store": ("int", "pliiipppppfpifpppppllllii" "piiiiiiiiifiiii" "plf" "p"),
     "ts_sigmoid_gate": ("int", "plplpliifip"),
     "ts_paged_attention_split": ("int", "plpppllllii" "pippiiiiifiip"),
     "ts_short_conv_silu": ("int", "plppppiplpiiiip"),
@@ -184,6 +189,8 @@ class Ops:
         self.swiglu_skinny_rows = self.skinny_max_rows
         # TINYSERVE_B200_TILES=0 keeps the recurrences that have a form of sixteen tokens at a time on the scan token by token
         self.recurrence_tiles = os.environ.get("TINYSERVE_B200_TILES", "1") != "0"
+        # TINYSERVE_B200_LRU=split keeps a gated linear recurrent unit's decode steps on the kernels of prompt portions
+        self.lru_fused_decode = os.environ.get("TINYSERVE_B200_LRU", "fused") != "split"
         # from this many (token, expert) pairs a routed feed-forward's bfloat16 products go to the library's grouped product
         self.grouped_mm_min_pairs = int(os.environ.get("TINYSERVE_B200_GROUPED_PAIRS", "256"))
 
@@ -454,7 +461,7 @@ class Ops:
                     table: torch.Tensor | None = None, ids: torch.Tensor | None = None, scale: float = 1.0,
                     centered: bool = False, plain_add: bool = False, positions: torch.Tensor | None = None,
                     position_frequencies: torch.Tensor | None = None, w_start: torch.Tensor | None = None,
-                    copy_out: bool = False, pair: tuple | None = None) -> torch.Tensor | None:
+                    copy_out: bool = False, pair: tuple | None = None, pairs: tuple | None = None) -> torch.Tensor | None:
         """
         stream (float32, in place) += closing norm of `branch` (if given; with `plain_add` the branch as
         it is); returns the opening norm of the sum in `dtype` (if `w_open` is given; with `centered` a
@@ -467,13 +474,18 @@ class Ops:
 
         `copy_out`: no opening norm; the new rows of the stream are returned in `dtype`.  `pair` (branch2, w1, w2,
         scale1, scale2): two branches of one sublayer, each RMS-normed with a weight of its own, whose sum
-        scale1 * norm(branch) * w1 + scale2 * norm(branch2) * w2 takes the branch's place.
+        scale1 * norm(branch) * w1 + scale2 * norm(branch2) * w2 takes the branch's place; with w1 and w2 None (and
+        `plain_add`) the branches are added as they are, scale1 * branch + scale2 * branch2 (branch2 may be None).
+        `pairs` (table, spec, step context), beside `table` and `ids`: table rows by (previous token, token) are added
+        to the gathered ones, as `PairEmbeddingSpec` says; the token ahead of a request's first row is ctx.prev_tokens'.
         """
         self._check(stream, "residual stream", torch.float32, 2)
         width = stream.shape[1]
         if copy_out and (w_open is not None or rows is not None):
             raise KernelError("stream_norm: a copy of the stream takes the place of the opening norm, for all rows")
         branch2, w_branch, w_branch2, scale1, scale2 = self._branch_pair(branch, pair, width)
+        if pair is not None and w_branch is None and not plain_add:
+            raise KernelError("stream_norm: branches without norms of their own are added as they are")
         if w_start is not None and ids is None:
             raise KernelError("stream_norm: a norm on the embedding rows needs token ids")
         for w, name in ((w_close, "closing weight"), (w_open, "opening weight"), (w_start, "embedding norm weight")):
@@ -495,6 +507,16 @@ class Ops:
             if ids is None or positions is None or position_frequencies.shape[0] < (width + 1) // 2:
                 raise KernelError("stream_norm: a position vector needs ids, positions and a frequency for every two columns")
             self._check(positions, "positions", torch.int32, 1)
+        pair_args = (0, 0, 0, 0, 0, 0, 0)
+        if pairs is not None:
+            pair_table, pair_spec, ctx = pairs
+            self._check(pair_table, "pair table", dtype, 2)
+            if ids is None or tuple(pair_table.shape) != (pair_spec.buckets + 1, width):
+                raise KernelError(f"stream_norm: a pair table of {tuple(pair_table.shape)}, expected {(pair_spec.buckets + 1, width)}, beside token ids")
+            if ctx.prev_tokens is None or ctx.prev_tokens.shape[0] != ctx.cu_q.shape[0] - 1 or ctx.seq_of_token.shape[0] != ids.shape[0]:
+                raise KernelError("stream_norm: a pair table needs the step's previous tokens, one a request")
+            pair_args = (_ptr(pair_table), _ptr(ctx.prev_tokens), _ptr(ctx.cu_q), _ptr(ctx.seq_of_token), pair_spec.buckets,
+                         pair_spec.mul_prev, pair_spec.mul_cur)
         count = stream.shape[0]
         if rows is not None:
             self._check(rows, "rows", torch.int32, 1)
@@ -506,19 +528,23 @@ class Ops:
                    width, eps, _ptr(table), _ptr(ids), table.shape[0] if table is not None else 0, scale,
                    (1 if centered else 0) | (2 if plain_add else 0) | (4 if copy_out else 0), _DTYPE_CODE[dtype],
                    _ptr(positions) if position_frequencies is not None else 0, _ptr(position_frequencies), _ptr(w_start),
-                   _ptr(branch2), _ptr(w_branch), _ptr(w_branch2), scale1, scale2, _stream())
+                   _ptr(branch2), _ptr(w_branch), _ptr(w_branch2), scale1, scale2, *pair_args, _stream())
         return out
 
     def _branch_pair(self, branch: torch.Tensor | None, pair: tuple | None, width: int) -> tuple:
         if pair is None:
-            return None, None, None, 0.0, 0.0
+            return None, None, None, 1.0, 0.0
         branch2, w1, w2, scale1, scale2 = pair
         if branch is None:
             raise KernelError("a pair of branches needs both")
+        if (w1 is None) != (w2 is None) or (branch2 is None and w1 is not None):
+            raise KernelError("the branches of a pair are both normed or neither")
+        if branch2 is None:
+            return None, None, None, float(scale1), 0.0
         self._check(branch2, "second branch", branch.dtype, 2)
         if branch2.shape != branch.shape:
             raise KernelError(f"the branches differ: {tuple(branch.shape)} and {tuple(branch2.shape)}")
-        for w in (w1, w2):
+        for w in (w1, w2) if w1 is not None else ():
             self._check(w, "branch norm weight", torch.float32, 1)
             if w.shape[0] != width:
                 raise KernelError(f"a branch norm weight has {w.shape[0]} elements for rows of {width}")
@@ -530,7 +556,7 @@ class Ops:
         branch2, w1, w2, scale1, scale2 = self._branch_pair(branch, pair, branch.shape[1])
         out = torch.empty_like(branch)
         self._call("ts_stream_norm", _ptr(branch), 0, 0, 0, _ptr(out), 0, branch.shape[0], branch.shape[1], eps, 0, 0, 0, 1.0, 0,
-                   _DTYPE_CODE[branch.dtype], 0, 0, 0, _ptr(branch2), _ptr(w1), _ptr(w2), scale1, scale2, _stream())
+                   _DTYPE_CODE[branch.dtype], 0, 0, 0, _ptr(branch2), _ptr(w1), _ptr(w2), scale1, scale2, 0, 0, 0, 0, 0, 0, 0, _stream())
         return out
 
     # ------------------------------------------------------------------ linear recurrences
@@ -602,7 +628,7 @@ class Ops:
     def qk_norm_rope_store(self, y: torch.Tensor, offsets: tuple[int, int, int], biases, weights, eps: float, position,
                            ctx, binding, heads: int, kv_heads: int, dim: int, vdim: int, *, norm_per_head: bool = False,
                            q_temperature: tuple[float, int] | None = None, value_heads: int = 0,
-                           unweighted_norm: bool = False) -> torch.Tensor:
+                           unweighted_norm: bool = False, value_mix: tuple[torch.Tensor, float] | None = None) -> torch.Tensor:
         """
         From the projection's output y (q, k, v at the column `offsets`): biases added (float32 tensors or
         None), q and k RMS-normed over the whole projection with `weights` (q's, k's; or None; with
@@ -611,6 +637,7 @@ class Ops:
         (coef, every), k and v stored into the token's cache slot.  `value_heads` (0: as many as key heads): v
         holds that many heads of vdim channels.  `unweighted_norm`: every head of q and of k is RMS-normed by
         itself without a weight.  The columns of v may be k's own: the value is then the key as projected.
+        `value_mix` (other, lambda): (1 - lambda) v + lambda other is stored, `other` a [T, v columns] stretch of y's dtype.
         Returns q [T, heads * dim].
         """
         if y.dtype not in _DTYPE_CODE or y.dim() != 2 or y.stride(1) != 1:
@@ -628,6 +655,10 @@ class Ops:
             if w is not None and w.numel() != (dim if norm_per_head else (heads if w is qw else kv_heads) * dim):
                 raise KernelError(f"qk_norm_rope_store: a norm weight of {w.numel()} elements")
         coef, every = q_temperature if q_temperature is not None else (0.0, 0)
+        other, lam = value_mix if value_mix is not None else (None, 0.0)
+        if other is not None and (other.dtype != y.dtype or other.dim() != 2 or other.stride(1) != 1
+                                  or tuple(other.shape) != (T, (value_heads or kv_heads) * vdim)):
+            raise KernelError(f"qk_norm_rope_store: the values to mix in must be a [T, {(value_heads or kv_heads) * vdim}] stretch of y's dtype")
         v_page_stride, v_entry_offset = binding.value_geometry()
         self._call("ts_qk_norm_rope_store", _ptr(y), y.stride(0), offsets[0], offsets[1], offsets[2], _ptr(qb), _ptr(kb),
                    _ptr(vb), _ptr(qw), _ptr(kw), eps, _ptr(freq), rot, magnitude, _ptr(ctx.positions),
@@ -635,7 +666,8 @@ class Ops:
                    binding.entry_offset, v_page_stride, v_entry_offset, binding.page_tokens, binding.num_pages,
                    _ptr(binding.block_table), binding.table_width, 1 if binding.writes else 0, T, heads, kv_heads, dim,
                    vdim, _DTYPE_CODE[y.dtype], 1 if norm_per_head or unweighted_norm else 0, float(coef), int(every),
-                   int(value_heads), 1 if unweighted_norm else 0, 1 if getattr(position, "interleaved", False) else 0, _stream())
+                   int(value_heads), 1 if unweighted_norm else 0, 1 if getattr(position, "interleaved", False) else 0,
+                   _ptr(other), other.stride(0) if other is not None else 0, float(lam), _stream())
         return q
 
     def paged_attention_split(self, q: torch.Tensor, ctx, binding, nh: int, nkv: int, hd: int, vd: int, scale: float,
@@ -870,6 +902,46 @@ class Ops:
                    _ptr(z_bias), _ptr(x_bias), _ptr(ctx.cu_q), _ptr(binding.state_slots), binding.state_slots.shape[0],
                    state.data_ptr(), stride, _ptr(out), width, T, int(getattr(ctx, "max_q_len", 0) or 0),
                    _DTYPE_CODE[dtype], _stream())
+        return out
+
+    def gated_lru(self, xy: torch.Tensor, unit, ctx, binding) -> torch.Tensor:
+        """
+        [T, width] in xy's dtype: from the projection's output xy [T, 2 width] = [y | x] to the input of the output
+        projection of a real-gated linear recurrent unit, S_t * gelu(y).  `unit` holds its tensors (`GatedLRU`): biases,
+        taps [taps, width], the gates' stacked matrices [blocks, 2 part, part] and biases [2, width], rates.
+        """
+        spec, dtype = unit.spec, xy.dtype
+        W, K = spec.width, spec.conv_taps
+        part = W // spec.blocks
+        if dtype not in _DTYPE_CODE or xy.dim() != 2 or xy.stride(1) != 1 or xy.shape[1] != 2 * W:
+            raise KernelError(f"gated_lru: xy must be a [T, {2 * W}] stretch of an activation dtype")
+        self._check(unit.gates, "gate matrices", dtype, 3)
+        T = xy.shape[0]
+        state, stride = self._state_floats(binding, W * (1 + (K if K > 1 else 0)), "gated_lru")
+        args = (_ptr(xy), xy.stride(0), 0, W, _ptr(unit.y_bias), _ptr(unit.x_bias), _ptr(unit.taps), _ptr(unit.conv_bias),
+                _ptr(unit.gate_bias), _ptr(unit.rate), _ptr(ctx.positions), _ptr(ctx.seq_of_token), _ptr(ctx.cu_q),
+                _ptr(binding.state_slots), binding.state_slots.shape[0], state.data_ptr(), stride)
+        out = torch.empty((T, W), dtype=dtype, device=xy.device)
+        if (ctx.max_q_len <= 1 and dtype == torch.bfloat16 and xy.data_ptr() % 16 == 0 and self.lru_fused_decode
+                and self.lib.ts_lru_decode_supported(T, W, part, xy.stride(0), W)):
+            self._call("ts_lru_decode", *args, _ptr(out), W, part, K, T, _ptr(unit.gates), _stream())
+            return out
+        u = torch.empty((T, W), dtype=dtype, device=xy.device)
+        self._call("ts_lru_conv", *args, _ptr(u), W, part, K, T, _DTYPE_CODE[dtype], _stream())
+        z = self.per_head_linear(u, unit.gates, spec.blocks, part, part)          # float32 [T, blocks, 2 part]
+        portions = getattr(ctx, "prefill_seqs", None)
+        if portions is not None and portions.shape[0] == 0:
+            portions = None
+        count, floats, scratch = 0, 0, None
+        if portions is not None:
+            count = portions.shape[0]
+            floats = int(self.lib.ts_lru_scan_scratch_floats(count, ctx.max_q_len, W))
+            if floats:
+                scratch = torch.empty((floats,), dtype=torch.float32, device=xy.device)
+        self._call("ts_lru_scan", *args, _ptr(out), W, part, K, T, _ptr(u), _ptr(z), z.stride(0), z.stride(1), _ptr(portions),
+                   count, int(ctx.max_q_len), _ptr(scratch), floats, _DTYPE_CODE[dtype], _stream())
+        if floats:
+            self.launches += 2                               # the stretches, then the walk over them
         return out
 
     UNARY_ACTIVATIONS = {"relu2": 0, "xielu": 1, "tanh": 2}
@@ -1149,11 +1221,12 @@ class Ops:
 
     # ------------------------------------------------------------------ attention over a cached latent
     def latent_prepare(self, y: torch.Tensor, ctx, binding, q_rank: int, rank: int, rot: int, q_weight: torch.Tensor,
-                       kv_weight: torch.Tensor, eps: float, freq: torch.Tensor) -> torch.Tensor:
+                       kv_weight: torch.Tensor, eps: float, freq: torch.Tensor, magnitude: float = 1.0) -> torch.Tensor:
         """
         y [T, q_rank + rank + rot] (the down projections' output, or a column stretch of it): returns the normed
         query latent [T, q_rank] and stores [norm(c) | rotated k_rot] into each token's slot of the cache entry.
-        q_rank 0 (queries without a latent) and rot 0 (no rotated part, `freq` None) are allowed.
+        q_rank 0 (queries without a latent) and rot 0 (no rotated part, `freq` None) are allowed; `magnitude` multiplies
+        cos and sin.
         """
         if y.dtype not in _DTYPE_CODE or y.dim() != 2 or y.stride(1) != 1 or not y.is_cuda:
             raise KernelError("latent_prepare: y must be a [T, columns] stretch of an activation dtype on the device")
@@ -1163,7 +1236,7 @@ class Ops:
             raise KernelError(f"cache pool is {binding.k_pool.dtype} but activations are {y.dtype}")
         c_q = torch.empty((y.shape[0], q_rank), dtype=y.dtype, device=y.device)
         self._call("ts_latent_prepare", _ptr(y), y.stride(0), q_rank, rank, rot, _ptr(q_weight), _ptr(kv_weight), eps,
-                   _ptr(freq), _ptr(ctx.positions), _ptr(ctx.seq_of_token), _ptr(c_q), _ptr(binding.k_pool),
+                   _ptr(freq), float(magnitude), _ptr(ctx.positions), _ptr(ctx.seq_of_token), _ptr(c_q), _ptr(binding.k_pool),
                    binding.page_stride, binding.entry_offset, binding.page_tokens, binding.num_pages,
                    _ptr(binding.block_table), binding.table_width, 1 if binding.writes else 0, y.shape[0],
                    _DTYPE_CODE[y.dtype], _stream())
@@ -1195,19 +1268,25 @@ class Ops:
         return torch.bmm(a, w.transpose(1, 2), out_dtype=out_dtype).transpose(0, 1)
 
     def latent_attention(self, q_lat: torch.Tensor, q: torch.Tensor, ctx, binding, heads: int, q_head_width: int,
-                         q_rot_offset: int, rank: int, rot: int, freq: torch.Tensor, scale: float, window: int) -> torch.Tensor:
+                         q_rot_offset: int, rank: int, rot: int, freq: torch.Tensor, scale: float, window: int, *,
+                         magnitude: float = 1.0, sink: torch.Tensor | None = None) -> torch.Tensor:
         """
         [T, heads, rank] in q's dtype: per head the softmax-weighted sum of the cached latents, scores
         (q_lat . c + rotated q_rot . k_rot) * scale over the keys the window leaves visible.  q_lat is
         float32 [T, heads, rank] (any token and head strides); the rotated part of the query is read from
         q [T, heads * q_head_width] (rows may be stretches of wider ones) at `q_rot_offset` inside each head and
-        rotated here; `rot` 0: there is no such part and `freq` may be None.
+        rotated here (cos and sin times `magnitude`); `rot` 0: there is no such part and `freq` may be None.  `sink`
+        (float32 [heads]): exp(sink[h]) takes part in the sum of every softmax of head h.
         """
         self._check_rows(q, "q")
         if q_lat.dtype != torch.float32 or q_lat.stride(2) != 1 or tuple(q_lat.shape) != (q.shape[0], heads, rank):
             raise KernelError("latent_attention: q_lat must be float32 [T, heads, rank] with unit channel stride")
         if binding.k_pool.dtype != q.dtype:
             raise KernelError(f"cache pool is {binding.k_pool.dtype} but activations are {q.dtype}")
+        if sink is not None:
+            self._check(sink, "sink", torch.float32, 1)
+            if sink.shape[0] != heads:
+                raise KernelError(f"latent_attention: {sink.shape[0]} sinks for {heads} heads")
         out = torch.empty((q.shape[0], heads, rank), dtype=q.dtype, device=q.device)
         # the most keys a token of this step sees: bounded by the window and by the longest request (a replayed step: its shape's bound)
         longest = getattr(ctx, "max_ctx_len", None)
@@ -1225,7 +1304,7 @@ class Ops:
                 if store is not None:
                     store[key] = scratch
         self._call("ts_latent_attention", _ptr(q_lat), q_lat.stride(0), q_lat.stride(1), _ptr(q), q.stride(0), q_head_width,
-                   q_rot_offset, _ptr(freq), _ptr(binding.k_pool), binding.page_stride, binding.entry_offset,
+                   q_rot_offset, _ptr(freq), float(magnitude), _ptr(sink), _ptr(binding.k_pool), binding.page_stride, binding.entry_offset,
                    binding.page_tokens, binding.num_pages, _ptr(binding.block_table), binding.table_width,
                    _ptr(ctx.positions), _ptr(ctx.seq_of_token), _ptr(out), q.shape[0], heads, rank, rot, scale, window,
                    max_keys, _ptr(scratch), floats, _DTYPE_CODE[q.dtype], _stream())

@@ -5,7 +5,7 @@ Arrangements: how a block wires its mixer, feed-forward and norms.
 into the following norm, so a block takes and returns (branch output, residual stream).
 "sandwich_norm" also norms each sublayer's output and keeps the stream in float32;
 "pre_norm_stream" is the pre-norm wiring around a float32 stream; "post_norm_stream" norms the
-sublayers' outputs only.
+sublayers' outputs only; in "parallel_stream" mixer and feed-forward read one norm's output side by side.
 """
 
 from __future__ import annotations
@@ -230,3 +230,55 @@ class PostNormStreamBlock:
             return branch, residual
         h = self.mixer_post_norm.close_and_copy(branch, residual)
         return PendingBranch(self.feed_forward.forward(h, ctx), self.feed_forward_post_norm), residual
+
+
+@register_arrangement("parallel_stream")
+class ParallelStreamBlock:
+    """
+    h = norm(x); x = x + branch_scale * (mixer(h) + ffn(h)) around a residual stream kept in float32: the two
+    sublayers' outputs travel on as one `PendingBranch`, and the next norm of the stream adds both to it and norms
+    the sum in one kernel.  A block without a feed-forward adds its mixer's output alone.
+    """
+
+    takes_token_ids = True
+    takes_embedding_scale = True
+    takes_embedding_position = True
+    takes_embedding_norm = True
+    takes_embedding_pairs = True
+
+    @staticmethod
+    def _members(spec: BlockSpec):
+        members = [("norm", spec.mixer_norm, spec.mixer_norm_prefix), ("mixer", spec.mixer, spec.mixer_prefix)]
+        if spec.feed_forward is not None:
+            members.append(("feed_forward", spec.feed_forward, spec.feed_forward_prefix))
+        return members
+
+    @classmethod
+    def declare(cls, spec: BlockSpec) -> dict[str, TensorDecl]:
+        if spec.mixer_norm is None or spec.feed_forward_norm is not None:
+            raise ValueError("a parallel_stream block has one norm, the mixer's, for both of its sublayers")
+        out: dict[str, TensorDecl] = {}
+        for role, part, prefix in cls._members(spec):
+            for name, decl in part_class(role, part).declare(part).items():
+                out[prefix + name] = decl
+        return out
+
+    def __init__(self, spec: BlockSpec, tensors: dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.spec = spec
+        built = [part_class(role, part)(part, _sub(tensors, prefix), rt) for role, part, prefix in self._members(spec)]
+        self.mixer_norm, self.mixer = built[:2]
+        self.feed_forward = built[2] if spec.feed_forward is not None else None
+        self.feed_forward_norm = None
+
+    def forward(self, x, residual: torch.Tensor | None, ctx, binding, embedding: torch.Tensor | None = None,
+                embedding_scale: float = 1.0, embedding_position=None, embedding_norm=None, embedding_pairs=None):
+        from tinyserve_llm_b200.parts.norm import PendingBranch
+        if embedding is not None:
+            h, residual = self.mixer_norm.forward_embedded(embedding, x, embedding_scale, positions=ctx.positions,
+                                                           position=embedding_position, start_norm=embedding_norm,
+                                                           pairs=embedding_pairs, ctx=ctx)
+        else:
+            h, residual = self.mixer_norm.forward(x, residual)
+        mixed = self.mixer.forward(h, ctx, binding)
+        fed = self.feed_forward.forward(h, ctx) if self.feed_forward is not None else None
+        return PendingBranch.scaled_sum(mixed, fed, self.spec.branch_scale), residual

@@ -17,7 +17,9 @@ positions, counted from the request's first token, outside of which a query sees
 the last n keys, as for a window of n); scores capped as c tanh(score / c); a norm of every head of q and of k
 without a weight; values that are the keys as projected (no tensor `v`: the same columns of the
 projection go to the key pool normed and rotated and to the value pool as they are); a sink, a score
-without a key or a value in every softmax's sum.  With a distance penalty, a head bias, sigmoid weights, a gate
+without a key or a value in every softmax's sum; values mixed with those an earlier layer made of the same token,
+v <- (1 - vmix) v + vmix v_source (the source layer leaves its columns of the projection in the step's scratch; the
+kernel that stores the values mixes them).  With a distance penalty, a head bias, sigmoid weights, a gate
 a head, chunks, a cap or a sink the attention runs on the kernels that carry them (`paged_attention_split`'s options).
 
 Keys (rotated) and values live in the paged cache; one kernel norms, rotates and stores, one attends
@@ -36,6 +38,7 @@ from tinyserve_llm_b200.parts.base import KVNeed, Mixer, Runtime, TensorDecl, pa
 from tinyserve_llm_b200.parts.linear import Linear, fuse_rows
 
 MAX_HEAD_DIM = 256      # csrc/attention_generic.cu
+SOURCE_VALUES = "values mixed into later layers"     # key of the step's scratch: [T, kv heads * value dim]
 
 
 def kept_keys(window: int, chunk: int) -> int:
@@ -64,6 +67,8 @@ class GatedAttention(Mixer):
             raise NotImplementedError("attention: values that are the keys have no bias of their own")
         if spec.sink is not None and spec.weights != "softmax":
             raise NotImplementedError("attention: a sink belongs to the softmax")
+        if spec.value_mix not in ("none", "source", "mixed") or (spec.value_mix != "none" and spec.values != "projected"):
+            raise NotImplementedError(f"attention: value mixing {spec.value_mix!r} with values {spec.values!r}")
         if spec.weights not in ("softmax", "sigmoid"):
             raise NotImplementedError(f"attention: weights {spec.weights!r}; have softmax and sigmoid")
         if spec.q_temperature_every < 0 or spec.distance_slope_exponent < 0 or spec.window < 0 or spec.chunk < 0 or spec.softcap < 0:
@@ -86,6 +91,8 @@ class GatedAttention(Mixer):
                         "k.norm": TensorDecl((spec.head_dim if per_head else nk,), init="unit")})
         if spec.head_bias:
             out["pb"] = TensorDecl((spec.num_heads,))
+        if spec.value_mix == "mixed":
+            out["vmix"] = TensorDecl(())
         if spec.output_gate:
             out["g"] = TensorDecl((spec.num_heads if spec.output_gate_scope == "head" else no, spec.hidden_size))
         return out
@@ -101,6 +108,7 @@ class GatedAttention(Mixer):
         self.biases = tuple(tensors[n].to(**f32).contiguous() for n in ("q.b", "k.b", "v.b")) if spec.bias else None
         self.norm_weights = tuple(tensors[n].to(**f32).contiguous() for n in ("q.norm", "k.norm")) if spec.qk_norm and spec.qk_norm_weight else None
         self.head_bias = tensors["pb"].to(**f32).contiguous() if spec.head_bias else None
+        self.value_mix = float(tensors["vmix"]) if spec.value_mix == "mixed" else 0.0
         self.slopes = None
         if spec.distance_slope_exponent > 0:
             c, H = float(spec.distance_slope_exponent), spec.num_heads
@@ -129,10 +137,15 @@ class GatedAttention(Mixer):
         v_at = nq + nk
         if s.values == "keys":
             v_at, nv = nq, 0
+        mix = None
+        if s.value_mix == "source":
+            ctx.scratch[SOURCE_VALUES] = y[:, v_at:v_at + nv]
+        elif s.value_mix == "mixed":
+            mix = (ctx.scratch[SOURCE_VALUES], self.value_mix)
         q = ops.qk_norm_rope_store(y, (0, nq, v_at), self.biases, self.norm_weights, s.qk_norm_eps, self.position,
                                    ctx, binding, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim,
                                    norm_per_head=s.qk_norm_scope == "head", q_temperature=self.q_temperature,
-                                   unweighted_norm=s.qk_norm and not s.qk_norm_weight)
+                                   unweighted_norm=s.qk_norm and not s.qk_norm_weight, value_mix=mix)
         gate = y[:, nq + nk + nv:nq + nk + nv + self.gate_width] if s.output_gate else None
         per_head_gate = s.output_gate and s.output_gate_scope == "head"
         o = ops.paged_attention_split(q, ctx, binding, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, s.scale, s.window,

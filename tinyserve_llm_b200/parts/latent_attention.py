@@ -15,7 +15,10 @@ a window makes it a layer group of its own whose pages are given back as the win
 Options of the description: `q_rank` 0 makes the queries a projection of the input, q = W_q h, without a
 latent and a norm of their own; `rot_dim` 0 leaves out the rotated part (attention without positions: the
 cache row is c alone and no position part is built); `output_gate` multiplies the concatenated heads by
-sigmoid(W_g h), read from the same input as the other projections, before W_o.
+sigmoid(W_g h), read from the same input as the other projections, before W_o; `sink` adds exp(sink_h) to every
+softmax's sum of head h.  A rotation of neighbouring channels is a rotation by halves of channels put in another
+order: the rows of W_dkv and W_q that make the rotated parts are reordered when the part is built (a score is a sum
+over the channels, so the order does not show), and the kernels rotate by halves throughout.
 
 Prompt portions of a step that is launched once (not replayed from a CUDA graph) take another way where the
 sizes allow (bfloat16, no rotated part, key and value heads of one size the tcgen05 prompt kernel takes): the
@@ -24,7 +27,7 @@ for the step (K = C W_uk^T, V = C W_uv^T, two library products: a quarter of the
 a latent of 512 channels and heads of 128) and the tcgen05 prompt kernel attends over them; requests that feed
 one token in the same step stay on the folded form.  The two ways differ by rounding only.
 
-Tensors (local names): dq, dq.norm, uq (or q), dkv, dkv.norm, uk, uv, o, and g with an output gate.
+Tensors (local names): dq, dq.norm, uq (or q), dkv, dkv.norm, uk, uv, o, g with an output gate, sink.
 """
 
 from __future__ import annotations
@@ -37,6 +40,11 @@ from tinyserve_llm_b200.parts.linear import Linear, fuse_rows
 
 MAX_KV_RANK = 512       # csrc/attention_latent.cu: 16 output channels a lane
 MATERIALIZE_MIN_TOKENS = 128    # prompt portions of a step, together, from which keys and values are worked out for the step
+
+
+def evens_then_odds(rows: torch.Tensor) -> torch.Tensor:
+    """[..., 2n, columns] with rows 0, 2, 4, ... first, then 1, 3, 5, ...: neighbours become halves."""
+    return torch.cat([rows[..., 0::2, :], rows[..., 1::2, :]], dim=-2)
 
 
 @register_part("mixer", "latent_attention")
@@ -68,35 +76,44 @@ class LatentAttention(Mixer):
             out["q"] = TensorDecl((H * (D + R), spec.hidden_size))
         if spec.output_gate:
             out["g"] = TensorDecl((H * V, spec.hidden_size))
+        if spec.sink:
+            out["sink"] = TensorDecl((H,))
         return out
 
     def __init__(self, spec: LatentAttentionSpec, tensors: dict[str, torch.Tensor], rt: Runtime) -> None:
         super().__init__(spec, tensors, rt)
         self.validate(spec)
         H, D, V, rank = spec.num_heads, spec.head_dim, spec.value_dim, spec.kv_rank
+        R = spec.rot_dim
+        self.position = None
+        if spec.position is not None:
+            self.position = part_class("position", spec.position)(spec.position, {}, rt)
+            if getattr(self.position, "frequencies", None) is None or self.position.dims != R:
+                raise NotImplementedError("latent attention rotates inside its kernels: it takes a position part with "
+                                          "`frequencies` over exactly rot_dim channels")
+        self.frequencies = getattr(self.position, "frequencies", None)
+        self.magnitude = float(getattr(self.position, "magnitude", 1.0))
+        q_name = "uq" if spec.q_rank > 0 else "q"
+        q_rows, dkv_rows = tensors[q_name], tensors["dkv"]
+        if getattr(self.position, "interleaved", False):
+            by_head = q_rows.view(H, D + R, -1)
+            q_rows = torch.cat([by_head[:, :D], evens_then_odds(by_head[:, D:])], dim=1).reshape(q_rows.shape)
+            dkv_rows = torch.cat([dkv_rows[:rank], evens_then_odds(dkv_rows[rank:])], dim=0)
         # one product of the input: columns [c_q raw (or q) | c raw | k_rot raw | gate logits]
-        rows = [tensors["dq"] if spec.q_rank > 0 else tensors["q"], tensors["dkv"]] + ([tensors["g"]] if spec.output_gate else [])
+        rows = [tensors["dq"] if spec.q_rank > 0 else q_rows, dkv_rows] + ([tensors["g"]] if spec.output_gate else [])
         self.down = Linear(fuse_rows(rows), rt)
         self.q_norm = self.up_q = None
         if spec.q_rank > 0:
             self.q_norm = tensors["dq.norm"].to(device=rt.device, dtype=torch.float32).contiguous()
-            self.up_q = Linear(tensors["uq"], rt)
+            self.up_q = Linear(q_rows, rt)
         self.kv_norm = tensors["dkv.norm"].to(device=rt.device, dtype=torch.float32).contiguous()
         # W_uk per head, transposed to [H, rank, D]: the product that folds it into the query reads rows of D
         self.uk_t = tensors["uk"].to(device=rt.device, dtype=rt.dtype).view(H, D, rank).transpose(1, 2).contiguous()
         self.uv = tensors["uv"].to(device=rt.device, dtype=rt.dtype).view(H, V, rank).contiguous()
         # the unfolded form of prompt portions: W_uk as stored, [H D, rank] (W_uv's stored form is self.uv's memory)
-        self.uk = self.uk_t.transpose(1, 2).reshape(H * D, rank).contiguous() if spec.rot_dim == 0 and D == V else None
+        self.uk = self.uk_t.transpose(1, 2).reshape(H * D, rank).contiguous() if R == 0 and D == V and not spec.sink else None
         self.out = Linear(tensors["o"], rt)
-        self.position = self.frequencies = None
-        if spec.position is not None:
-            self.position = part_class("position", spec.position)(spec.position, {}, rt)
-            if getattr(self.position, "frequencies", None) is None or self.position.dims != spec.rot_dim:
-                raise NotImplementedError("latent attention rotates inside its kernels: it takes a position part with "
-                                          "`frequencies` over exactly rot_dim channels")
-            if getattr(self.position, "interleaved", False):
-                raise NotImplementedError("latent attention rotates by halves, not by neighbouring channels")
-            self.frequencies = self.position.frequencies
+        self.sink = tensors["sink"].to(device=rt.device, dtype=torch.float32).contiguous() if spec.sink else None
 
     def kv_need(self) -> KVNeed:
         return KVNeed(1, self.spec.kv_rank + self.spec.rot_dim, self.spec.window, values=False)
@@ -148,21 +165,21 @@ class LatentAttention(Mixer):
         if spec.q_rank > 0:
             latents = spec.q_rank + rank + R
             c_q = ops.latent_prepare(y[:, :latents], ctx, binding, spec.q_rank, rank, R, self.q_norm, self.kv_norm,
-                                     spec.norm_eps, self.frequencies)    # normed query latent; [c | k_rot] is in the cache
+                                     spec.norm_eps, self.frequencies, self.magnitude)   # normed query latent; [c | k_rot] is in the cache
             q = self.up_q(c_q)                                            # [T, H (D + R)]
         else:
             latents = H * (D + R) + rank + R
             q = y[:, :H * (D + R)]
             ops.latent_prepare(y[:, H * (D + R):latents], ctx, binding, 0, rank, R, None, self.kv_norm, spec.norm_eps,
-                               self.frequencies)
+                               self.frequencies, self.magnitude)
         portions = self._portions(q, ctx)
         if portions is not None and ctx.min_q_len > 1:
             o = self._attend_unfolded(q, ctx, binding, portions, None)
         else:
             folded_ctx = ctx if portions is None else self._single_tokens_only(ctx)
             q_lat = ops.per_head_linear(q, self.uk_t, H, D + R, D)        # float32 [T, H, rank]: W_uk^T q_flat
-            o_lat = ops.latent_attention(q_lat, q, folded_ctx, binding, H, D + R, D, rank, R, self.frequencies,
-                                         spec.scale, spec.window)         # [T, H, rank]: softmax-weighted sums of c
+            o_lat = ops.latent_attention(q_lat, q, folded_ctx, binding, H, D + R, D, rank, R, self.frequencies, spec.scale,
+                                         spec.window, magnitude=self.magnitude, sink=self.sink)   # [T, H, rank]: softmax-weighted sums of c
             o = ops.per_head_linear(o_lat.view(-1, H * rank), self.uv, H, rank, rank, out_dtype=x.dtype)   # [T, H, V]
             o = o.reshape(-1, H * V)
             if portions is not None:                                      # the portions' rows are written over

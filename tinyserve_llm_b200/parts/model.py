@@ -12,8 +12,9 @@ from __future__ import annotations
 import torch
 
 from tinyserve_llm_b200.config.spec import ModelSpec
-from tinyserve_llm_b200.parts import (attention, delta_rule, differential_attention, gated_attention, latent_attention,  # noqa: F401  (registration)
-                                      mingru, mlp, mlstm, norm, parallel, recurrence, rotary, routed_experts, time_mixing)
+from tinyserve_llm_b200.parts import (attention, delta_rule, differential_attention, embedding, gated_attention, gated_lru,  # noqa: F401  (registration)
+                                      latent_attention, mingru, mlp, mlstm, norm, parallel, recurrence, rotary, routed_experts,
+                                      time_mixing)
 from tinyserve_llm_b200.parts.base import KVNeed, Runtime, TensorDecl, arrangement_class, part_class
 from tinyserve_llm_b200.parts.block import _sub
 from tinyserve_llm_b200.parts.linear import Linear
@@ -32,6 +33,8 @@ def declared_tensors(spec: ModelSpec) -> dict[str, TensorDecl]:
     if spec.embedding_norm is not None:
         for name, decl in part_class("norm", spec.embedding_norm).declare(spec.embedding_norm).items():
             out[spec.embedding_norm_prefix + name] = decl
+    if spec.embedding_pairs is not None:
+        out.update(part_class("embedding", spec.embedding_pairs).declare(spec.embedding_pairs))
     return out
 
 
@@ -59,6 +62,9 @@ class DecoderModel:
         if spec.embedding_norm is not None:
             self.embedding_norm = part_class("norm", spec.embedding_norm)(
                 spec.embedding_norm, _sub(tensors, spec.embedding_norm_prefix), rt)
+        self.embedding_pairs = None              # with pairs, a step needs the token ahead of each request's first one
+        if spec.embedding_pairs is not None:
+            self.embedding_pairs = part_class("embedding", spec.embedding_pairs)(spec.embedding_pairs, tensors, rt)
         self._check_run_list()
         # A CUDA graph may replay the model only if no part runs host code that depends on the step.
         self.graph_safe = all(getattr(part, "graph_safe", False) for block in self.blocks
@@ -103,6 +109,8 @@ class DecoderModel:
             raise NotImplementedError("a position vector on the embedding needs a first block whose arrangement takes it")
         if self.embedding_norm is not None and not getattr(first, "takes_embedding_norm", False):
             raise NotImplementedError("a norm on the embedding needs a first block whose arrangement takes it")
+        if self.embedding_pairs is not None and not getattr(first, "takes_embedding_pairs", False):
+            raise NotImplementedError("an embedding of token pairs needs a first block whose arrangement takes it")
         if first is not None and getattr(first, "takes_token_ids", False) and (
                 scale == 1.0 or getattr(first, "takes_embedding_scale", False)):
             extra = {"embedding_scale": scale} if scale != 1.0 else {}
@@ -110,6 +118,8 @@ class DecoderModel:
                 extra["embedding_position"] = self.embedding_position
             if self.embedding_norm is not None:
                 extra["embedding_norm"] = self.embedding_norm
+            if self.embedding_pairs is not None:
+                extra["embedding_pairs"] = self.embedding_pairs
             x, residual = first.forward(ctx.token_ids, None, ctx, ctx.binding(run[0]), embedding=self.embedding, **extra)
             run = run[1:]
         elif scale != 1.0:

@@ -53,7 +53,12 @@ class PendingBranch:
     def __init__(self, tensor: torch.Tensor, closing: "StreamRMSNorm | None", pair: tuple | None = None) -> None:
         self.tensor = tensor
         self.closing = closing
-        self.pair = pair          # a sublayer of two normed branches: the second one and the norms (see `Ops.stream_norm`)
+        self.pair = pair          # a second branch, the two branches' norms and their scales (see `Ops.stream_norm`)
+
+    @classmethod
+    def scaled_sum(cls, tensor: torch.Tensor, other: torch.Tensor | None, scale: float) -> "PendingBranch":
+        """scale * (tensor + other), added to the stream without any norm (`other` None: scale * tensor)."""
+        return cls(tensor, None, None if other is None and scale == 1.0 else (other, None, None, scale, scale))
 
 
 @register_part("norm", "rmsnorm_stream")
@@ -84,7 +89,7 @@ class StreamRMSNorm(Norm):
         branch = closing = pair = None
         if isinstance(x, PendingBranch):
             branch, closing, pair = x.tensor, (x.closing.weight if x.closing is not None else None), x.pair
-            if pair is not None and self.centered:
+            if pair is not None and pair[1] is not None and self.centered:
                 raise NotImplementedError("the branches of a pair are RMS-normed")
         elif x is not None:
             raise ValueError("a stream norm takes a PendingBranch (a sublayer's output and its closing norm) or nothing")
@@ -110,10 +115,11 @@ class StreamRMSNorm(Norm):
         self.rt.ops.stream_norm(branch, self.weight, residual, None, self.eps, self.rt.dtype)
 
     def forward_embedded(self, table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0, positions: torch.Tensor | None = None,
-                         position=None, start_norm: "StreamRMSNorm | None" = None):
+                         position=None, start_norm: "StreamRMSNorm | None" = None, pairs=None, ctx=None):
         """
         `position` (a part with `frequencies`) and `positions`: its vector is added to the scaled rows.
         `start_norm` (a stream norm of this norm's kind and eps): the rows are normed by it before they start the stream.
+        `pairs` (a `PairEmbedding`) and the step's `ctx`: its rows by (previous token, token) are added to the scaled rows.
         """
         if start_norm is not None and (start_norm.centered != self.centered or start_norm.eps != self.eps):
             raise NotImplementedError("a norm on the embedding runs inside the first norm's kernel: both must be of one kind and eps")
@@ -121,7 +127,8 @@ class StreamRMSNorm(Norm):
         out = self.rt.ops.stream_norm(None, None, residual, self.weight, self.eps, self.rt.dtype, table=table, ids=ids,
                                       scale=scale, centered=self.centered, positions=positions,
                                       position_frequencies=position.frequencies if position is not None else None,
-                                      w_start=start_norm.weight if start_norm is not None else None)
+                                      w_start=start_norm.weight if start_norm is not None else None,
+                                      pairs=(pairs.table, pairs.spec, ctx) if pairs is not None else None)
         return out, residual
 
 
