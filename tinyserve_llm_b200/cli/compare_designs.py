@@ -1,9 +1,9 @@
 """
 Prefill and decode throughput of a design at layer sizes that resemble a real model's, beside the
 engine's closest other design at equal width and depth (Duduvik beside Llama, Nipizen beside
-Duduvik, Lugipel beside Nipizen, Folavik beside Llama, Fuvipel beside Nipizen), both with random weights through the engine's own step function:
+Duduvik, Lugipel beside Nipizen, Folavik beside Llama, Fuvipel beside Nipizen, Gimotar beside Lugipel and Duduvik), all with random weights through the engine's own step function:
 
-    python bench.py --design duduvik|nipizen|lugipel|folavik|fuvipel [--size small|medium|large] [--steps K] [--warmup W]
+    python bench.py --design duduvik|nipizen|lugipel|folavik|fuvipel|gimotar [--size small|medium|large] [--steps K] [--warmup W]
 
 For each design: a prompt of `prefill` tokens in one step (launched kernel by kernel), and decode
 steps of `batch` requests at `context` tokens each (replayed from a CUDA graph), timed on the device
@@ -137,6 +137,32 @@ def fuvipel_config(s: dict) -> dict:
     mixers = (rule, par, rule)
     return {"architecture": "Fuvipel", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6},
             "layers": [dict(mixers[i % 3], mlp=dense) for i in range(s["layers"])]}
+
+
+def gimotar_config(s: dict) -> dict:
+    """
+    Layers in the order chunked attention / Griffin's recurrent block / latent attention, every one with routed
+    experts (top 4) and a shared expert of the same kind and sizes as the Duduvik model's.  Attention heads of 128 channels,
+    4 query heads a key/value head, chunks of 1,024 tokens, rotation over half a head; the recurrence twice as wide as the
+    stream, as the Lugipel model's, its gates in parts of 256 channels; the latent layers sized as the Duduvik model's, over
+    every earlier key.
+    """
+    width, heads = s["width"], s["heads"]
+    dim = width // heads                                   # 128 at every size
+    att = {"type": "attention",
+           "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                     "mask": {"size": 1024}, "v_mix": True, "rot": {"base": 500000.0, "dims": dim // 2}}}
+    lru = {"type": "rglru", "mixer": {"width": 2 * width, "blocks": heads, "conv": 4}}
+    lat = {"type": "latent_attention",
+           "mixer": {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "kv_rank": 512, "scale": (dim + dim // 2) ** -0.5,
+                     "rot": {"base": 10000.0, "dims": dim // 2,
+                             "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    moe = {"kind": "moe", "router": {"experts": s["experts"], "top": 4}, "expert": {"ff": s["expert_ff"]},
+           "shared": {"ff": 2 * s["expert_ff"]}}
+    mixers = (att, lru, lat)
+    return {"architecture": "Gimotar", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 31337, "mul_cur": 17}},
+            "layers": [dict(mixers[i % 3], mlp=moe) for i in range(s["layers"])]}
 
 
 def llama_config(s: dict) -> dict:
@@ -274,8 +300,10 @@ def run(design: str, size: str, steps: int, warmup: int, peaks: dict) -> int:
         pair = (("llama", llama_config(s), True), ("folavik", folavik_config(s), True))
     elif design == "fuvipel":
         pair = (("nipizen", nipizen_config(s), True), ("fuvipel", fuvipel_config(s), True))
+    elif design == "gimotar":
+        pair = (("duduvik", duduvik_config(s), True), ("lugipel", lugipel_config(s), True), ("gimotar", gimotar_config(s), True))
     else:
-        raise SystemExit(f"--design {design!r}: have ['duduvik', 'nipizen', 'lugipel', 'folavik', 'fuvipel']")
+        raise SystemExit(f"--design {design!r}: have ['duduvik', 'nipizen', 'lugipel', 'folavik', 'fuvipel', 'gimotar']")
     for name, cfg, profile in pair:
         record = {"design": name, "size": size, "width": s["width"], "layers": s["layers"], "dtype": "bf16",
                   "data": "synthetic", "timing": "CUDA events, median, L2 flushed between timed steps", "peaks": peaks}
