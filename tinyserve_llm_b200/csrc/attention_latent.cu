@@ -265,7 +265,14 @@ latent_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, lo
     __syncthreads();
     for (int d = threadIdx.x; d < rank; d += blockDim.x) {
         float acc = 0.f;
-        for (int z = 0; z < splits; ++z) acc = fmaf(p[(long long)z * (rank + 2) + 2 + d], weight[z], acc);
+        for (int z = 0; z < splits; z += 8) {              // eight splits' loads under way together, added in order
+            float x[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[i] = p[(long long)min(z + i, splits - 1) * (rank + 2) + 2 + d];
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+                if (z + i < splits) acc = fmaf(x[i], weight[z + i], acc);
+        }
         out[item * rank + d] = from_float<T>(acc);
     }
 }
@@ -362,4 +369,45 @@ TS_API int ts_latent_attention(const float* q_lat, long long ql_token_stride, lo
                                             freq, magnitude, sink, k_pool, geo, block_table, table_width, positions, seq_of_token, out,
                                             num_tokens, heads, rank, rot, scale, window, split_keys, splits, scratch, stream);
     return ts_fail("latent_attention: unknown dtype code %d", dtype);
+}
+
+// The queries' rotated parts for the unfolded form: out[t, h, 0 .. pitch) = rotated q[t, h * head_width + rot_offset ..],
+// zeros past `rot` channels; rotation by halves, angle position * freq[i] in float32, cos and sin times `magnitude`.
+__global__ void latent_rotate_queries_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, int head_width,
+                                             int rot_offset, const float* __restrict__ freq, float magnitude,
+                                             const int* __restrict__ positions, __nv_bfloat16* __restrict__ out, int heads,
+                                             int rot, int pitch) {
+    extern __shared__ float turn[];                       // cos, sin of the token's rot / 2 angles
+    const int t = blockIdx.x, half = rot / 2;
+    const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, cs;
+        sincosf(pos * freq[i], &sn, &cs);
+        turn[i] = cs * magnitude;
+        turn[half + i] = sn * magnitude;
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < heads * pitch; e += blockDim.x) {
+        const int h = e / pitch, c = e % pitch;
+        float x = 0.f;
+        if (c < rot) {
+            const __nv_bfloat16* src = q + (long long)t * q_stride + (long long)h * head_width + rot_offset;
+            const int i = c < half ? c : c - half;
+            const float u = __bfloat162float(src[i]), v = __bfloat162float(src[i + half]);
+            x = c < half ? u * turn[i] - v * turn[half + i] : v * turn[i] + u * turn[half + i];
+        }
+        out[(long long)t * heads * pitch + e] = __float2bfloat16_rn(x);
+    }
+}
+
+TS_API int ts_latent_rotate_queries(const void* q, long long q_stride, int head_width, int rot_offset, const float* freq,
+                                    float magnitude, const int* positions, void* out, int num_tokens, int heads, int rot,
+                                    int pitch, cudaStream_t stream) {
+    TS_REQUIRE(num_tokens >= 0 && heads > 0 && rot > 0 && rot % 2 == 0 && rot <= pitch && rot_offset + rot <= head_width,
+               "latent_rotate_queries: bad sizes");
+    if (num_tokens == 0) return 0;
+    latent_rotate_queries_kernel<<<num_tokens, 256, rot * sizeof(float), stream>>>(
+        (const __nv_bfloat16*)q, q_stride, head_width, rot_offset, freq, magnitude, positions, (__nv_bfloat16*)out, heads, rot, pitch);
+    TS_LAUNCH_CHECK("latent_rotate_queries");
+    return 0;
 }

@@ -23,6 +23,9 @@
 // (attention/torch_paged.py:36-45 of the reference, by positions); value rows beyond the request's
 // length are zeroed in shared memory before they are multiplied.
 //
+// A form for keys of which every head has its own part and all heads share a second, rotated one (ROT): queries and keys
+// have a further sub-tile of 64 channels, the keys' read from a matrix of its own, once for all heads.
+//
 // Every mbarrier wait gives up after about two seconds and records where in an error word.
 #include <cuda.h>
 
@@ -31,18 +34,21 @@
 namespace {
 
 constexpr int QROWS = 128;                   // queries per CTA
-constexpr int TMEM_COLS = 256;
 // Sizes that follow from the head size.  A tile row of more than 64 dims lies in shared memory as
 // sub-tiles of 64 dims (128 bytes, the widest row the 128-byte swizzle takes), one after the other.
-template <int HD>
+// ROT (0 or 64): channels of the shared part of queries and keys, a sub-tile behind the others.
+template <int HD, int ROT = 0>
 struct Shape {
-    static constexpr int KEYS = HD == 64 ? 128 : 64;     // keys per tile: two CTAs must fit an SM
-    static constexpr int SUBS = HD / 64;                           // sub-tiles of 64 dims
+    static constexpr int KEYS = (HD == 64) == (ROT == 0) ? 128 : 64;     // keys per tile: two CTAs must fit an SM (HD 128 with ROT: one)
+    static constexpr int SUBS = HD / 64, QK_SUBS = (HD + ROT) / 64;      // sub-tiles of 64 dims: of values, of queries and keys
     static constexpr int SUB_Q = QROWS * 128, SUB_KV = KEYS * 128; // bytes of a sub-tile
-    static constexpr int Q_BYTES = QROWS * HD * 2, KV_BYTES = KEYS * HD * 2, STAGE_BYTES = 2 * KV_BYTES;
+    static constexpr int Q_BYTES = QK_SUBS * SUB_Q, K_BYTES = QK_SUBS * SUB_KV, STAGE_BYTES = K_BYTES + SUBS * SUB_KV;
     static constexpr int O_COL = KEYS;       // S at columns 0..KEYS-1, O after it, P (bfloat16 pairs) after O
     static constexpr int P_COL = KEYS + HD;
+    static constexpr int TMEM_COLS = P_COL + KEYS / 2 <= 256 ? 256 : 512;
+    static constexpr int CTAS = TMEM_COLS == 256 ? 2 : 1;                // on an SM
     static_assert(HD == 64 || HD == 128, "head sizes 64 and 128");
+    static_assert(ROT == 0 || ROT == 64, "one shared sub-tile or none");
     static_assert(P_COL + KEYS / 2 <= TMEM_COLS, "S, O and P must fit the allocation");
 };
 constexpr int SOFTMAX_WARPS = 8;             // two threads a query row: each takes half of the tile's keys and half of O's dims
@@ -219,6 +225,8 @@ struct FlashParams {
     float sink2;                      // a score (times log2(e)) that joins the softmax's sum without a key or a value; -inf: none
     // keys and values in matrices of their own instead of pages: [rows, nkv * HD], request s's key j in row kv_start[s] + j
     const int* kv_start;              // null: keys and values come from the paged pools
+    int q_head_cols;                  // columns of a head in q's rows (HD, and more where q holds other parts between the heads)
+    const float* sinks;               // [nh], not null: a sink a head, in place of sink2
 };
 
 // SIG: a visible key's weight is sigmoid(score * scale - slope (position - key) + bias): no maximum, no sum, no
@@ -226,15 +234,16 @@ struct FlashParams {
 // This form and BOUNDED take a window: the first key tile is the one that holds the first key the tile's first query sees.
 // BOUNDED: softmax as in the plain form; a row's keys begin at first_visible(position); capped scores go through
 // tanh in registers before the maximum is taken.
-template <int HD, int FORM>
-__global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
-                                                                        const __grid_constant__ CUtensorMap map_k,
-                                                                        const __grid_constant__ CUtensorMap map_v,
-                                                                        FlashParams p) {
-    using S_ = Shape<HD>;
+// ROT: map_q_rot [T, nh * 64] and map_k_rot [keys, <= 64] are the shared part of queries and keys (dense keys only).
+template <int HD, int FORM, int ROT>
+__global__ void __launch_bounds__(THREADS, (Shape<HD, ROT>::CTAS)) prefill_attention_tcgen05_kernel(
+        const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
+        const __grid_constant__ CUtensorMap map_q_rot, const __grid_constant__ CUtensorMap map_k_rot, FlashParams p) {
+    using S_ = Shape<HD, ROT>;
+    constexpr int TMEM_COLS = S_::TMEM_COLS;
     constexpr bool SIG = FORM == SIGMOID, LOW = FORM == BOUNDED;
     constexpr int KEYS = S_::KEYS, SUBS = S_::SUBS, SUB_Q = S_::SUB_Q, SUB_KV = S_::SUB_KV, Q_BYTES = S_::Q_BYTES,
-                  KV_BYTES = S_::KV_BYTES, STAGE_BYTES = S_::STAGE_BYTES, O_COL = S_::O_COL, P_COL = S_::P_COL;
+                  K_BYTES = S_::K_BYTES, STAGE_BYTES = S_::STAGE_BYTES, O_COL = S_::O_COL, P_COL = S_::P_COL;
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t q_full, kv_full[2], stage_free[2], s_done, p_ready, all_done;
     __shared__ uint32_t tmem_base_slot;
@@ -302,12 +311,13 @@ __global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(c
         // ---------------------------------------------------------------- TMA producer
         mbar_expect_tx(&q_full, Q_BYTES);
 #pragma unroll
-        for (int h = 0; h < SUBS; ++h) tma_load_2d(q_tile + h * SUB_Q, &map_q, &q_full, head * HD + h * 64, q_begin + row0);
+        for (int h = 0; h < SUBS; ++h) tma_load_2d(q_tile + h * SUB_Q, &map_q, &q_full, head * p.q_head_cols + h * 64, q_begin + row0);
+        if (ROT) tma_load_2d(q_tile + SUBS * SUB_Q, &map_q_rot, &q_full, head * 64, q_begin + row0);
         for (int j = kv_begin; j < num_kv; ++j) {
             const int it = j - kv_begin, s = it & 1;
             if (!mbar_wait(&stage_free[s], ((it >> 1) & 1) ^ 1, p.error, 11)) { failed = 1; break; }
             unsigned char* k_tile = kv_tiles + s * STAGE_BYTES;
-            unsigned char* v_tile = k_tile + KV_BYTES;
+            unsigned char* v_tile = k_tile + K_BYTES;
             mbar_expect_tx(&kv_full[s], STAGE_BYTES);
 #pragma unroll
             for (int b = 0; b < KEYS / 64; ++b) {    // boxes of 64 keys x 64 dims: a box never crosses a page
@@ -328,6 +338,7 @@ __global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(c
                     tma_load_2d(k_tile + h * SUB_KV + b * (64 * 128), &map_k, &kv_full[s], col + h * 64, row);
                     tma_load_2d(v_tile + h * SUB_KV + b * (64 * 128), &map_v, &kv_full[s], v_col + h * 64, v_row);
                 }
+                if (ROT) tma_load_2d(k_tile + SUBS * SUB_KV + b * (64 * 128), &map_k_rot, &kv_full[s], 0, row);
             }
         }
     } else if (warp == MMA_WARP && lane == 0) {
@@ -341,7 +352,7 @@ __global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(c
             if (!mbar_wait(&kv_full[s], (it >> 1) & 1, p.error, 13)) return false;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
-            for (int h = 0; h < SUBS; ++h) {
+            for (int h = 0; h < S_::QK_SUBS; ++h) {
                 const uint64_t q_desc = smem_desc(q_tile + h * SUB_Q);
                 const uint64_t k_desc = smem_desc(kv_tiles + s * STAGE_BYTES + h * SUB_KV);
 #pragma unroll
@@ -362,7 +373,7 @@ __global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(c
             if (j + 1 < num_it && !issue_scores(j + 1)) { ok = false; break; }
 #pragma unroll
             for (int h = 0; h < SUBS; ++h) {         // O += P V: 16 keys are 8 columns of packed P and 16 rows (2048 bytes) of a V sub-tile
-                const uint64_t v_desc = smem_desc(kv_tiles + s * STAGE_BYTES + KV_BYTES + h * SUB_KV);
+                const uint64_t v_desc = smem_desc(kv_tiles + s * STAGE_BYTES + K_BYTES + h * SUB_KV);
 #pragma unroll
                 for (int k = 0; k < KEYS / 16; ++k)
                     umma_ts(tmem + O_COL + 64 * h, tmem + P_COL + 8 * k, v_desc + 128 * k, idesc_o, (j | k) != 0);
@@ -445,7 +456,7 @@ __global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(c
                 if (half == 0 && r < KEYS && ((key0 + KEYS > ctx && key0 + r >= ctx) || key0 + r < first_seen)) {
 #pragma unroll
                     for (int h = 0; h < SUBS; ++h) {
-                        unsigned char* v_row = kv_tiles + s * STAGE_BYTES + KV_BYTES + h * SUB_KV + r * 128;
+                        unsigned char* v_row = kv_tiles + s * STAGE_BYTES + K_BYTES + h * SUB_KV + r * 128;
 #pragma unroll
                         for (int i = 0; i < 128; i += 16) *reinterpret_cast<uint4*>(v_row + i) = make_uint4(0, 0, 0, 0);
                     }
@@ -554,7 +565,7 @@ __global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(c
             if (half == 0 && r < KEYS && ((key0 + KEYS > ctx && key0 + r >= ctx) || (LOW && key0 + r < first_seen))) {
 #pragma unroll
                 for (int h = 0; h < SUBS; ++h) {
-                    unsigned char* v_row = kv_tiles + s * STAGE_BYTES + KV_BYTES + h * SUB_KV + r * 128;
+                    unsigned char* v_row = kv_tiles + s * STAGE_BYTES + K_BYTES + h * SUB_KV + r * 128;
 #pragma unroll
                     for (int i = 0; i < 128; i += 16) *reinterpret_cast<uint4*>(v_row + i) = make_uint4(0, 0, 0, 0);
                 }
@@ -573,7 +584,8 @@ __global__ void __launch_bounds__(THREADS, 2) prefill_attention_tcgen05_kernel(c
             half_sum[half][r] = l_run;
             pair_barrier(quadrant);
             l_run += half_sum[half ^ 1][r];
-            if (p.sink2 > -INFINITY) l_run += fast_exp2_any(p.sink2 - m_run);    // +inf where every score is far below it
+            const float sink2 = p.sinks ? p.sinks[head] * LOG2E : p.sink2;
+            if (sink2 > -INFINITY) l_run += fast_exp2_any(sink2 - m_run);    // +inf where every score is far below it
         }
         if (ok && !failed) {                         // every thread of the warp takes part in the loads; only real rows store
             float inv = l_run > 0.f ? 1.f / l_run : 0.f;
@@ -645,13 +657,24 @@ TS_API int ts_attention_tcgen05_supported(int hd, int page_tokens, int nh, int n
 
 namespace {
 
+// The part of queries and keys beside the heads' own: q_rot [T, nh * 64] (zeros past `rot` channels of a head), k_rot rows of
+// `rot` channels, k_rot_stride elements apart; sinks [nh] or null.
+struct SharedPart {
+    const void* q_rot;
+    const void* k_rot;
+    long long k_rot_stride;
+    int rot;                          // 0: no such part
+    int q_head_cols;
+    const float* sinks;
+};
+
 int run_prefill(const void* q, long long q_cols, long long q_stride, void* out, const void* k_pool, const void* v_pool,
                 int num_pages, int entries, int entry, int page_tokens, const int* block_table, int table_width,
                 const int* cu_q, const int* ctx_lens, int num_seqs, int num_tokens, int max_q_len, int nh, int nkv, int hd,
                 float scale, const int* prefill_seqs, int num_prefill_seqs, int* error, bool sigmoid, int window,
                 const float* slopes, const float* head_bias, const void* gate, long long gate_stride, cudaStream_t stream,
                 bool bounded = false, int chunk = 0, float softcap = 0.f, int value_heads = 0, const int* kv_start = nullptr,
-                long long dense_rows = 0, float sink = -INFINITY) {
+                long long dense_rows = 0, float sink = -INFINITY, const SharedPart* shared = nullptr) {
     TS_REQUIRE(ts_attention_tcgen05_supported(hd, page_tokens, nh, nkv, 0), "attention_tcgen05: sizes not taken (head_dim %d, page %d)", hd, page_tokens);
     TS_REQUIRE(sigmoid || bounded || window == 0, "attention_tcgen05: the plain form takes no window");
     TS_REQUIRE(window >= 0 && chunk >= 0 && softcap >= 0.f, "attention_tcgen05: a negative window, chunk or cap");
@@ -668,7 +691,7 @@ int run_prefill(const void* q, long long q_cols, long long q_stride, void* out, 
     if (prefill_seqs != nullptr && num_prefill_seqs == 0) return 0;
     const long long pool_rows = (long long)num_pages * entries * nkv * page_tokens;
     TS_REQUIRE(pool_rows < 0x7fffffffll, "attention_tcgen05: the pool has too many rows for 32-bit TMA coordinates");
-    CUtensorMap map_q, map_k, map_v;
+    CUtensorMap map_q, map_k, map_v, map_q_rot, map_k_rot;
     if (make_map(&map_q, q, num_tokens, q_cols, q_stride, QROWS)) return 1;
     if (kv_start != nullptr) {                           // matrices [dense_rows, heads * hd]
         TS_REQUIRE(dense_rows > 0 && dense_rows < 0x7fffffffll, "attention_tcgen05: %lld rows of keys", dense_rows);
@@ -678,7 +701,21 @@ int run_prefill(const void* q, long long q_cols, long long q_stride, void* out, 
         if (make_map(&map_k, k_pool, pool_rows, hd, hd, 64)) return 1;
         if (make_map(&map_v, v_pool, pool_rows / nkv * value_heads, hd, hd, 64)) return 1;
     }
+    const int rot = shared ? shared->rot : 0;
+    if (rot > 0) {
+        TS_REQUIRE(kv_start != nullptr && !sigmoid && !bounded, "attention_tcgen05: a shared key part comes with dense keys in the plain form");
+        TS_REQUIRE(rot <= 64 && rot % 8 == 0 && shared->q_head_cols % 8 == 0 && shared->k_rot_stride % 8 == 0 &&
+                   (uintptr_t)shared->q_rot % 16 == 0 && (uintptr_t)shared->k_rot % 16 == 0,
+                   "attention_tcgen05: a shared key part of %d channels, or its alignment", rot);
+        if (make_map(&map_q_rot, shared->q_rot, num_tokens, (long long)nh * 64, (long long)nh * 64, QROWS)) return 1;
+        if (make_map(&map_k_rot, shared->k_rot, dense_rows, rot, shared->k_rot_stride, 64)) return 1;
+    } else {
+        map_q_rot = map_q;                               // not read
+        map_k_rot = map_k;
+    }
     FlashParams p;
+    p.q_head_cols = shared ? shared->q_head_cols : hd;
+    p.sinks = shared ? shared->sinks : nullptr;
     p.out = (__nv_bfloat16*)out;
     p.block_table = block_table;
     p.table_width = table_width;
@@ -704,19 +741,22 @@ int run_prefill(const void* q, long long q_cols, long long q_stride, void* out, 
     p.gate = (const __nv_bfloat16*)gate;
     p.gate_stride = gate_stride;
     dim3 grid(nh, (max_q_len + QROWS - 1) / QROWS, prefill_seqs ? num_prefill_seqs : num_seqs);
-#define TS_FLASH_LAUNCH(HD, FORM)                                                                                         \
+#define TS_FLASH_LAUNCH(HD, FORM, ROT)                                                                                    \
     do {                                                                                                                  \
-        const size_t smem = (size_t)Shape<HD>::Q_BYTES + 2 * Shape<HD>::STAGE_BYTES + 1024;                               \
-        auto kernel = prefill_attention_tcgen05_kernel<HD, FORM>;                                                         \
+        const size_t smem = (size_t)Shape<HD, ROT>::Q_BYTES + 2 * Shape<HD, ROT>::STAGE_BYTES + 1024;                     \
+        auto kernel = prefill_attention_tcgen05_kernel<HD, FORM, ROT>;                                                    \
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                             \
-        TS_CHAINED_CHECK("attention_tcgen05", launch_chained(kernel, grid, dim3(THREADS), smem, stream, map_q, map_k, map_v, p)); \
+        TS_CHAINED_CHECK("attention_tcgen05", launch_chained(kernel, grid, dim3(THREADS), smem, stream, map_q, map_k, map_v, \
+                                                             map_q_rot, map_k_rot, p));                                   \
     } while (0)
-    if (hd == 64 && sigmoid) TS_FLASH_LAUNCH(64, SIGMOID);
-    else if (hd == 64 && bounded) TS_FLASH_LAUNCH(64, BOUNDED);
-    else if (hd == 64) TS_FLASH_LAUNCH(64, PLAIN);
-    else if (sigmoid) TS_FLASH_LAUNCH(128, SIGMOID);
-    else if (bounded) TS_FLASH_LAUNCH(128, BOUNDED);
-    else TS_FLASH_LAUNCH(128, PLAIN);
+    if (hd == 64 && rot > 0) TS_FLASH_LAUNCH(64, PLAIN, 64);
+    else if (rot > 0) TS_FLASH_LAUNCH(128, PLAIN, 64);
+    else if (hd == 64 && sigmoid) TS_FLASH_LAUNCH(64, SIGMOID, 0);
+    else if (hd == 64 && bounded) TS_FLASH_LAUNCH(64, BOUNDED, 0);
+    else if (hd == 64) TS_FLASH_LAUNCH(64, PLAIN, 0);
+    else if (sigmoid) TS_FLASH_LAUNCH(128, SIGMOID, 0);
+    else if (bounded) TS_FLASH_LAUNCH(128, BOUNDED, 0);
+    else TS_FLASH_LAUNCH(128, PLAIN, 0);
 #undef TS_FLASH_LAUNCH
     return 0;
 }
@@ -776,14 +816,20 @@ TS_API int ts_prefill_attention_tcgen05_masked(const void* q, long long q_stride
 // Causal softmax attention of prompt portions over keys and values that lie in matrices of their own,
 // k [kv_rows, nkv * hd] and v [kv_rows, nkv * hd] (bfloat16, rows back to back), request s's key j in row kv_start[s] + j
 // (kv_start: int32 [num_seqs] on the device; ctx_lens[s] keys a request).  For keys and values that are worked out
-// for the step instead of read from pages.  Queries [T, nh * hd] in a matrix of their own, q_stride elements a row.
+// for the step instead of read from pages.  Queries [T, q_stride] in a matrix of their own, head h's hd columns from
+// h * q_head_cols on.  With `rot` > 0 a score also has q_rot . k_rot, q_rot [T, nh * 64] (a head's channels past `rot` zero)
+// and k_rot one row of `rot` channels a key for all heads, k_rot_stride elements apart, in the same row order as k.
+// `sinks` [nh] (null: none): a score a head that joins every softmax's sum without a key or a value.
 TS_API int ts_prefill_attention_tcgen05_dense(const void* q, long long q_stride, void* out, const void* k, const void* v,
                                               long long kv_rows, const int* kv_start, const int* cu_q, const int* ctx_lens,
                                               int num_seqs, int num_tokens, int max_q_len, int nh, int nkv, int hd,
                                               float scale, const int* prefill_seqs, int num_prefill_seqs, int* error,
-                                              cudaStream_t stream) {
+                                              int q_head_cols, const void* q_rot, const void* k_rot, long long k_rot_stride, int rot,
+                                              const float* sinks, cudaStream_t stream) {
     TS_REQUIRE(kv_start != nullptr, "attention_tcgen05: the first rows of the requests' keys are needed");
-    return run_prefill(q, (long long)nh * hd, q_stride, out, k, v, 1, 1, 0, 64, nullptr, 1, cu_q, ctx_lens, num_seqs, num_tokens,
+    TS_REQUIRE(q_head_cols >= hd && (rot == 0 || (q_rot && k_rot)), "attention_tcgen05: the queries' columns, or the shared key part");
+    const SharedPart shared{q_rot, k_rot, k_rot_stride, rot, q_head_cols, sinks};
+    return run_prefill(q, (long long)nh * q_head_cols, q_stride, out, k, v, 1, 1, 0, 64, nullptr, 1, cu_q, ctx_lens, num_seqs, num_tokens,
                        max_q_len, nh, nkv, hd, scale, prefill_seqs, num_prefill_seqs, error, false, 0, nullptr, nullptr,
-                       nullptr, 0, stream, false, 0, 0.f, 0, kv_start, kv_rows);
+                       nullptr, 0, stream, false, 0, 0.f, 0, kv_start, kv_rows, -INFINITY, &shared);
 }

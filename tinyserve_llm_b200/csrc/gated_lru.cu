@@ -12,7 +12,7 @@
 // floats each.  The ring has an entry more than the convolution looks back, so the entry that a decoded token
 // writes is one that no thread of that launch reads.
 //
-// lru_conv_kernel            u of every row of the step (a thread eight channels and a few tokens, a rolling window).
+// lru_conv_kernel            u of every row of the step.
 // lru_scan_kernel            requests of up to LRU_STRETCH tokens: a thread a (request, channel), tokens in order.
 // lru_stretch_kernel,        longer portions: stretches of LRU_STRETCH tokens side by side; the first kernel turns the
 // lru_finish_kernel          gates' logits into (a, sqrt(1 - a^2) i u) in place and each stretch into one step
@@ -78,77 +78,106 @@ __device__ __forceinline__ void lru_advance_ring(const LRUArgs& p, float* ring, 
         ring[(long long)(p.positions[t] % p.taps) * p.channels + c] = lru_value<T>(p, t, c);
 }
 
-template <typename T, int VEC, int TAPS>
-__global__ void __launch_bounds__(128) lru_conv_kernel(LRUArgs p, int group) {
+template <int N>
+__device__ __forceinline__ void load_floats(const float* src, float (&dst)[N]) {     // 16-byte aligned where N is a multiple of 4
+    if (N % 4 == 0)
+#pragma unroll
+        for (int i = 0; i < N; i += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(src + i);
+            dst[i] = v.x; dst[(i + 1) % N] = v.y; dst[(i + 2) % N] = v.z; dst[(i + 3) % N] = v.w;
+        }
+    else
+#pragma unroll
+        for (int i = 0; i < N; ++i) dst[i] = src[i];
+}
+
+constexpr int LRU_GROUP = 8;             // tokens a thread of the convolution takes in a step of many tokens
+
+// A thread: 16 bytes of neighbouring channels, GROUP tokens whose rows are asked for together, a window that rolls over them.
+template <typename T, int TAPS, int GROUP>
+__global__ void __launch_bounds__(128) lru_conv_kernel(LRUArgs p) {
+    constexpr int VEC = 16 / sizeof(T);
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
     if (c >= p.channels) return;
-    const int taps = TAPS > 0 ? TAPS : p.taps;
-    const int t_begin = blockIdx.y * group, t_end = min(p.num_tokens, t_begin + group);
-    T* u = (T*)p.u;
-    if (TAPS > 0) {
-        constexpr int K = TAPS > 0 ? TAPS : 1;
-        float w[K][VEC], bias[VEC], xb[VEC], win[K][VEC];
+    const int t_begin = blockIdx.y * GROUP, count = min(GROUP, p.num_tokens - t_begin);
+    const T* x = (const T*)p.xy + p.x_off + c;
+    uint4 rows[GROUP];
+    int seqs[GROUP];
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) {
-            bias[i] = p.conv_bias[c + i];
-            xb[i] = p.x_bias[c + i];
-#pragma unroll
-            for (int j = 0; j < K; ++j) w[j][i] = p.taps_w[(long long)j * p.channels + c + i];
-        }
-        int current = -2;
-        for (int t = t_begin; t < t_end; ++t) {
-            const int seq = p.seq_of_token[t];
-            T* dst = u + (long long)t * p.channels + c;
-            alignas(16) T o[VEC];
-            if (seq < 0) {                                       // a padding row
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) o[i] = from_float<T>(0.f);
-            } else {
-                if (seq != current) {                            // the values before this row
-                    const int begin = p.cu_q[seq], slot = p.state_slots[seq], pos = p.positions[t];
-                    const float* ring = slot >= 0 ? p.state + (long long)slot * p.state_stride : nullptr;
-#pragma unroll
-                    for (int j = 0; j < K - 1; ++j)
-#pragma unroll
-                        for (int i = 0; i < VEC; ++i) win[j + 1][i] = lru_earlier<T>(p, t, begin, pos, ring, K - 1 - j, c + i);
-                    current = seq;
-                }
-                alignas(16) T x[VEC];
-                const T* src = (const T*)p.xy + (long long)t * p.xy_stride + p.x_off + c;
-                if (VEC * sizeof(T) == 16) *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(src);
-                else
-#pragma unroll
-                    for (int i = 0; i < VEC; ++i) x[i] = src[i];
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) {
-#pragma unroll
-                    for (int j = 0; j < K - 1; ++j) win[j][i] = win[j + 1][i];
-                    win[K - 1][i] = to_float<T>(x[i]) + xb[i];
-                    float acc = bias[i];
-#pragma unroll
-                    for (int j = 0; j < K; ++j) acc = fmaf(w[j][i], win[j][i], acc);
-                    o[i] = from_float<T>(acc);
-                }
-            }
-            if (VEC * sizeof(T) == 16) *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(o);
-            else
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) dst[i] = o[i];
-        }
-    } else {                                                     // any number of taps, a channel a thread
-        for (int t = t_begin; t < t_end; ++t) {
-            const int seq = p.seq_of_token[t];
-            float acc = 0.f;
-            if (seq >= 0) {
-                const int begin = p.cu_q[seq], slot = p.state_slots[seq], pos = p.positions[t];
-                const float* ring = slot >= 0 ? p.state + (long long)slot * p.state_stride : nullptr;
-                acc = p.conv_bias[c];
-                for (int j = 0; j < taps; ++j)
-                    acc = fmaf(p.taps_w[(long long)j * p.channels + c], lru_earlier<T>(p, t, begin, pos, ring, taps - 1 - j, c), acc);
-            }
-            u[(long long)t * p.channels + c] = from_float<T>(acc);
+    for (int g = 0; g < GROUP; ++g) {
+        rows[g] = make_uint4(0, 0, 0, 0);
+        seqs[g] = -1;
+        if (g < count) {
+            rows[g] = *reinterpret_cast<const uint4*>(x + (long long)(t_begin + g) * p.xy_stride);
+            seqs[g] = p.seq_of_token[t_begin + g];
         }
     }
+    float w[TAPS][VEC], bias[VEC], xb[VEC], win[TAPS][VEC];
+    load_floats(p.conv_bias + c, bias);
+    load_floats(p.x_bias + c, xb);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load_floats(p.taps_w + (long long)j * p.channels + c, w[j]);
+    auto values = [&](const uint4& raw, float (&v)[VEC]) {
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = to_float<T>(e[i]) + xb[i];
+    };
+    int current = -2;
+#pragma unroll
+    for (int g = 0; g < GROUP; ++g) {
+        if (g >= count) break;
+        const int t = t_begin + g, seq = seqs[g];
+        alignas(16) T o[VEC];
+        if (seq < 0) {                                           // a padding row
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) o[i] = from_float<T>(0.f);
+        } else {
+            if (seq != current) {                                // the values before this row: of the batch, of the ring, or zeros
+                const int begin = p.cu_q[seq], slot = p.state_slots[seq], pos = p.positions[t];
+                const float* ring = p.state + (long long)max(slot, 0) * p.state_stride + c;
+#pragma unroll
+                for (int back = TAPS - 1; back > 0; --back) {
+                    float (&v)[VEC] = win[TAPS - back];          // moves one place down before it is used
+                    if (t - back >= begin) values(*reinterpret_cast<const uint4*>(x + (long long)(t - back) * p.xy_stride), v);
+                    else if (slot >= 0 && pos - back >= 0) load_floats(ring + (long long)((pos - back) % TAPS) * p.channels, v);
+                    else
+#pragma unroll
+                        for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+                }
+                current = seq;
+            }
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) win[j][i] = win[j + 1][i];
+            values(rows[g], win[TAPS - 1]);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) {
+                float acc = bias[i];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j][i], win[j][i], acc);
+                o[i] = from_float<T>(acc);
+            }
+        }
+        *reinterpret_cast<uint4*>((T*)p.u + (long long)t * p.channels + c) = *reinterpret_cast<const uint4*>(o);
+    }
+}
+
+// Any sizes: a thread a channel and token.
+template <typename T>
+__global__ void __launch_bounds__(128) lru_conv_any_kernel(LRUArgs p) {
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, t = blockIdx.y;
+    if (c >= p.channels) return;
+    const int seq = p.seq_of_token[t];
+    float acc = 0.f;
+    if (seq >= 0) {
+        const int begin = p.cu_q[seq], slot = p.state_slots[seq], pos = p.positions[t];
+        const float* ring = slot >= 0 ? p.state + (long long)slot * p.state_stride : nullptr;
+        acc = p.conv_bias[c];
+        for (int j = 0; j < p.taps; ++j)
+            acc = fmaf(p.taps_w[(long long)j * p.channels + c], lru_earlier<T>(p, t, begin, pos, ring, p.taps - 1 - j, c), acc);
+    }
+    ((T*)p.u)[(long long)t * p.channels + c] = from_float<T>(acc);
 }
 
 constexpr int LRU_AHEAD = 4;
@@ -305,7 +334,10 @@ __device__ __forceinline__ void lru_mma(float (&c)[4], unsigned a0, unsigned a1,
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-template <int CHUNKS>        // stretches of 32 k's a warp holds: part <= 128 CHUNKS
+// What the kernel does not get from the projection just ahead (weights, index data, the slot's ring and state, which earlier
+// steps left) is asked for before it waits for that kernel.
+// CHUNKS: stretches of 32 k's a warp holds, part <= 128 CHUNKS; TAPS 0: any number of them, loaded as they are used.
+template <int CHUNKS, int TAPS>
 __global__ void __launch_bounds__(LD_THREADS) lru_decode_kernel(LRUArgs p, const __nv_bfloat16* __restrict__ gates_w) {
     extern __shared__ __align__(16) unsigned char lru_smem[];
     const int part = p.part, pitch = part + 8;
@@ -328,31 +360,84 @@ __global__ void __launch_bounds__(LD_THREADS) lru_decode_kernel(LRUArgs p, const
             fi[j] = *reinterpret_cast<const uint4*>(wr + (long long)part * part + k);
         }
     }
-    chain_wait();
-    // ---- u of the part, eight channels of a token an item
-    const int vecs = part / 8;
-    for (int e = tid; e < padded * vecs; e += LD_THREADS) {
-        const int t = e / vecs, c0 = (e % vecs) * 8, c = b * part + c0;
+    const int state_at = p.taps > 1 ? p.taps * p.channels : 0;
+    // this thread's eight channels of u, and the tokens it takes them of
+    const int vecs = part / 8, per_pass = LD_THREADS / vecs;
+    const int c0 = (tid % vecs) * 8, c = b * part + c0, first = tid / vecs < per_pass ? tid / vecs : padded;
+    constexpr int K = TAPS > 0 ? TAPS : 1;
+    float w[K][8], bias[8], xb[8], past[K][8];
+    load_floats(p.conv_bias + c, bias);
+    load_floats(p.x_bias + c, xb);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load_floats(p.taps_w + (long long)j * p.channels + c, w[j]);
+    auto slot_of = [&](int t) {
         const int seq = t < p.num_tokens ? p.seq_of_token[t] : -1;
-        const int slot = seq >= 0 ? p.state_slots[seq] : -1;
+        return seq >= 0 ? p.state_slots[seq] : -1;
+    };
+    auto load_past = [&](int pos, const float* ring) {           // the token `back` before: entry TAPS - 1 - back
+#pragma unroll
+        for (int back = 1; back < TAPS; ++back) {
+            if (back <= pos) load_floats(ring + (long long)((pos - back) % K) * p.channels + c, past[K - 1 - back < 0 ? 0 : K - 1 - back]);
+            else
+#pragma unroll
+                for (int i = 0; i < 8; ++i) past[K - 1 - back < 0 ? 0 : K - 1 - back][i] = 0.f;
+        }
+    };
+    int slot = slot_of(first), pos = slot >= 0 ? p.positions[first] : 0;
+    if (slot >= 0) load_past(pos, p.state + (long long)slot * p.state_stride);
+    // this thread's first (token, channel) of the last part
+    const int mine_t = tid / LD_CHANNELS, mine_n = n0 + tid % LD_CHANNELS;
+    const bool channel = mine_n < part;
+    const int mc = b * part + (channel ? mine_n : n0);
+    const int mine_slot = slot_of(mine_t);
+    const float rb = p.gate_bias[mc], ib = p.gate_bias[p.channels + mc], rate = p.rate[mc], yb = p.y_bias[mc], mxb = p.x_bias[mc];
+    float mine_S = mine_slot >= 0 ? p.state[(long long)mine_slot * p.state_stride + state_at + mc] : 0.f;
+    chain_wait();
+    const __nv_bfloat16* xy = (const __nv_bfloat16*)p.xy;
+    float mine_y = 0.f, mine_x = 0.f;
+    if (mine_slot >= 0) {
+        mine_y = __bfloat162float(xy[(long long)mine_t * p.xy_stride + p.y_off + mc]);
+        mine_x = __bfloat162float(xy[(long long)mine_t * p.xy_stride + p.x_off + mc]);
+    }
+    // ---- u of the part
+    for (int t = first; t < padded; t += per_pass) {
         alignas(16) __nv_bfloat16 o[8];
+        if (t != first) {
+            slot = slot_of(t);
+            if (slot >= 0) {
+                pos = p.positions[t];
+                load_past(pos, p.state + (long long)slot * p.state_stride);
+            }
+        }
         if (slot < 0) {
 #pragma unroll
             for (int i = 0; i < 8; ++i) o[i] = __float2bfloat16_rn(0.f);
         } else {
-            const int pos = p.positions[t];
-            const float* ring = p.state + (long long)slot * p.state_stride;
             alignas(16) __nv_bfloat16 x[8];
-            *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.xy + (long long)t * p.xy_stride + p.x_off + c);
+            *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(xy + (long long)t * p.xy_stride + p.x_off + c);
             float acc[8];
-            const float* w = p.taps_w + (long long)(p.taps - 1) * p.channels + c;
+            if (TAPS > 0) {
 #pragma unroll
-            for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[i], __bfloat162float(x[i]) + p.x_bias[c + i], p.conv_bias[c + i]);
-            for (int back = 1; back < p.taps && back <= pos; ++back) {
-                const float* v = ring + (long long)((pos - back) % p.taps) * p.channels + c;
-                w = p.taps_w + (long long)(p.taps - 1 - back) * p.channels + c;
+                for (int i = 0; i < 8; ++i) {
+                    acc[i] = bias[i];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[i], v[i], acc[i]);
+                    for (int j = 0; j < K - 1; ++j) acc[i] = fmaf(w[j][i], past[j][i], acc[i]);
+                    acc[i] = fmaf(w[K - 1][i], __bfloat162float(x[i]) + xb[i], acc[i]);
+                }
+            } else {
+                const float* ring = p.state + (long long)slot * p.state_stride;
+                float wt[8], v[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) acc[i] = bias[i];
+                for (int back = min(p.taps - 1, pos); back > 0; --back) {
+                    load_floats(p.taps_w + (long long)(p.taps - 1 - back) * p.channels + c, wt);
+                    load_floats(ring + (long long)((pos - back) % p.taps) * p.channels + c, v);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) acc[i] = fmaf(wt[i], v[i], acc[i]);
+                }
+                load_floats(p.taps_w + (long long)(p.taps - 1) * p.channels + c, wt);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) acc[i] = fmaf(wt[i], __bfloat162float(x[i]) + xb[i], acc[i]);
             }
 #pragma unroll
             for (int i = 0; i < 8; ++i) o[i] = __float2bfloat16_rn(acc[i]);
@@ -378,31 +463,33 @@ __global__ void __launch_bounds__(LD_THREADS) lru_decode_kernel(LRUArgs p, const
     }
     __syncthreads();
     chain_release();
-    for (int e = tid; e < p.num_tokens * LD_CHANNELS; e += LD_THREADS) {
-        const int t = e / LD_CHANNELS, ch = e % LD_CHANNELS;
-        const int seq = p.seq_of_token[t];
-        if (seq < 0 || n0 + ch >= part) continue;
-        const int slot = p.state_slots[seq];
+    if (!channel) return;
+    for (int t = mine_t; t < p.num_tokens; t += LD_THREADS / LD_CHANNELS) {
+        if (t != mine_t) {
+            slot = slot_of(t);
+            if (slot >= 0) {
+                mine_S = p.state[(long long)slot * p.state_stride + state_at + mc];
+                mine_y = __bfloat162float(xy[(long long)t * p.xy_stride + p.y_off + mc]);
+                mine_x = __bfloat162float(xy[(long long)t * p.xy_stride + p.x_off + mc]);
+            }
+        } else {
+            slot = mine_slot;
+        }
         if (slot < 0) continue;
-        float zr = 0.f, zi = 0.f;
+        float zr = rb, zi = ib;
 #pragma unroll
         for (int s = 0; s < LD_SPLITS; ++s) {
-            const float2 v = zs[((long long)s * padded + t) * LD_CHANNELS + ch];
+            const float2 v = zs[((long long)s * padded + t) * LD_CHANNELS + tid % LD_CHANNELS];
             zr += v.x;
             zi += v.y;
         }
-        const int c = b * part + n0 + ch;
-        const __nv_bfloat16* row = (const __nv_bfloat16*)p.xy + (long long)t * p.xy_stride;
         float* ring = p.state + (long long)slot * p.state_stride;
-        float* sp = ring + (p.taps > 1 ? (long long)p.taps * p.channels : 0) + c;
         float a, in;
-        lru_gates<true>(zr + p.gate_bias[c], zi + p.gate_bias[p.channels + c], p.rate[c],
-                        __bfloat162float(us[t * pitch + n0 + ch]), a, in);
-        const float S = fmaf(a, *sp, in);
-        *sp = S;
-        if (p.taps > 1) ring[(long long)(p.positions[t] % p.taps) * p.channels + c] = __bfloat162float(row[p.x_off + c]) + p.x_bias[c];
-        ((__nv_bfloat16*)p.out)[(long long)t * p.channels + c] =
-            __float2bfloat16_rn(S * lru_gelu(__bfloat162float(row[p.y_off + c]) + p.y_bias[c]));
+        lru_gates<true>(zr, zi, rate, __bfloat162float(us[t * pitch + mine_n]), a, in);
+        const float S = fmaf(a, mine_S, in);
+        ring[state_at + mc] = S;
+        if (p.taps > 1) ring[(long long)(p.positions[t] % p.taps) * p.channels + mc] = mine_x + mxb;
+        ((__nv_bfloat16*)p.out)[(long long)t * p.channels + mc] = __float2bfloat16_rn(S * lru_gelu(mine_y + yb));
     }
 }
 
@@ -437,19 +524,28 @@ TS_API int ts_lru_decode(TS_LRU_PARAMS, const void* gates_w, cudaStream_t stream
     if (lru_check(p)) return 1;
     if (num_tokens == 0 || num_seqs == 0) return 0;
     TS_REQUIRE(ts_lru_decode_supported(num_tokens, channels, part, xy_stride, x_off) && (uintptr_t)xy % 16 == 0 &&
-               (uintptr_t)gates_w % 16 == 0, "lru_decode: sizes not taken");
+               (uintptr_t)gates_w % 16 == 0 && (uintptr_t)state % 16 == 0 && state_stride % 4 == 0,
+               "lru_decode: sizes or alignment not taken");
     const size_t smem = lru_decode_smem(num_tokens, part);
     const dim3 grid((channels / part) * ((part + LD_CHANNELS - 1) / LD_CHANNELS));
     const __nv_bfloat16* w = (const __nv_bfloat16*)gates_w;
-#define TS_LRU_DECODE(CHUNKS)                                                                                             \
+#define TS_LRU_DECODE(CHUNKS, TAPS)                                                                                       \
     do {                                                                                                                  \
         if (smem > 48 * 1024)                                                                                             \
-            cudaFuncSetAttribute(lru_decode_kernel<CHUNKS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);      \
-        TS_CHAINED_CHECK("lru_decode", launch_chained(lru_decode_kernel<CHUNKS>, grid, dim3(LD_THREADS), smem, stream, p, w)); \
+            cudaFuncSetAttribute(lru_decode_kernel<CHUNKS, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        TS_CHAINED_CHECK("lru_decode", launch_chained(lru_decode_kernel<CHUNKS, TAPS>, grid, dim3(LD_THREADS), smem, stream, p, w)); \
     } while (0)
-    if (part <= 128) TS_LRU_DECODE(1);
-    else if (part <= 256) TS_LRU_DECODE(2);
-    else TS_LRU_DECODE(4);
+#define TS_LRU_DECODE_PART(TAPS)                    \
+    do {                                            \
+        if (part <= 128) TS_LRU_DECODE(1, TAPS);      \
+        else if (part <= 256) TS_LRU_DECODE(2, TAPS); \
+        else TS_LRU_DECODE(4, TAPS);                  \
+    } while (0)
+    if (taps == 4) TS_LRU_DECODE_PART(4);
+    else if (taps == 3) TS_LRU_DECODE_PART(3);
+    else if (taps == 2) TS_LRU_DECODE_PART(2);
+    else TS_LRU_DECODE_PART(0);
+#undef TS_LRU_DECODE_PART
 #undef TS_LRU_DECODE
     return 0;
 }
@@ -457,15 +553,19 @@ TS_API int ts_lru_decode(TS_LRU_PARAMS, const void* gates_w, cudaStream_t stream
 template <typename T>
 static int lru_conv_launch(const LRUArgs& p, cudaStream_t stream) {
     constexpr int VEC = 16 / sizeof(T);
-    const bool vector = p.channels % VEC == 0 && p.xy_stride % VEC == 0 && p.x_off % VEC == 0 && (uintptr_t)p.xy % 16 == 0 &&
-                        (uintptr_t)p.u % 16 == 0;
-    const int group = p.num_tokens >= 256 ? 8 : 1;
-    TS_REQUIRE(p.num_tokens <= 65535 * group, "gated_lru: %d tokens a step are not supported", p.num_tokens);
-    const int per_thread = vector && p.taps <= 8 ? VEC : 1;
-    const int threads = (p.channels + per_thread - 1) / per_thread;
-    const dim3 grid((threads + 127) / 128, (p.num_tokens + group - 1) / group);
-#define TS_LRU_CONV(K) lru_conv_kernel<T, VEC, K><<<grid, 128, 0, stream>>>(p, group)
-    if (per_thread == 1) lru_conv_kernel<T, 1, 0><<<grid, 128, 0, stream>>>(p, group);
+    const bool vector = p.channels % 8 == 0 && p.xy_stride % VEC == 0 && p.x_off % VEC == 0 && (uintptr_t)p.xy % 16 == 0 &&
+                        (uintptr_t)p.u % 16 == 0 && (uintptr_t)p.state % 16 == 0 && p.state_stride % 4 == 0 && p.taps <= 8;
+    const bool many = p.num_tokens >= 256;
+    const int rows = vector && many ? (p.num_tokens + LRU_GROUP - 1) / LRU_GROUP : p.num_tokens;
+    TS_REQUIRE(rows <= 65535, "gated_lru: %d tokens a step are not supported", p.num_tokens);
+    const int threads = vector ? p.channels / VEC : p.channels;
+    const dim3 grid((threads + 127) / 128, rows);
+#define TS_LRU_CONV(K)                                                                     \
+    do {                                                                                   \
+        if (many) lru_conv_kernel<T, K, LRU_GROUP><<<grid, 128, 0, stream>>>(p);           \
+        else lru_conv_kernel<T, K, 1><<<grid, 128, 0, stream>>>(p);                        \
+    } while (0)
+    if (!vector) lru_conv_any_kernel<T><<<grid, 128, 0, stream>>>(p);
     else switch (p.taps) {
         case 1: TS_LRU_CONV(1); break;
         case 2: TS_LRU_CONV(2); break;

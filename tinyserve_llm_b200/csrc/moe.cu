@@ -21,7 +21,8 @@
 //                    stores relu(s)^2 and `row_scale` (one factor a pair) multiplies the sum first: an
 //                    expert whose input is weighted, since W (c x) = c (W x).  Input rows are
 //                    gathered by token for the first product; the second reads the sorted rows.
-//                    A step of up to 64 pairs takes a weight-streaming kernel instead (further down); large
+//                    A step of few pairs takes a weight-streaming kernel instead (further down: bfloat16 up to 256
+//                    pairs on mma.sync, float32 up to 64); large
 //                    bfloat16 steps may be given to the library's grouped product by the caller.
 //   ts_moe_combine   out[t] = sum_j share[t, j] * y[row of (t, j)] (+ the shared expert's output), in the
 //                    order of j, float32, rounded once.  Without `share` every weight is 1.  With
@@ -344,6 +345,35 @@ moe_linear_kernel(const T* __restrict__ x, long long x_stride, const int* __rest
 // lane at a time, for all rows of the tile at once.  A row's sum over k has one order, whatever the batch.
 constexpr int SR = 8, SWARPS = 8;
 
+// Which expert's stretch row tile `tile` belongs to (tiles of SR rows, numbered expert by expert); `experts`: none.  On
+// return `tile` counts from the expert's first one, its stretch is [first, last).  Every warp looks at 32
+// experts at a time, a lane an expert, and a scan over the lanes' tile counts finds the one; walking the
+// offsets one dependent load after the other cost the last experts' CTAs some thousand cycles before their first byte.
+__device__ __forceinline__ int expert_of_tile(const int* __restrict__ offsets, int experts, int& tile, int& first, int& last) {
+    const int ln = threadIdx.x & 31;
+    for (int e0 = 0; e0 < experts; e0 += 32) {
+        const int le = e0 + ln;
+        const int f = le < experts ? offsets[le] : 0, l = le < experts ? offsets[le + 1] : 0;
+        const int tiles = le < experts ? (l - f + SR - 1) / SR : 0;
+        int incl = tiles;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int v = __shfl_up_sync(0xffffffffu, incl, o);
+            if (ln >= o) incl += v;
+        }
+        const unsigned hit = __ballot_sync(0xffffffffu, tile < incl);
+        if (hit) {
+            const int src = __ffs(hit) - 1;
+            first = __shfl_sync(0xffffffffu, f, src);
+            last = __shfl_sync(0xffffffffu, l, src);
+            tile -= __shfl_sync(0xffffffffu, incl - tiles, src);
+            return e0 + src;
+        }
+        tile -= __shfl_sync(0xffffffffu, incl, 31);
+    }
+    return experts;
+}
+
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(SWARPS * 32)
 moe_linear_rows_kernel(const T* __restrict__ x, long long x_stride, const int* __restrict__ pair_of_row, int top,
@@ -354,34 +384,8 @@ moe_linear_rows_kernel(const T* __restrict__ x, long long x_stride, const int* _
     __shared__ float rows_scale[SR];
     T* xs = reinterpret_cast<T*>(raw);                    // [SR][K]
     constexpr int VN = 16 / sizeof(T);
-    // Which expert's stretch this row tile belongs to (tiles are numbered expert by expert): every warp looks at 32
-    // experts at a time, a lane an expert, and a scan over the lanes' tile counts finds the one; walking the
-    // offsets one dependent load after the other cost the last experts' CTAs some thousand cycles before their first byte.
-    int tile = blockIdx.y, e = experts, first = 0, last = 0;
-    {
-        const int ln = threadIdx.x & 31;
-        for (int e0 = 0; e0 < experts; e0 += 32) {
-            const int le = e0 + ln;
-            const int f = le < experts ? offsets[le] : 0, l = le < experts ? offsets[le + 1] : 0;
-            const int tiles = le < experts ? (l - f + SR - 1) / SR : 0;
-            int incl = tiles;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const int v = __shfl_up_sync(0xffffffffu, incl, o);
-                if (ln >= o) incl += v;
-            }
-            const unsigned hit = __ballot_sync(0xffffffffu, tile < incl);
-            if (hit) {
-                const int src = __ffs(hit) - 1;
-                e = e0 + src;
-                first = __shfl_sync(0xffffffffu, f, src);
-                last = __shfl_sync(0xffffffffu, l, src);
-                tile -= __shfl_sync(0xffffffffu, incl - tiles, src);
-                break;
-            }
-            tile -= __shfl_sync(0xffffffffu, incl, 31);
-        }
-    }
+    int tile = blockIdx.y, first = 0, last = 0;
+    const int e = expert_of_tile(offsets, experts, tile, first, last);
     if (e == experts) return;
     const int row0 = first + tile * SR;
     const int nrows = min(SR, last - row0);
@@ -460,6 +464,86 @@ moe_linear_rows_kernel(const T* __restrict__ x, long long x_stride, const int* _
     }
 }
 
+// The bfloat16 form: 16 weight rows (gated: 8 gate rows, then the same 8 up rows) times up to 8 pairs of one expert as
+// m16n8k16 products, a warp's 16 rows streamed once from global memory straight into fragments.  The k's of a product
+// may come in any order as long as both operands agree, so lane q of a row takes k's 8q .. 8q + 7 of every 32: one 16-byte
+// load a row for two products.  MR_AHEAD stretches of 32 k's are under way at once; the pairs' rows of x come the same way
+// (they stay in L1).  No shared memory, no barrier: a CTA is MR_WARPS warps that work alone.
+constexpr int MR_WARPS = 4, MR_AHEAD = 8;
+
+__device__ __forceinline__ void moe_mma(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3, unsigned b0, unsigned b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+__device__ __forceinline__ uint4 load_streamed(const __nv_bfloat16* p) {      // read once: not kept in L1
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+
+template <bool GATED>
+__global__ void __launch_bounds__(MR_WARPS * 32)
+moe_linear_rows_mma_kernel(const __nv_bfloat16* __restrict__ x, long long x_stride, const int* __restrict__ pair_of_row, int top,
+                           const int* __restrict__ offsets, int experts, const __nv_bfloat16* __restrict__ w, int N, int K,
+                           __nv_bfloat16* __restrict__ y, int out_cols, int kind, float limit, float alpha,
+                           const float* __restrict__ row_scale, int unary) {
+    int tile = blockIdx.y, first = 0, last = 0;
+    const int e = expert_of_tile(offsets, experts, tile, first, last);
+    if (e == experts) return;
+    constexpr int COLS = GATED ? 8 : 16;                  // output columns a warp
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, q = lane & 3, g = lane >> 2;
+    const int col0 = (blockIdx.x * MR_WARPS + warp) * COLS;
+    if (col0 >= out_cols) return;
+    const int row0 = first + tile * SR, nrows = min(SR, last - row0);
+    const __nv_bfloat16* we = w + (long long)e * N * K;
+    // rows past the last column: the last one again, not stored
+    const __nv_bfloat16* wa = we + (long long)min(col0 + g, out_cols - 1) * K + q * 8;
+    const __nv_bfloat16* wb = GATED ? we + (long long)(N / 2 + min(col0 + g, out_cols - 1)) * K + q * 8
+                                    : we + (long long)min(col0 + 8 + g, out_cols - 1) * K + q * 8;
+    const bool have = g < nrows;
+    const int src = have ? (pair_of_row ? pair_of_row[row0 + g] / top : row0 + g) : 0;
+    const __nv_bfloat16* xr = x + (long long)src * x_stride + q * 8;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int k0 = 0; k0 < K; k0 += 32 * MR_AHEAD) {
+        uint4 a[MR_AHEAD], b[MR_AHEAD], v[MR_AHEAD];
+#pragma unroll
+        for (int j = 0; j < MR_AHEAD; ++j) {
+            const int k = k0 + 32 * j;
+            a[j] = b[j] = v[j] = make_uint4(0, 0, 0, 0);
+            if (k + q * 8 < K) {
+                a[j] = load_streamed(wa + k);
+                b[j] = load_streamed(wb + k);
+                if (have) v[j] = *reinterpret_cast<const uint4*>(xr + k);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < MR_AHEAD; ++j) {
+            moe_mma(acc, a[j].x, b[j].x, a[j].y, b[j].y, v[j].x, v[j].y);
+            moe_mma(acc, a[j].z, b[j].z, a[j].w, b[j].w, v[j].z, v[j].w);
+        }
+    }
+    // weight rows g (acc 0, 1) and g + 8 (acc 2, 3); pairs 2q and 2q + 1
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int r = 2 * q + i;
+        if (r >= nrows) break;
+        __nv_bfloat16* dst = y + (long long)(row0 + r) * out_cols + col0 + g;
+        if (GATED) {
+            if (col0 + g < out_cols) *dst = __float2bfloat16_rn(ts_gated_activation(kind, acc[i], acc[i + 2], limit, alpha));
+            continue;
+        }
+        const float scale = row_scale ? row_scale[pair_of_row ? pair_of_row[row0 + r] : row0 + r] : 1.f;
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            float s = acc[i + 2 * h] * scale;
+            if (unary == 1) s = fmaxf(s, 0.f) * fmaxf(s, 0.f);
+            if (col0 + g + 8 * h < out_cols) dst[8 * h] = __float2bfloat16_rn(s);
+        }
+    }
+}
+
 TS_API int ts_moe_linear(const void* x, long long x_stride, const int* pair_of_row, int top, const int* offsets,
                          int experts, const void* w, int N, int K, void* y, int pairs, int gated, int kind, float limit,
                          float alpha, const float* row_scale, int unary, int dtype, cudaStream_t stream) {
@@ -469,6 +553,21 @@ TS_API int ts_moe_linear(const void* x, long long x_stride, const int* pair_of_r
     if (pairs <= 0) return 0;
     const int out_cols = gated ? N / 2 : N;
     const int elem = dtype == TS_F32 ? 4 : 2, vn = 16 / elem;
+    if (dtype == TS_BF16 && pairs <= 256 && K % 8 == 0 && x_stride % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0) {
+        const int tiles = (pairs + SR - 1) / SR + experts;
+        const int cols = MR_WARPS * (gated ? 8 : 16);
+        TS_REQUIRE(tiles <= 65535, "moe_linear: too many row tiles");
+        const dim3 grid((out_cols + cols - 1) / cols, tiles);
+#define TS_MOE_ROWS_MMA(G)                                                                                                  \
+        moe_linear_rows_mma_kernel<G><<<grid, MR_WARPS * 32, 0, stream>>>(                                                  \
+            (const __nv_bfloat16*)x, x_stride, pair_of_row, top, offsets, experts, (const __nv_bfloat16*)w, N, K,           \
+            (__nv_bfloat16*)y, out_cols, kind, limit, alpha, row_scale, unary)
+        if (gated) TS_MOE_ROWS_MMA(true);
+        else TS_MOE_ROWS_MMA(false);
+#undef TS_MOE_ROWS_MMA
+        TS_LAUNCH_CHECK("moe_linear (rows, mma)");
+        return 0;
+    }
     if (pairs <= 64 && K % vn == 0 && (x_stride * elem) % 16 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
         (size_t)SR * K * elem <= 200 * 1024 && (dtype == TS_F32 || dtype == TS_BF16)) {
         const int tiles = (pairs + SR - 1) / SR + experts;
@@ -505,6 +604,47 @@ TS_API int ts_moe_linear(const void* x, long long x_stride, const int* pair_of_r
     return 0;
 }
 
+// Rows of a multiple of 16 bytes: a thread 16 bytes of neighbouring channels, four choices' rows asked for together.
+template <typename T>
+__global__ void moe_combine_vec_kernel(const T* __restrict__ y, const int* __restrict__ row_of_pair,
+                                       const float* __restrict__ share, const T* __restrict__ shared_out, T* __restrict__ out,
+                                       int width, int top, const T* __restrict__ x, const float* __restrict__ identity_share) {
+    constexpr int VEC = 16 / sizeof(T);
+    const long long t = blockIdx.x;
+    auto add = [](float (&s)[VEC], float w, const uint4& raw) {
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s[i] = fmaf(w, to_float<T>(e[i]), s[i]);
+    };
+    for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {
+        float s[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s[i] = 0.f;
+        uint4 extra = make_uint4(0, 0, 0, 0), own = make_uint4(0, 0, 0, 0);
+        if (shared_out) extra = *reinterpret_cast<const uint4*>(shared_out + t * width + c);
+        if (identity_share) own = *reinterpret_cast<const uint4*>(x + t * width + c);
+        for (int j0 = 0; j0 < top; j0 += 4) {
+            uint4 raw[4];
+            float w[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int row = j0 + j < top ? row_of_pair[t * top + j0 + j] : -1;
+                w[j] = row < 0 ? 0.f : share ? share[t * top + j0 + j] : 1.f;
+                raw[j] = make_uint4(0, 0, 0, 0);
+                if (row >= 0) raw[j] = *reinterpret_cast<const uint4*>(y + (long long)row * width + c);
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) add(s, w[j], raw[j]);
+        }
+        if (shared_out) add(s, 1.f, extra);
+        if (identity_share) add(s, identity_share[t], own);
+        alignas(16) T o[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) o[i] = from_float<T>(s[i]);
+        *reinterpret_cast<uint4*>(out + t * width + c) = *reinterpret_cast<const uint4*>(o);
+    }
+}
+
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ row_of_pair,
                                    const float* __restrict__ share, const T* __restrict__ shared_out, T* __restrict__ out,
@@ -527,6 +667,19 @@ TS_API int ts_moe_combine(const void* y, const int* row_of_pair, const float* sh
                           cudaStream_t stream) {
     TS_REQUIRE(!identity_share || x, "moe_combine: identity experts need the experts' input");
     if (num_tokens <= 0) return 0;
+    const int vec = dtype == TS_F32 ? 4 : 8;
+    const uintptr_t all = (uintptr_t)y | (uintptr_t)shared_out | (uintptr_t)out | (identity_share ? (uintptr_t)x : 0);
+    if (width % vec == 0 && all % 16 == 0 && (dtype == TS_F32 || dtype == TS_BF16)) {
+        const int threads = min(256, (width / vec + 31) / 32 * 32);
+        if (dtype == TS_F32)
+            moe_combine_vec_kernel<float><<<num_tokens, threads, 0, stream>>>((const float*)y, row_of_pair, share,
+                (const float*)shared_out, (float*)out, width, top, (const float*)x, identity_share);
+        else
+            moe_combine_vec_kernel<__nv_bfloat16><<<num_tokens, threads, 0, stream>>>((const __nv_bfloat16*)y, row_of_pair, share,
+                (const __nv_bfloat16*)shared_out, (__nv_bfloat16*)out, width, top, (const __nv_bfloat16*)x, identity_share);
+        TS_LAUNCH_CHECK("moe_combine");
+        return 0;
+    }
     if (dtype == TS_F32)
         moe_combine_kernel<float><<<num_tokens, 128, 0, stream>>>((const float*)y, row_of_pair, share,
                                                                   (const float*)shared_out, (float*)out, width, top,

@@ -33,7 +33,8 @@ _SIGNATURES = {
     "ts_paged_attention_bf16_sigmoid": ("int", "pl" "ppp" "lliipippiiiiiiifiplpi" "pppl" "p"),
     "ts_paged_attention_bf16_masked": ("int", "pl" "ppp" "lllliipippiiiiiiifiifi" "plpi" "fp"),
     "ts_attention_tcgen05_supported": ("int", "iiiii"),
-    "ts_prefill_attention_tcgen05_dense": ("int", "pl" "ppp" "lpppiiiiiifpipp"),
+    "ts_prefill_attention_tcgen05_dense": ("int", "pl" "ppp" "lpppiiiiiifpip" "ipplip" "p"),
+    "ts_latent_rotate_queries": ("int", "pliipfppiiiip"),
     "ts_prefill_attention_tcgen05_masked": ("int", "pl" "ppp" "iiiipippiiiiiifiifi" "pipfp"),
     "ts_prefill_attention_tcgen05": ("int", "ppppiiiipippiiiiiifpipp"),
     "ts_prefill_attention_tcgen05_sigmoid": ("int", "pl" "ppp" "iiiipippiiiiiifi" "pppl" "pipp"),
@@ -825,29 +826,58 @@ class Ops:
                     and self.lib.ts_attention_tcgen05_supported(hd, 64, nh, nkv, 0))
 
     def dense_prompt_attention(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, kv_start: torch.Tensor, ctx, nh: int,
-                               nkv: int, hd: int, scale: float, out: torch.Tensor | None = None) -> torch.Tensor:
+                               nkv: int, hd: int, scale: float, out: torch.Tensor | None = None, *, q_head_cols: int = 0,
+                               shared: tuple[torch.Tensor, torch.Tensor] | None = None, sink: torch.Tensor | None = None) -> torch.Tensor:
         """
         Causal softmax attention of the step's prompt portions (requests that feed more than one token) over keys
         and values worked out for the step: k, v [rows, nkv * hd] bfloat16, request s's key j in row kv_start[s] + j
         (int32 [requests] on the device), ctx.ctx_lens[s] keys a request.  Rows of requests that feed one token are
         left as they are in `out` ([T, nh * hd]; made here if not given).  The tcgen05 prompt kernel.
+
+        `q_head_cols` (0: hd): columns of a head in q's rows, its first hd being the ones that meet k.  `shared` (q_rot
+        [T, nh * 64], k_rot [rows, rot <= 64]): a score also has q_rot . k_rot, k_rot being the same for all heads and
+        q_rot's channels past rot zero.  `sink` (float32 [nh]): exp(sink[h]) joins every softmax's sum of head h.
         """
+        q_head_cols = q_head_cols or hd
         self._check_rows(q, "q")
         self._check(k, "k", torch.bfloat16, 2)
         self._check(v, "v", torch.bfloat16, 2)
         self._check(kv_start, "kv_start", torch.int32, 1)
-        if k.shape != v.shape or k.shape[1] != nkv * hd or q.shape[1] != nh * hd or kv_start.shape[0] != ctx.ctx_lens.shape[0]:
+        if k.shape != v.shape or k.shape[1] != nkv * hd or q.shape[1] != nh * q_head_cols or kv_start.shape[0] != ctx.ctx_lens.shape[0]:
             raise KernelError(f"dense_prompt_attention: q {tuple(q.shape)}, k {tuple(k.shape)}, v {tuple(v.shape)} for "
                               f"{nh}:{nkv} heads of {hd}")
         if not self.dense_prompt_attention_supported(q, nh, nkv, hd):
             raise KernelError(f"dense_prompt_attention: sizes not taken ({nh}:{nkv} heads of {hd}, {q.dtype})")
+        q_rot = k_rot = None
+        if shared is not None:
+            q_rot, k_rot = shared
+            self._check(q_rot, "q_rot", torch.bfloat16, 2)
+            self._check_rows(k_rot, "k_rot")
+            if tuple(q_rot.shape) != (q.shape[0], nh * 64) or k_rot.shape[0] != k.shape[0] or k_rot.shape[1] > 64 or k_rot.dtype != torch.bfloat16:
+                raise KernelError(f"dense_prompt_attention: a shared part of {tuple(q_rot.shape)} and {tuple(k_rot.shape)}")
+        if sink is not None:
+            self._check(sink, "sink", torch.float32, 1)
+            if sink.shape[0] != nh:
+                raise KernelError(f"dense_prompt_attention: {sink.shape[0]} sinks for {nh} heads")
         if out is None:
             out = torch.empty((q.shape[0], nh * hd), dtype=q.dtype, device=q.device)
         prefill_seqs = getattr(ctx, "prefill_seqs", None)
         num_prefill = prefill_seqs.shape[0] if prefill_seqs is not None else 0
         self._call("ts_prefill_attention_tcgen05_dense", _ptr(q), q.stride(0), _ptr(out), _ptr(k), _ptr(v), k.shape[0],
                    _ptr(kv_start), _ptr(ctx.cu_q), _ptr(ctx.ctx_lens), ctx.ctx_lens.shape[0], q.shape[0], ctx.max_q_len, nh, nkv,
-                   hd, scale, _ptr(prefill_seqs), num_prefill, self.error_word().data_ptr(), _stream())
+                   hd, scale, _ptr(prefill_seqs), num_prefill, self.error_word().data_ptr(), q_head_cols, _ptr(q_rot), _ptr(k_rot),
+                   k_rot.stride(0) if k_rot is not None else 0, k_rot.shape[1] if k_rot is not None else 0, _ptr(sink), _stream())
+        return out
+
+    def latent_rotate_queries(self, q: torch.Tensor, ctx, heads: int, head_width: int, rot_offset: int, rot: int,
+                              freq: torch.Tensor, magnitude: float) -> torch.Tensor:
+        """bfloat16 [T, heads * 64]: every head's `rot` channels of q from `rot_offset` on, rotated by halves, zeros behind them."""
+        self._check_rows(q, "q")
+        if q.dtype != torch.bfloat16 or q.shape[1] != heads * head_width or not 0 < rot <= 64:
+            raise KernelError(f"latent_rotate_queries: q {tuple(q.shape)} {q.dtype}, {heads} heads of {head_width}, rotation over {rot}")
+        out = torch.empty((q.shape[0], heads * 64), dtype=q.dtype, device=q.device)
+        self._call("ts_latent_rotate_queries", _ptr(q), q.stride(0), head_width, rot_offset, _ptr(freq), float(magnitude),
+                   _ptr(ctx.positions), _ptr(out), q.shape[0], heads, rot, 64, _stream())
         return out
 
     def tensor_core_attention(self, q: torch.Tensor, binding, nh: int, nkv: int, hd: int, vd: int, ctx=None) -> bool:

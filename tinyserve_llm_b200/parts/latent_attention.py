@@ -21,9 +21,9 @@ order: the rows of W_dkv and W_q that make the rotated parts are reordered when 
 over the channels, so the order does not show), and the kernels rotate by halves throughout.
 
 Prompt portions of a step that is launched once (not replayed from a CUDA graph) take another way where the
-sizes allow (bfloat16, no rotated part, key and value heads of one size the tcgen05 prompt kernel takes): the
-latents of the requests' whole contexts are gathered from the pages, a head's keys and values are worked out
-for the step (K = C W_uk^T, V = C W_uv^T, two library products: a quarter of the folded form's arithmetic at
+sizes allow (bfloat16, key and value heads of one size the tcgen05 prompt kernel takes, up to 64 rotated channels): the
+latents of the requests' whole contexts are gathered from the pages (their rotated parts, one for all heads, go to the
+kernel as they lie), a head's keys and values are worked out for the step (K = C W_uk^T, V = C W_uv^T, two library products: a quarter of the folded form's arithmetic at
 a latent of 512 channels and heads of 128) and the tcgen05 prompt kernel attends over them; requests that feed
 one token in the same step stay on the folded form.  The two ways differ by rounding only.
 
@@ -111,7 +111,8 @@ class LatentAttention(Mixer):
         self.uk_t = tensors["uk"].to(device=rt.device, dtype=rt.dtype).view(H, D, rank).transpose(1, 2).contiguous()
         self.uv = tensors["uv"].to(device=rt.device, dtype=rt.dtype).view(H, V, rank).contiguous()
         # the unfolded form of prompt portions: W_uk as stored, [H D, rank] (W_uv's stored form is self.uv's memory)
-        self.uk = self.uk_t.transpose(1, 2).reshape(H * D, rank).contiguous() if R == 0 and D == V and not spec.sink else None
+        # (rotated parts go to the kernel as TMA sub-tiles of 64 channels out of rows [c | k_rot]: 16-byte boundaries)
+        self.uk = self.uk_t.transpose(1, 2).reshape(H * D, rank).contiguous() if D == V and R <= 64 and R % 8 == 0 and (R == 0 or rank % 8 == 0) else None
         self.out = Linear(tensors["o"], rt)
         self.sink = tensors["sink"].to(device=rt.device, dtype=torch.float32).contiguous() if spec.sink else None
 
@@ -143,20 +144,26 @@ class LatentAttention(Mixer):
 
     def _attend_unfolded(self, q: torch.Tensor, ctx, binding, portions: list[int], out: torch.Tensor | None) -> torch.Tensor:
         spec, ops, host = self.spec, self.rt.ops, ctx.host
-        H, D, rank, B = spec.num_heads, spec.head_dim, spec.kv_rank, binding.page_tokens
-        entries = binding.page_stride // (B * rank)
-        pool = binding.k_pool.view(binding.num_pages, entries, B, rank)[:, binding.entry_offset // (B * rank)]
+        H, D, R, rank, B = spec.num_heads, spec.head_dim, spec.rot_dim, spec.kv_rank, binding.page_tokens
+        width = rank + R
+        entries = binding.page_stride // (B * width)
+        pool = binding.k_pool.view(binding.num_pages, entries, B, width)[:, binding.entry_offset // (B * width)]
         starts, latents, at = [0] * len(host.ctx_lens), [], 0
         for s in portions:                                  # the latents of the whole context, page by page
             n = host.ctx_lens[s]
             pages = binding.block_table[s, :-(-n // B)].long()
-            latents.append(pool[pages].reshape(-1, rank)[:n])
+            latents.append(pool[pages].reshape(-1, width)[:n])
             starts[s], at = at, at + n
-        c = torch.cat(latents) if len(latents) > 1 else latents[0].contiguous()
+        rows = torch.cat(latents) if len(latents) > 1 else latents[0].contiguous()
+        c, shared = rows, None
+        if R:
+            c = rows[:, :rank].contiguous()
+            shared = ops.latent_rotate_queries(q, ctx, H, D + R, D, R, self.frequencies, self.magnitude), rows[:, rank:]
         kv_start = torch.tensor(starts, dtype=torch.int32).to(q.device, non_blocking=True)
         k = ops.linear(c, self.uk)                          # [keys, H D]
         v = ops.linear(c, self.uv.view(H * spec.value_dim, rank))
-        return ops.dense_prompt_attention(q, k, v, kv_start, ctx, H, H, D, spec.scale, out)
+        return ops.dense_prompt_attention(q, k, v, kv_start, ctx, H, H, D, spec.scale, out, q_head_cols=D + R, shared=shared,
+                                          sink=self.sink)
 
     def forward(self, x: torch.Tensor, ctx, binding) -> torch.Tensor:
         spec, ops = self.spec, self.rt.ops
