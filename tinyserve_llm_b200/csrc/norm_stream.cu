@@ -176,6 +176,89 @@ __global__ void stream_norm_kernel(const T* __restrict__ branch, const float* __
     for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_float<T>((row[i] - mean) * inv * w_open[i]);
 }
 
+// The commonest case, a branch (or two, each times its scale) added as it is and the sum normed, for rows of a multiple of 16
+// bytes of the branch's type: a thread VEC neighbouring columns, up to STREAM_ITEMS times, the row in registers.
+constexpr int STREAM_ITEMS = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+stream_add_norm_kernel(const T* __restrict__ branch, const T* __restrict__ branch2, float scale, float scale2, float* stream,
+                       const float* __restrict__ w_open, T* __restrict__ out, const int* __restrict__ rows, int width, float eps,
+                       int write_stream, int centered) {
+    constexpr int VEC = 16 / sizeof(T);
+    __shared__ float scratch[64];
+    const int r = blockIdx.x;
+    const int src = rows ? rows[r] : r;
+    if (src < 0) return;                          // a padding row
+    float* sr = stream + (long long)src * width;
+    float x[STREAM_ITEMS][VEC];
+    float sum = 0.f, sq = 0.f;
+#pragma unroll
+    for (int m = 0; m < STREAM_ITEMS; ++m) {
+        const int c = (m * blockDim.x + threadIdx.x) * VEC;
+        if (c >= width) break;
+        const uint4 raw = *reinterpret_cast<const uint4*>(branch + (long long)src * width + c);
+        uint4 raw2 = make_uint4(0, 0, 0, 0);
+        if (branch2) raw2 = *reinterpret_cast<const uint4*>(branch2 + (long long)src * width + c);
+        const T* e = reinterpret_cast<const T*>(&raw);
+        const T* e2 = reinterpret_cast<const T*>(&raw2);
+#pragma unroll
+        for (int i = 0; i < VEC; i += 4) {
+            const float4 s = *reinterpret_cast<const float4*>(sr + c + i);
+            x[m][i] = s.x; x[m][i + 1] = s.y; x[m][i + 2] = s.z; x[m][i + 3] = s.w;
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            const float b = branch2 ? scale * to_float<T>(e[i]) + scale2 * to_float<T>(e2[i]) : scale * to_float<T>(e[i]);
+            x[m][i] += b;
+            sum += x[m][i];
+            sq += x[m][i] * x[m][i];
+        }
+        if (write_stream)
+#pragma unroll
+            for (int i = 0; i < VEC; i += 4)
+                *reinterpret_cast<float4*>(sr + c + i) = make_float4(x[m][i], x[m][i + 1], x[m][i + 2], x[m][i + 3]);
+    }
+    float mean = 0.f;
+    if (centered) {
+        mean = block_sum(sum, scratch) / (float)width;
+        sq = 0.f;
+#pragma unroll
+        for (int m = 0; m < STREAM_ITEMS; ++m) {
+            if ((m * blockDim.x + threadIdx.x) * VEC >= width) break;
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) sq += (x[m][i] - mean) * (x[m][i] - mean);
+        }
+    }
+    const float inv = 1.f / sqrtf(block_sum(sq, scratch + 32) / (float)width + eps);
+#pragma unroll
+    for (int m = 0; m < STREAM_ITEMS; ++m) {
+        const int c = (m * blockDim.x + threadIdx.x) * VEC;
+        if (c >= width) break;
+        alignas(16) T o[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; i += 4) {
+            const float4 w = *reinterpret_cast<const float4*>(w_open + c + i);
+            o[i] = from_float<T>((x[m][i] - mean) * inv * w.x);
+            o[i + 1] = from_float<T>((x[m][i + 1] - mean) * inv * w.y);
+            o[i + 2] = from_float<T>((x[m][i + 2] - mean) * inv * w.z);
+            o[i + 3] = from_float<T>((x[m][i + 3] - mean) * inv * w.w);
+        }
+        *reinterpret_cast<uint4*>(out + (long long)r * width + c) = *reinterpret_cast<const uint4*>(o);
+    }
+}
+
+template <typename T>
+static void launch_stream_add_norm(const void* branch, const void* branch2, float scale, float scale2, float* stream, const float* w_open,
+                                   void* out, const int* rows, int count, int width, float eps, int write, int centered, cudaStream_t s) {
+    constexpr int VEC = 16 / sizeof(T);
+    const int items = width / VEC;                // spread evenly: as many threads as take the row in the fewest rounds
+    const int rounds = count <= 512 ? (items + 255) / 256 : (items + 127) / 128 <= STREAM_ITEMS ? (items + 127) / 128 : (items + 255) / 256;
+    const int threads = ((items + rounds - 1) / rounds + 31) / 32 * 32;
+    stream_add_norm_kernel<T><<<count, threads, 0, s>>>((const T*)branch, (const T*)branch2, scale, scale2, stream, w_open, (T*)out,
+                                                        rows, width, eps, write, centered);
+}
+
 TS_API int ts_stream_norm(const void* branch, const float* w_close, float* stream, const float* w_open, void* out,
                           const int* rows, int count, int width, float eps, const void* table, const int* ids,
                           int table_rows, float scale, int flags, int dtype, const int* positions, const float* pos_freq,
@@ -206,6 +289,16 @@ TS_API int ts_stream_norm(const void* branch, const float* w_close, float* strea
     const BranchPair pair{branch2, w_branch, w_branch2, branch_scale, branch_scale2};
     const PairTable pairs{pair_table, prev_tokens, cu_q, seq_of_token, buckets, mul_prev, mul_cur};
     const int write = rows ? 0 : 1;
+    const int vec = dtype == TS_F32 ? 4 : 8;
+    const uintptr_t all = (uintptr_t)branch | (uintptr_t)branch2 | (uintptr_t)stream | (uintptr_t)w_open | (uintptr_t)out;
+    if (branch && (flags & TS_NORM_PLAIN_ADD) && !w_branch && w_open && width % vec == 0 && width / vec <= 256 * STREAM_ITEMS &&
+        all % 16 == 0 && (dtype == TS_F32 || dtype == TS_BF16)) {
+        const int centered = flags & TS_NORM_CENTERED;
+        if (dtype == TS_F32) launch_stream_add_norm<float>(branch, branch2, branch_scale, branch_scale2, stream, w_open, out, rows, count, width, eps, write, centered, stream_handle);
+        else launch_stream_add_norm<__nv_bfloat16>(branch, branch2, branch_scale, branch_scale2, stream, w_open, out, rows, count, width, eps, write, centered, stream_handle);
+        TS_LAUNCH_CHECK("stream_norm (add)");
+        return 0;
+    }
 #define TS_STREAM_NORM(TYPE)                                                                                      \
     do {                                                                                                          \
         if (smem > 48 * 1024)                                                                                     \

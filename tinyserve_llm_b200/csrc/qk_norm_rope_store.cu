@@ -34,12 +34,19 @@ struct QKPrepareArgs {
     const void* v_mix; long long v_mix_stride; float v_lambda;
 };
 
-template <typename T>
+// VEC (1 or 2) neighbouring channels a lane: 2 where head sizes, half the rotation and all offsets are even.
+template <typename T, int VEC>
+struct alignas(sizeof(T) * VEC) Pack {
+    T v[VEC];
+};
+
+template <typename T, int VEC>
 __global__ void qk_norm_rope_store_kernel(QKPrepareArgs p) {
     __shared__ float scratch[32];
+    extern __shared__ float turn[];                   // cos, then sin, of the token's rot / 2 angles, times the magnitude
     const int t = blockIdx.x;
     const int seq = p.seq_of_token[t];
-    const int nq = p.heads * p.dim, nk = p.kv_heads * p.dim, nv = p.v_heads * p.vdim;
+    const int nq = p.heads * p.dim, nk = p.kv_heads * p.dim;
     T* q_out = (T*)p.q_out + (long long)t * nq;
     if (seq < 0) {                                    // a padding row
         for (int e = threadIdx.x; e < nq; e += blockDim.x) q_out[e] = from_float<T>(0.f);
@@ -51,28 +58,16 @@ __global__ void qk_norm_rope_store_kernel(QKPrepareArgs p) {
     const T* yv = row + p.v_off;
     // what does not depend on the sums is asked for first: the position and the page
     const int pos = p.positions[t];
-    const int half = p.rot / 2;
+    const int half = p.freq ? p.rot / 2 : 0, rot = 2 * half;
     const int page = p.writes ? p.block_table[(long long)seq * p.table_width + pos / p.k_geo.page_tokens] : -1;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {        // one sine and cosine an angle, for all heads
+        float sn, cs;
+        sincosf((float)pos * p.freq[i], &sn, &cs);
+        turn[i] = cs * p.magnitude;
+        turn[half + i] = sn * p.magnitude;
+    }
     float inv_q = 1.f, inv_k = 1.f;
-    extern __shared__ float inv_heads[];              // norm_per_head: 1 / rms of every q head, then of every k head
-    if (p.norm_per_head && (p.q_weight || p.k_weight || p.unweighted)) {
-        const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
-        for (int hh = warp; hh < p.heads + p.kv_heads; hh += nwarps) {      // a warp a head
-            const bool is_q = hh < p.heads;
-            const int e0 = (is_q ? hh : hh - p.heads) * p.dim;
-            const T* y = is_q ? yq : yk;
-            const float* bias = is_q ? p.q_bias : p.k_bias;
-            float acc = 0.f;
-            if (p.unweighted || (is_q ? p.q_weight != nullptr : p.k_weight != nullptr))
-                for (int i = lane; i < p.dim; i += 32) {
-                    const float x = to_float<T>(y[e0 + i]) + (bias ? bias[e0 + i] : 0.f);
-                    acc += x * x;
-                }
-            acc = warp_sum(acc);
-            if (lane == 0) inv_heads[hh] = 1.f / sqrtf(acc / (float)p.dim + p.eps);
-        }
-        __syncthreads();
-    } else if (p.q_weight || p.k_weight) {            // both sums in one pass over the row, then two reductions
+    if (!p.norm_per_head && (p.q_weight || p.k_weight)) {         // both sums in one pass over the row, then two reductions
         float acc_q = 0.f, acc_k = 0.f;
         if (p.q_weight)
             for (int e = threadIdx.x; e < nq; e += blockDim.x) {
@@ -90,52 +85,99 @@ __global__ void qk_norm_rope_store_kernel(QKPrepareArgs p) {
         }
         if (p.k_weight) inv_k = 1.f / sqrtf(block_sum(acc_k, scratch) / (float)nk + p.eps);
     }
-    // `heads_at`: where this projection's heads start in inv_heads; `gain` multiplies every element (the query's temperature)
-    auto element = [&](const T* y, const float* bias, const float* weight, float inv, int heads_at, float gain, int e) {
-        const float x = to_float<T>(y[e]) + (bias ? bias[e] : 0.f);
-        if (p.unweighted) return x * inv_heads[heads_at + e / p.dim] * gain;
-        if (!weight) return x * gain;
-        if (p.norm_per_head) return x * inv_heads[heads_at + e / p.dim] * weight[e % p.dim] * gain;
-        return x * inv * weight[e] * gain;
-    };
+    __syncthreads();                                  // turn
     const float temperature = p.temp_every > 0
         ? 1.f + p.temp_coef * logf((float)((pos + 1) / p.temp_every) + 1.f) : 1.f;
-    // One thread a rotated pair (i, i + rot/2): one sincosf for both; channels past `rot` pass unchanged.
-    auto rotate_into = [&](const T* y, const float* bias, const float* weight, float inv, int heads_at, float gain, int n,
-                           auto&& store) {
-        for (int e = threadIdx.x; e < n; e += blockDim.x) {
-            const int i = e % p.dim;
-            if (p.freq && i < p.rot) {
-                if (p.interleaved ? (i & 1) : i >= half) continue;                 // written by the pair's first channel
-                const int other = p.interleaved ? e + 1 : e + half;
-                const float u = element(y, bias, weight, inv, heads_at, gain, e);
-                const float v = element(y, bias, weight, inv, heads_at, gain, other);
-                float sn, cs;
-                sincosf((float)pos * p.freq[p.interleaved ? i >> 1 : i], &sn, &cs);
-                sn *= p.magnitude;
-                cs *= p.magnitude;
-                store(e, u * cs - v * sn);
-                store(other, v * cs + u * sn);
-            } else {
-                store(e, element(y, bias, weight, inv, heads_at, gain, e));
+    const bool stores = p.writes && page >= 0 && page < p.k_geo.num_pages;
+    const int slot = pos % p.k_geo.page_tokens;
+    T* kp = stores ? (T*)p.k_pool + (long long)page * p.k_geo.page_stride + p.k_geo.entry_offset : nullptr;
+    T* vp = stores ? (T*)p.v_pool + (long long)page * p.v_geo.page_stride + p.v_geo.entry_offset : nullptr;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+    for (int hh = warp; hh < p.heads + (stores ? p.kv_heads : 0); hh += nwarps) {     // a warp a head of q or k
+        const bool is_q = hh < p.heads;
+        const int h = is_q ? hh : hh - p.heads, e0 = h * p.dim;
+        const T* y = (is_q ? yq : yk) + e0;
+        const float* bias = is_q ? p.q_bias : p.k_bias;
+        if (bias) bias += e0;
+        const float* weight = is_q ? p.q_weight : p.k_weight;
+        if (weight && !p.norm_per_head) weight += e0;
+        T* dst = is_q ? q_out + e0 : kp + ((long long)h * p.k_geo.page_tokens + slot) * p.dim;
+        auto load = [&](int i, float (&x)[VEC]) {
+            const Pack<T, VEC> raw = *reinterpret_cast<const Pack<T, VEC>*>(y + i);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) x[j] = to_float<T>(raw.v[j]) + (bias ? bias[i + j] : 0.f);
+        };
+        float gain = is_q ? temperature : 1.f;
+        if (p.norm_per_head) {
+            if (weight || p.unweighted) {
+                float acc = 0.f, x[VEC];
+                for (int i = lane * VEC; i < p.dim; i += 32 * VEC) {
+                    load(i, x);
+#pragma unroll
+                    for (int j = 0; j < VEC; ++j) acc += x[j] * x[j];
+                }
+                gain *= 1.f / sqrtf(warp_sum(acc) / (float)p.dim + p.eps);
+            }
+        } else if (weight) {
+            gain *= is_q ? inv_q : inv_k;
+        }
+        auto element = [&](int i, float (&x)[VEC]) {
+            load(i, x);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) x[j] *= weight ? gain * weight[i + j] : gain;
+        };
+        auto store = [&](int i, const float (&x)[VEC]) {
+            Pack<T, VEC> raw;
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) raw.v[j] = from_float<T>(x[j]);
+            *reinterpret_cast<Pack<T, VEC>*>(dst + i) = raw;
+        };
+        if (p.interleaved) {                          // channels 2i and 2i + 1
+            for (int i = lane; i < half; i += 32) {
+                float u[2];
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+                    u[j] = (to_float<T>(y[2 * i + j]) + (bias ? bias[2 * i + j] : 0.f)) * (weight ? gain * weight[2 * i + j] : gain);
+                dst[2 * i] = from_float<T>(u[0] * turn[i] - u[1] * turn[half + i]);
+                dst[2 * i + 1] = from_float<T>(u[1] * turn[i] + u[0] * turn[half + i]);
+            }
+        } else {
+            for (int i = lane * VEC; i < half; i += 32 * VEC) {
+                float u[VEC], v[VEC], a[VEC], b[VEC];
+                element(i, u);
+                element(i + half, v);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) {
+                    a[j] = u[j] * turn[i + j] - v[j] * turn[half + i + j];
+                    b[j] = v[j] * turn[i + j] + u[j] * turn[half + i + j];
+                }
+                store(i, a);
+                store(i + half, b);
             }
         }
-    };
-    rotate_into(yq, p.q_bias, p.q_weight, inv_q, 0, temperature, nq, [&](int e, float x) { q_out[e] = from_float<T>(x); });
-    if (!p.writes || page < 0 || page >= p.k_geo.num_pages) return;
-    const int slot = pos % p.k_geo.page_tokens;
-    T* kp = (T*)p.k_pool + (long long)page * p.k_geo.page_stride + p.k_geo.entry_offset;
-    T* vp = (T*)p.v_pool + (long long)page * p.v_geo.page_stride + p.v_geo.entry_offset;
-    rotate_into(yk, p.k_bias, p.k_weight, inv_k, p.heads, 1.f, nk, [&](int e, float x) {
-        const int h = e / p.dim, i = e % p.dim;
-        kp[((long long)h * p.k_geo.page_tokens + slot) * p.dim + i] = from_float<T>(x);
-    });
+        for (int i = rot + lane * VEC; i < p.dim; i += 32 * VEC) {       // channels past the rotation
+            float x[VEC];
+            element(i, x);
+            store(i, x);
+        }
+    }
+    if (!stores) return;
     const T* mix = p.v_mix ? (const T*)p.v_mix + (long long)t * p.v_mix_stride : nullptr;
-    for (int e = threadIdx.x; e < nv; e += blockDim.x) {
-        const int h = e / p.vdim, i = e % p.vdim;
-        float v = to_float<T>(yv[e]) + (p.v_bias ? p.v_bias[e] : 0.f);
-        if (mix) v = (1.f - p.v_lambda) * v + p.v_lambda * to_float<T>(mix[e]);
-        vp[((long long)h * p.v_geo.page_tokens + slot) * p.vdim + i] = from_float<T>(v);
+    for (int h = warp; h < p.v_heads; h += nwarps) {
+        T* dst = vp + ((long long)h * p.v_geo.page_tokens + slot) * p.vdim;
+        const int e0 = h * p.vdim;
+        for (int i = lane * VEC; i < p.vdim; i += 32 * VEC) {
+            const Pack<T, VEC> raw = *reinterpret_cast<const Pack<T, VEC>*>(yv + e0 + i);
+            Pack<T, VEC> other{}, o;
+            if (mix) other = *reinterpret_cast<const Pack<T, VEC>*>(mix + e0 + i);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) {
+                float v = to_float<T>(raw.v[j]) + (p.v_bias ? p.v_bias[e0 + i + j] : 0.f);
+                if (mix) v = (1.f - p.v_lambda) * v + p.v_lambda * to_float<T>(other.v[j]);
+                o.v[j] = from_float<T>(v);
+            }
+            *reinterpret_cast<Pack<T, VEC>*>(dst + i) = o;
+        }
     }
 }
 
@@ -161,13 +203,23 @@ TS_API int ts_qk_norm_rope_store(const void* y, long long y_stride, int q_off, i
                     KVGeometry{v_page_stride, v_entry_offset, page_tokens, num_pages}, block_table, table_width, writes,
                     heads, kv_heads, dim, vdim, value_heads > 0 ? value_heads : kv_heads, norm_per_head, temp_coef, temp_every,
                     unweighted, interleaved, v_mix, v_mix_stride, v_lambda};
-    const size_t smem = norm_per_head ? (size_t)(heads + kv_heads) * sizeof(float) : 0;
-    TS_REQUIRE(smem <= 32 * 1024, "qk_norm_rope_store: %d heads are not supported", heads + kv_heads);
+    const size_t smem = (size_t)(p.freq ? rot : 0) * sizeof(float);
+    TS_REQUIRE(smem <= 32 * 1024, "qk_norm_rope_store: rotation over %d channels is not supported", rot);
+    const bool even = dim % 2 == 0 && vdim % 2 == 0 && (interleaved || (rot / 2) % 2 == 0) && y_stride % 2 == 0 && q_off % 2 == 0 &&
+                      k_off % 2 == 0 && v_off % 2 == 0 && v_mix_stride % 2 == 0 && k_page_stride % 2 == 0 && k_entry_offset % 2 == 0 &&
+                      v_page_stride % 2 == 0 && v_entry_offset % 2 == 0 &&
+                      ((uintptr_t)y | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)v_mix) % 8 == 0;
     // many tokens: small CTAs, many of them on an SM (a CTA's life is a chain of loads and two sums); few tokens: wide ones
     const int threads = num_tokens >= 512 ? 128 : (heads * dim >= 2048 ? 512 : 256);
-    if (dtype == TS_F32) qk_norm_rope_store_kernel<float><<<num_tokens, threads, smem, stream>>>(p);
-    else if (dtype == TS_BF16) qk_norm_rope_store_kernel<__nv_bfloat16><<<num_tokens, threads, smem, stream>>>(p);
+#define TS_QK_PREPARE(T)                                                                          \
+    do {                                                                                          \
+        if (even) qk_norm_rope_store_kernel<T, 2><<<num_tokens, threads, smem, stream>>>(p);      \
+        else qk_norm_rope_store_kernel<T, 1><<<num_tokens, threads, smem, stream>>>(p);           \
+    } while (0)
+    if (dtype == TS_F32) TS_QK_PREPARE(float);
+    else if (dtype == TS_BF16) TS_QK_PREPARE(__nv_bfloat16);
     else return ts_fail("qk_norm_rope_store: unknown dtype code %d", dtype);
+#undef TS_QK_PREPARE
     TS_LAUNCH_CHECK("qk_norm_rope_store");
     return 0;
 }

@@ -190,6 +190,8 @@ class Ops:
         self.swiglu_skinny_rows = self.skinny_max_rows
         # TINYSERVE_B200_TILES=0 keeps the recurrences that have a form of sixteen tokens at a time on the scan token by token
         self.recurrence_tiles = os.environ.get("TINYSERVE_B200_TILES", "1") != "0"
+        # TINYSERVE_B200_OVERLAP=0 keeps a replayed step's kernels on one stream (see parts/overlap.py)
+        self.overlap = os.environ.get("TINYSERVE_B200_OVERLAP", "1") != "0"
         # TINYSERVE_B200_LRU=split keeps a gated linear recurrent unit's decode steps on the kernels of prompt portions
         self.lru_fused_decode = os.environ.get("TINYSERVE_B200_LRU", "fused") != "split"
         # from this many (token, expert) pairs a routed feed-forward's bfloat16 products go to the library's grouped product

@@ -13,6 +13,7 @@ from __future__ import annotations
 import torch
 
 from tinyserve_llm_b200.config.spec import BlockSpec
+from tinyserve_llm_b200.parts import overlap
 from tinyserve_llm_b200.parts.base import Runtime, TensorDecl, part_class, register_arrangement
 
 
@@ -237,7 +238,7 @@ class ParallelStreamBlock:
     """
     h = norm(x); x = x + branch_scale * (mixer(h) + ffn(h)) around a residual stream kept in float32: the two
     sublayers' outputs travel on as one `PendingBranch`, and the next norm of the stream adds both to it and norms
-    the sum in one kernel.  A block without a feed-forward adds its mixer's output alone.
+    the sum in one kernel.  In a step replayed from a graph the two run side by side.  A block without a feed-forward adds its mixer's output alone.
     """
 
     takes_token_ids = True
@@ -279,6 +280,12 @@ class ParallelStreamBlock:
                                                            pairs=embedding_pairs, ctx=ctx)
         else:
             h, residual = self.mixer_norm.forward(x, residual)
+        fed = None
+        if self.feed_forward is not None:
+            side = overlap.fork(self.mixer.rt, ctx, "feed-forward")
+            with overlap.on(side):
+                fed = self.feed_forward.forward(h, ctx)
         mixed = self.mixer.forward(h, ctx, binding)
-        fed = self.feed_forward.forward(h, ctx) if self.feed_forward is not None else None
+        if self.feed_forward is not None:
+            overlap.join(side)
         return PendingBranch.scaled_sum(mixed, fed, self.spec.branch_scale), residual

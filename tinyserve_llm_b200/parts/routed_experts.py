@@ -26,6 +26,7 @@ from __future__ import annotations
 import torch
 
 from tinyserve_llm_b200.config.spec import GatedMLPSpec, RoutedExpertsSpec
+from tinyserve_llm_b200.parts import overlap
 from tinyserve_llm_b200.parts.base import FeedForward, Runtime, TensorDecl, part_class, register_part
 from tinyserve_llm_b200.parts.linear import Linear
 
@@ -94,6 +95,11 @@ class RoutedExperts(FeedForward):
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         spec, ops = self.spec, self.rt.ops
         T, top = x.shape[0], spec.top
+        shared = None
+        if self.shared is not None:                        # beside the routed experts in a step replayed from a graph
+            side = overlap.fork(self.rt, ctx, "shared expert")
+            with overlap.on(side):
+                shared = self.shared.forward(x, ctx)
         logits = self.router(x, out_dtype=torch.float32)
         identity_share = None
         if spec.scoring == "softmax_all":
@@ -110,5 +116,6 @@ class RoutedExperts(FeedForward):
             hidden = ops.moe_linear(x, self.gate_up, offsets, pair_of_row, top, T * top, e.activation,
                                     row_scale=share if on_input else None)
         y = ops.moe_linear(hidden, self.down, offsets, None, top, T * top)
-        shared = self.shared.forward(x, ctx) if self.shared is not None else None
+        if self.shared is not None:
+            overlap.join(side)
         return ops.moe_combine(y, row_of_pair, None if on_input else share, shared, T, x=x, identity_share=identity_share)
