@@ -641,12 +641,12 @@ def test_pair_rows_follow_the_previous_token_across_steps_and_requests(dtype, bu
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("experts, top, shared, rows", [(7, 2, 24, 5), (5, 5, 0, 90), (33, 3, 40, 130), (2, 1, 16, 1)])
-def test_routed_experts_with_a_shared_one_alone(dtype, experts, top, shared, rows):
+@pytest.mark.parametrize("width, experts, top, shared, rows", [(64, 7, 2, 24, 5), (64, 5, 5, 0, 90), (64, 33, 3, 40, 130), (72, 2, 1, 16, 1),
+                                                               (320, 9, 3, 40, 40), (72, 40, 4, 8, 33)])
+def test_routed_experts_with_a_shared_one_alone(dtype, width, experts, top, shared, rows):
     from tinyserve_llm_b200.config.gimotar import GimotarConfig
     from tinyserve_llm_b200.parts.base import part_class
     from tinyserve_llm_b200.weights import random_tensors
-    width = 64
     raw = C.model(50, width, 1e-6, 1.0, 1.0, (5, 1, 1), [(C.rglru(16, 1, 2), C.moe(experts, top, 40, shared))])
     spec = GimotarConfig.from_dict(raw).feed_forward_spec(0)
     cls = part_class("feed_forward", spec)

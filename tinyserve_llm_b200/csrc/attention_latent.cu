@@ -371,43 +371,42 @@ TS_API int ts_latent_attention(const float* q_lat, long long ql_token_stride, lo
     return ts_fail("latent_attention: unknown dtype code %d", dtype);
 }
 
-// The queries' rotated parts for the unfolded form: out[t, h, 0 .. pitch) = rotated q[t, h * head_width + rot_offset ..],
+// The queries' rotated parts for the unfolded form: out[t, h, 0 .. 63] = rotated q[t, h * head_width + rot_offset ..],
 // zeros past `rot` channels; rotation by halves, angle position * freq[i] in float32, cos and sin times `magnitude`.
-__global__ void latent_rotate_queries_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, int head_width,
-                                             int rot_offset, const float* __restrict__ freq, float magnitude,
-                                             const int* __restrict__ positions, __nv_bfloat16* __restrict__ out, int heads,
-                                             int rot, int pitch) {
-    extern __shared__ float turn[];                       // cos, sin of the token's rot / 2 angles
-    const int t = blockIdx.x, half = rot / 2;
-    const float pos = (float)positions[t];
-    for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        float sn, cs;
-        sincosf(pos * freq[i], &sn, &cs);
-        turn[i] = cs * magnitude;
-        turn[half + i] = sn * magnitude;
+// A thread a pair of channels (i, i + rot / 2), the threads past the last pair write the zeros.
+__global__ void __launch_bounds__(256)
+latent_rotate_queries_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, int head_width, int rot_offset,
+                             const float* __restrict__ freq, float magnitude, const int* __restrict__ positions,
+                             __nv_bfloat16* __restrict__ out, int heads, int rot) {
+    const int t = blockIdx.x, half = rot / 2, i = threadIdx.x & 31;
+    float sn = 0.f, cs = 0.f;
+    if (i < half) {                                       // a thread keeps its pair of channels over all heads
+        sincosf((float)positions[t] * freq[i], &sn, &cs);
+        sn *= magnitude;
+        cs *= magnitude;
     }
-    __syncthreads();
-    for (int e = threadIdx.x; e < heads * pitch; e += blockDim.x) {
-        const int h = e / pitch, c = e % pitch;
-        float x = 0.f;
-        if (c < rot) {
-            const __nv_bfloat16* src = q + (long long)t * q_stride + (long long)h * head_width + rot_offset;
-            const int i = c < half ? c : c - half;
-            const float u = __bfloat162float(src[i]), v = __bfloat162float(src[i + half]);
-            x = c < half ? u * turn[i] - v * turn[half + i] : v * turn[i] + u * turn[half + i];
+    const __nv_bfloat16* src = q + (long long)t * q_stride + rot_offset + i;
+    __nv_bfloat16* dst = out + (long long)t * heads * 64;
+    for (int h = threadIdx.x >> 5; h < heads; h += 8) {
+        if (i < half) {
+            const float u = __bfloat162float(src[(long long)h * head_width]), v = __bfloat162float(src[(long long)h * head_width + half]);
+            dst[h * 64 + i] = __float2bfloat16_rn(u * cs - v * sn);
+            dst[h * 64 + i + half] = __float2bfloat16_rn(v * cs + u * sn);
+        } else {
+            const int c = rot + 2 * (i - half);
+            dst[h * 64 + c] = dst[h * 64 + c + 1] = __float2bfloat16_rn(0.f);
         }
-        out[(long long)t * heads * pitch + e] = __float2bfloat16_rn(x);
     }
 }
 
 TS_API int ts_latent_rotate_queries(const void* q, long long q_stride, int head_width, int rot_offset, const float* freq,
                                     float magnitude, const int* positions, void* out, int num_tokens, int heads, int rot,
-                                    int pitch, cudaStream_t stream) {
-    TS_REQUIRE(num_tokens >= 0 && heads > 0 && rot > 0 && rot % 2 == 0 && rot <= pitch && rot_offset + rot <= head_width,
+                                    cudaStream_t stream) {
+    TS_REQUIRE(num_tokens >= 0 && heads > 0 && rot > 0 && rot % 2 == 0 && rot <= 64 && rot_offset + rot <= head_width,
                "latent_rotate_queries: bad sizes");
     if (num_tokens == 0) return 0;
-    latent_rotate_queries_kernel<<<num_tokens, 256, rot * sizeof(float), stream>>>(
-        (const __nv_bfloat16*)q, q_stride, head_width, rot_offset, freq, magnitude, positions, (__nv_bfloat16*)out, heads, rot, pitch);
+    latent_rotate_queries_kernel<<<num_tokens, 256, 0, stream>>>((const __nv_bfloat16*)q, q_stride, head_width, rot_offset, freq,
+                                                                 magnitude, positions, (__nv_bfloat16*)out, heads, rot);
     TS_LAUNCH_CHECK("latent_rotate_queries");
     return 0;
 }

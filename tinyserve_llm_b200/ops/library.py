@@ -34,7 +34,7 @@ _SIGNATURES = {
     "ts_paged_attention_bf16_masked": ("int", "pl" "ppp" "lllliipippiiiiiiifiifi" "plpi" "fp"),
     "ts_attention_tcgen05_supported": ("int", "iiiii"),
     "ts_prefill_attention_tcgen05_dense": ("int", "pl" "ppp" "lpppiiiiiifpip" "ipplip" "p"),
-    "ts_latent_rotate_queries": ("int", "pliipfppiiiip"),
+    "ts_latent_rotate_queries": ("int", "pliipfppiiip"),
     "ts_prefill_attention_tcgen05_masked": ("int", "pl" "ppp" "iiiipippiiiiiifiifi" "pipfp"),
     "ts_prefill_attention_tcgen05": ("int", "ppppiiiipippiiiiiifpipp"),
     "ts_prefill_attention_tcgen05_sigmoid": ("int", "pl" "ppp" "iiiipippiiiiiifi" "pppl" "pipp"),
@@ -879,7 +879,7 @@ class Ops:
             raise KernelError(f"latent_rotate_queries: q {tuple(q.shape)} {q.dtype}, {heads} heads of {head_width}, rotation over {rot}")
         out = torch.empty((q.shape[0], heads * 64), dtype=q.dtype, device=q.device)
         self._call("ts_latent_rotate_queries", _ptr(q), q.stride(0), head_width, rot_offset, _ptr(freq), float(magnitude),
-                   _ptr(ctx.positions), _ptr(out), q.shape[0], heads, rot, 64, _stream())
+                   _ptr(ctx.positions), _ptr(out), q.shape[0], heads, rot, _stream())
         return out
 
     def tensor_core_attention(self, q: torch.Tensor, binding, nh: int, nkv: int, hd: int, vd: int, ctx=None) -> bool:

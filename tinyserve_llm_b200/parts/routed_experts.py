@@ -30,6 +30,10 @@ from tinyserve_llm_b200.parts import overlap
 from tinyserve_llm_b200.parts.base import FeedForward, Runtime, TensorDecl, part_class, register_part
 from tinyserve_llm_b200.parts.linear import Linear
 
+# A shared expert of up to this many bytes of weights runs beside the routed ones in a replayed step; a larger one streams its
+# weights for as long as they do, and two such streams (three with a mixer beside them) only disturb one another.
+SHARED_BESIDE_BYTES = 48 << 20
+
 
 @register_part("feed_forward", "routed_experts")
 class RoutedExperts(FeedForward):
@@ -91,13 +95,15 @@ class RoutedExperts(FeedForward):
         if spec.shared is not None:
             sub = {k[len(spec.shared_prefix):]: v for k, v in tensors.items() if k.startswith(spec.shared_prefix)}
             self.shared = part_class("feed_forward", spec.shared)(spec.shared, sub, rt)
+            weights = sum(t.numel() for t in sub.values()) * rt.dtype.itemsize
+            self.shared_beside = weights <= SHARED_BESIDE_BYTES
 
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         spec, ops = self.spec, self.rt.ops
         T, top = x.shape[0], spec.top
         shared = None
         if self.shared is not None:                        # beside the routed experts in a step replayed from a graph
-            side = overlap.fork(self.rt, ctx, "shared expert")
+            side = overlap.fork(self.rt, ctx, "shared expert") if self.shared_beside else None
             with overlap.on(side):
                 shared = self.shared.forward(x, ctx)
         logits = self.router(x, out_dtype=torch.float32)
