@@ -727,12 +727,21 @@ def test_replay_program_on_a_model_folder(folders, tmp_path):
 
 
 @pytest.mark.parametrize("name", ["mixed", "latent", "recurrent"])
-def test_greedy_generation_through_the_entry_point(folders, name):
-    """LLM.generate with the scheduler, prompt portions, CUDA graphs and running ahead: the plain model's greedy tokens."""
+def test_greedy_generation_through_the_entry_point(name, tmp_path):
+    """
+    LLM.generate with the scheduler, prompt portions, CUDA graphs and running ahead: the plain model's greedy tokens.  The
+    token embedding is scaled down and the pair embedding up, so that a tied head does not answer every token with itself.
+    """
     from tinyserve_llm_b200 import LLM, CacheConfig, SamplingParams, SchedulerConfig
-    raw, folder = CONFIGS[name], folders[name, "float32"]
+    from tinyserve_llm_b200.weights.safetensors_io import write_safetensors
+    raw = copy.deepcopy(CONFIGS[name])
+    raw["embedding"]["scale"] = 0.05
+    folder = str(tmp_path / "model")
+    _write(folder, raw, SEEDS[name], C.WEIGHTS)
     tensors = read_tensors(folder)
-    prompts = [ids_of(raw["vocab"], n, 30 + n) for n in (3, 41, 18, 77, 1)]
+    tensors["bigram"] = tensors["bigram"] * 3
+    write_safetensors(os.path.join(folder, "model.safetensors"), tensors)
+    prompts = [ids_of(raw["vocab"], n, 130 + n) for n in (3, 41, 18, 77, 1)]
     new = 12
     want = []
     for p in prompts:
@@ -740,6 +749,7 @@ def test_greedy_generation_through_the_entry_point(folders, name):
         for _ in range(new):
             ids.append(int(plain.forward(raw, tensors, ids)[-1].argmax()))
         want.append(ids[len(p):])
+    assert min(len(set(w)) for w in want) > 3                             # the premise: the answers vary
     llm = LLM(folder, SchedulerConfig(max_model_len=128, max_num_seqs=3, max_num_batched_tokens=48, prefill_chunk=20),
               CacheConfig(block_size=16), dtype="float32", num_blocks=24, seed=0)
     for _ in range(2):                                                    # the second time over cached prefixes, where the model allows it
